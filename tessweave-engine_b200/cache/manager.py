@@ -1,7 +1,7 @@
 """The cache manager: pages of keys and values, block tables, prefix sharing, state slots.
 
-Layers are sorted into *groups* by what they need: all keys of a request, or a
-window of them (per head count and head size).  Every group has its own pool of
+Layers are sorted into *groups* by what they need: all keys of a request, a window
+of them, or those of the chunk being filled (per head count and head size).  Every group has its own pool of
 pages, its own reference counts and free list, and its own block table per
 request; a page of a group holds the keys and values of *every* layer of that
 group for ``page_size`` consecutive tokens.  Pages go back to the free list when a
@@ -127,7 +127,7 @@ class CacheManager:
         # ---- request slots and the prefix index
         self.free_slots = list(reversed(range(max_requests)))
         self.leases: dict[int, Lease] = {}
-        shareable = bool(self.groups) and not self.state and all(g.window is None for g in self.groups)
+        shareable = bool(self.groups) and not self.state and all(g.need.span is None for g in self.groups)
         self.prefix_cache = bool(prefix_cache and shareable)
         self.prefixes: "OrderedDict[bytes, tuple[int, ...]]" = OrderedDict()   # key -> page per group
         self.hits = 0
@@ -216,12 +216,12 @@ class CacheManager:
     # ------------------------------------------------------------------ request life cycle
     def pages_needed(self, total_tokens: int, step_tokens: int = 1) -> list[int]:
         """Worst number of pages a request of ``total_tokens`` holds at a time, per group.
-        A windowed group never needs more than its window plus one step's tokens."""
+        A windowed group never needs more than its window (or its chunk) plus one step's tokens."""
         out = []
         for g in self.groups:
             full = math.ceil(total_tokens / self.page_size)
-            if g.window is not None:
-                full = min(full, math.ceil((g.window + step_tokens) / self.page_size) + 1)
+            if g.need.span is not None:
+                full = min(full, math.ceil((g.need.span + step_tokens) / self.page_size) + 1)
             out.append(full)
         return out
 
@@ -327,8 +327,8 @@ class CacheManager:
 
     def advance(self, lease: Lease, tokens, computed: int) -> None:
         """Tell the manager that ``computed`` tokens of the request are now in the cache:
-        full blocks become shareable, and pages that every later token's window has left
-        behind go back to the free list."""
+        full blocks become shareable, and pages that every later token's window (or the chunk
+        being filled) has left behind go back to the free list."""
         ps = self.page_size
         if self.prefix_cache and tokens is not None:
             full = min(computed, len(tokens)) // ps
@@ -346,10 +346,10 @@ class CacheManager:
                                 self.groups[gi].refs[page] += 1
                 lease.published_blocks = full
         for gi, g in enumerate(self.groups):
-            if g.window is None:
+            if g.need.span is None:
                 continue
-            # the next token sits at position `computed` and sees keys > computed - window
-            dead_before = max(0, computed - g.window + 1) // ps
+            # the next token sits at position `computed`: pages before the first key it sees are not read again
+            dead_before = g.need.first_needed(computed) // ps
             table = lease.tables[gi]
             for b in range(lease.first_live_block[gi], min(dead_before, len(table))):
                 if table[b] >= 0:

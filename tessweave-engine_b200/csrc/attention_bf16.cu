@@ -1,6 +1,9 @@
 // Paged grouped-query attention in bfloat16 on the tensor cores, for one head size
 // (compile with -DTW_HEAD_DIM=<multiple of 16, 16..256>).
 //
+// Values may have another size than queries and keys (-DTW_V_DIM=<multiple of 16>; default: the same); the output
+// then has heads of that size.
+//
 // Two kernels share the tile machinery:
 //   * decode:  requests that bring ONE token.  A block serves one (request, key/value head,
 //     slice of the keys); the query heads of the group are the columns of one MMA tile, so keys
@@ -18,7 +21,7 @@
 // bf16 only as the operand of the P.V product.  Keys beyond the visible range are never
 // read: their shared-memory rows are zero-filled, so stale page contents cannot leak in.
 //
-//   score = (q . k) * scale,  visible iff  position - window < p <= position
+//   score = (q . k) * scale,  visible iff  tw_first_key(position, window) <= p <= position
 // Reference: flow_engine/model.py:193-200 and flow_engine/kernels/paged_decode.py:13-43.
 #include "common.cuh"
 #include "attention_common.cuh"
@@ -29,23 +32,32 @@ namespace cg = cooperative_groups;
 #ifndef TW_HEAD_DIM
 #define TW_HEAD_DIM 128
 #endif
+#ifndef TW_V_DIM
+#define TW_V_DIM TW_HEAD_DIM
+#endif
 
 namespace {
 
 constexpr int D = TW_HEAD_DIM;
 static_assert(D % 16 == 0 && D >= 16 && D <= 256, "head size must be a multiple of 16 in 16..256");
+constexpr int DV = TW_V_DIM;     // size of a value, and of a head of the output
+static_assert(DV % 16 == 0 && DV >= 16 && DV <= 256, "value size must be a multiple of 16 in 16..256");
+constexpr bool SAME_DIMS = D == DV;
 constexpr int DP = D + 8;        // padded row: consecutive rows fall into different 16-byte bank groups
+constexpr int VP = DV + 8;       // the same for values
 constexpr int KSTEPS = D / 16;   // k-steps of Q.K^T
-constexpr int NT_O = D / 8;      // n-tiles of P.V
-constexpr int CHUNKS = D / 8;    // 16-byte chunks of a row
+constexpr int NT_O = DV / 8;     // n-tiles of P.V
+constexpr int CHUNKS = D / 8;    // 16-byte chunks of a row of q or k
+constexpr int VCHUNKS = DV / 8;  // 16-byte chunks of a row of v
+constexpr int DMAX = D > DV ? D : DV;
 constexpr float NEG_INF = -INFINITY;
 
 using namespace tw_attn;
 
-// Element offset of key p's row in the cache, or -1 if p is outside [first, limit) or has no page.  Keys before
+// Row of key p in the cache (in rows of D or DV values), or -1 if p is outside [first, limit) or has no page.  Keys before
 // `first` (the start of the earliest window of the block) are seen by no row, and their pages may have been
 // given back already: they are not looked up.
-__device__ __forceinline__ long long key_offset(int p, int first, int limit, const int* table, int table_stride, int page_size,
+__device__ __forceinline__ long long key_row(int p, int first, int limit, const int* table, int table_stride, int page_size,
                                                 int num_pages, int Hkv, int kvh, int* status) {
     if (p < first || p >= limit) return -1;
     const int blk = p / page_size;
@@ -54,7 +66,7 @@ __device__ __forceinline__ long long key_offset(int p, int first, int limit, con
         atomicOr(status, TW_ERR_PAGE);
         return -1;
     }
-    return (((long long)page * Hkv + kvh) * page_size + (p - blk * page_size)) * D;
+    return ((long long)page * Hkv + kvh) * page_size + (p - blk * page_size);
 }
 
 // ---------------------------------------------------------------------------------------
@@ -72,17 +84,18 @@ constexpr int DEC_WARPS = 4;
 constexpr int DEC_TILE = DEC_WARPS * 16;                      // keys per block and iteration
 constexpr int DEC_HEADS = 8;                                  // query heads per block (columns of the MMA)
 constexpr int DEC_STAGES = 3;                                 // V tiles of a warp in shared memory (2 in flight)
-constexpr int DEC_STAGE = 16 * DP;                            // elements of one warp stage of V
+constexpr int DEC_STAGE = 16 * VP;                            // elements of one warp stage of V
 constexpr int DEC_PAGE_CACHE = 256;                           // block-table entries kept in shared memory
 constexpr int DEC_SMEM_STAGES = DEC_WARPS * DEC_STAGES * DEC_STAGE * 2;
 constexpr int DEC_SMEM_OFFS = DEC_WARPS * DEC_STAGES * 16 * 8;  // row offsets of the tiles in flight
 constexpr int DEC_SMEM = DEC_SMEM_STAGES + DEC_SMEM_OFFS + DEC_PAGE_CACHE * 4;
+static_assert(DEC_STAGE * 2 % 16 == 0 && DEC_SMEM_STAGES % 16 == 0, "stages start on 16-byte boundaries");
 constexpr int DB32 = D / 32;                                  // whole 32-wide blocks of d
 constexpr bool DTAIL16 = (D % 32) != 0;                       // plus one 16-wide block
-constexpr int MT_O = D / 16;                                  // m-tiles of O^T
+constexpr int MT_O = DV / 16;                                 // m-tiles of O^T
 constexpr int DEC_MAX_CLUSTER = 16;                           // slices that can merge through distributed shared memory
 // after the last tile the stage buffers hold the warps' partial results and this block's merged slice
-static_assert((DEC_WARPS + 1) * DEC_HEADS * (D + 2) * 4 <= DEC_SMEM_STAGES, "merge area must fit the stage buffers");
+static_assert((DEC_WARPS + 1) * DEC_HEADS * (DV + 2) * 4 <= DEC_SMEM_STAGES, "merge area must fit the stage buffers");
 
 struct KFrag {                    // the d values of one key row this thread feeds to the MMAs
     uint4 blk[DB32 > 0 ? DB32 : 1];
@@ -111,7 +124,7 @@ __device__ __forceinline__ long long global_ns() {
 #endif
 
 template <bool CLUSTER, bool FUSED>
-__global__ void __launch_bounds__(DEC_WARPS * 32, (D <= 128 ? 4 : 2))
+__global__ void __launch_bounds__(DEC_WARPS * 32, (DMAX <= 128 ? 4 : 2))
 attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restrict__ q, int q_stride,
                    const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                    const int* __restrict__ seq_kv_len, const int* __restrict__ seq_slot,
@@ -123,6 +136,7 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
     // position's key and value through fq.k_cache / fq.v_cache, which are the same memory, and reads them back
     // below: that one key row with ld.global.cg (L2, coherent) and the values with cp.async.cg, never through
     // the non-coherent path, which may hold a line from before the write.
+    static_assert(!FUSED || SAME_DIMS, "the fused form packs q, k and v as heads of one size");
     extern __shared__ __align__(16) unsigned char smem_raw[];
     __shared__ int s_is_last;
     __shared__ float s_row_max[DEC_HEADS];
@@ -142,7 +156,7 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
     const int nheads = min(DEC_HEADS, G - h0);
     const int n = seq_q_start[s];
     const int pos = seq_kv_len[s] - 1;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = tw_first_key(pos, window);
     const int nkeys = pos + 1 - lo;
     const int per = ((nkeys + nsplit - 1) / nsplit + DEC_TILE - 1) / DEC_TILE * DEC_TILE;
     const int k_begin = lo + split * per;
@@ -234,17 +248,17 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
                     const int page = blk - first_blk < DEC_PAGE_CACHE ? page_cache[blk - first_blk]
                                                                       : (blk < table_stride ? table[blk] : -1);
                     if (page < 0 || page >= num_pages) atomicOr(status, TW_ERR_PAGE);
-                    else off = (((long long)page * Hkv + kvh) * page_size + (p - blk * page_size)) * D;
+                    else off = ((long long)page * Hkv + kvh) * page_size + (p - blk * page_size);
                 }
                 offs[lane] = off;
             }
             __syncwarp();
             bf16* vs_ = stage_base + st * DEC_STAGE;
 #pragma unroll
-            for (int i = lane; i < 16 * CHUNKS; i += 32) {
-                const int row = i / CHUNKS, col = i - row * CHUNKS;
+            for (int i = lane; i < 16 * VCHUNKS; i += 32) {
+                const int row = i / VCHUNKS, col = i - row * VCHUNKS;
                 const long long off = offs[row];
-                cp_async16(vs_ + row * DP + col * 8, v_cache + (off >= 0 ? off + col * 8 : 0), off >= 0 ? 16 : 0);
+                cp_async16(vs_ + row * VP + col * 8, v_cache + (off >= 0 ? off * DV + col * 8 : 0), off >= 0 ? 16 : 0);
             }
         }
         cp_async_commit();      // one group per tile slot, empty past the end, so the wait count is constant
@@ -253,7 +267,8 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
     // Keys that earlier steps wrote come through the read-only path (ld.global.nc).  With FUSED the row of the
     // newest position was written by this very block a moment ago: it alone is read with ld.global.cg, because
     // the read-only path may still hold its line from before the write.
-    auto load_row = [&](long long off, bool fresh, KFrag& k) {
+    auto load_row = [&](long long row, bool fresh, KFrag& k) {
+        const long long off = row < 0 ? -1 : row * D;
 #pragma unroll
         for (int jb = 0; jb < DB32; ++jb) {
             const uint4* p = reinterpret_cast<const uint4*>(k_cache + off + 32 * jb + 8 * c);
@@ -410,7 +425,7 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
 #pragma unroll
             for (int mt = 0; mt < MT_O; ++mt) {
                 uint32_t a[4];
-                ldmatrix_x4_trans(a, vs_ + ((j >> 1) * 8 + r) * DP + mt * 16 + (j & 1) * 8);
+                ldmatrix_x4_trans(a, vs_ + ((j >> 1) * 8 + r) * VP + mt * 16 + (j & 1) * 8);
                 mma_bf16_regs(oacc[mt], a[0], a[1], a[2], a[3], pb0, pb1);
             }
         }
@@ -431,13 +446,13 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
 
     // merge the warps through shared memory (the stage buffers are free now)
     __syncthreads();
-    float* mo = reinterpret_cast<float*>(smem_raw);              // [warps][heads][D]
-    float* mml = mo + DEC_WARPS * DEC_HEADS * D;                 // [warps][heads][2]
+    float* mo = reinterpret_cast<float*>(smem_raw);              // [warps][heads][DV]
+    float* mml = mo + DEC_WARPS * DEC_HEADS * DV;                // [warps][heads][2]
 #pragma unroll
     for (int mt = 0; mt < MT_O; ++mt) {
         const int d = mt * 16 + g;
-        float* p0 = mo + (warp * DEC_HEADS + 2 * c) * D;
-        float* p1 = p0 + D;
+        float* p0 = mo + (warp * DEC_HEADS + 2 * c) * DV;
+        float* p1 = p0 + DV;
         p0[d] = oacc[mt][0]; p1[d] = oacc[mt][1];
         p0[d + 8] = oacc[mt][2]; p1[d + 8] = oacc[mt][3];
     }
@@ -445,11 +460,11 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
         mml[(warp * DEC_HEADS + 2 * c) * 2] = m0; mml[(warp * DEC_HEADS + 2 * c) * 2 + 1] = l0;
         mml[(warp * DEC_HEADS + 2 * c + 1) * 2] = m1; mml[(warp * DEC_HEADS + 2 * c + 1) * 2 + 1] = l1;
     }
-    float* part_o = mml + DEC_WARPS * DEC_HEADS * 2;             // [heads][D]: this block's slice, for the cluster
-    float* part_ml = part_o + DEC_HEADS * D;                     // [heads][2]
+    float* part_o = mml + DEC_WARPS * DEC_HEADS * 2;             // [heads][DV]: this block's slice, for the cluster
+    float* part_ml = part_o + DEC_HEADS * DV;                    // [heads][2]
     __syncthreads();
-    for (int idx = threadIdx.x; idx < nheads * D; idx += DEC_WARPS * 32) {
-        const int row = idx / D, d = idx - row * D;
+    for (int idx = threadIdx.x; idx < nheads * DV; idx += DEC_WARPS * 32) {
+        const int row = idx / DV, d = idx - row * DV;
         float M = NEG_INF;
 #pragma unroll
         for (int w = 0; w < DEC_WARPS; ++w) M = fmaxf(M, mml[(w * DEC_HEADS + row) * 2]);
@@ -460,19 +475,20 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
                 const float mw = mml[(w * DEC_HEADS + row) * 2];
                 const float f = mw == NEG_INF ? 0.f : exp2f(mw - M);
                 L += mml[(w * DEC_HEADS + row) * 2 + 1] * f;
-                o += mo[(w * DEC_HEADS + row) * D + d] * f;
+                o += mo[(w * DEC_HEADS + row) * DV + d] * f;
             }
         }
         const int head = kvh * G + h0 + row;
         if (nsplit == 1) {
             if (terms.sink) L += exp2f(__ldg(terms.sink + head) * LOG2E - M);
-            out[(size_t)n * out_stride + (size_t)head * D + d] = __float2bfloat16_rn(L > 0.f ? o / L : 0.f);
+            out[(size_t)n * out_stride + (size_t)head * DV + d] =
+                __float2bfloat16_rn(L > 0.f ? o / L * head_gate(terms.gate, n, Hq, head) : 0.f);
         } else if (CLUSTER) {
-            part_o[row * D + d] = o;
+            part_o[row * DV + d] = o;
             if (d == 0) { part_ml[row * 2] = M; part_ml[row * 2 + 1] = L; }
         } else {
             const size_t base = ((size_t)s * Hq + head) * nsplit + split;
-            partial_o[base * D + d] = o;
+            partial_o[base * DV + d] = o;
             if (d == 0) { partial_ml[base * 2] = M; partial_ml[base * 2 + 1] = L; }
         }
     }
@@ -486,8 +502,8 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
         cg::cluster_group cluster = cg::this_cluster();
         TW_DTRACE(8);
         cluster.sync();
-        for (int idx = split * (DEC_WARPS * 32) + threadIdx.x; idx < nheads * D; idx += nsplit * (DEC_WARPS * 32)) {
-            const int row = idx / D, d = idx - row * D;
+        for (int idx = split * (DEC_WARPS * 32) + threadIdx.x; idx < nheads * DV; idx += nsplit * (DEC_WARPS * 32)) {
+            const int row = idx / DV, d = idx - row * DV;
             float M = NEG_INF;
             for (int i = 0; i < nsplit; ++i) M = fmaxf(M, *cluster.map_shared_rank(part_ml + row * 2, i));
             float L = 0.f, o = 0.f;
@@ -496,10 +512,11 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
                 const float mi = ml[0];
                 const float f = (mi == NEG_INF || M == NEG_INF) ? 0.f : exp2f(mi - M);
                 L += ml[1] * f;
-                o += *cluster.map_shared_rank(part_o + row * D + d, i) * f;
+                o += *cluster.map_shared_rank(part_o + row * DV + d, i) * f;
             }
             if (terms.sink) L += exp2f(__ldg(terms.sink + kvh * G + h0 + row) * LOG2E - M);
-            out[(size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * D + d] = __float2bfloat16_rn(L > 0.f ? o / L : 0.f);
+            out[(size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * DV + d] =
+                __float2bfloat16_rn(L > 0.f ? o / L * head_gate(terms.gate, n, Hq, kvh * G + h0 + row) : 0.f);
         }
         cluster.sync();          // nobody leaves while a neighbour may still read its shared memory
         TW_DTRACE(9);
@@ -546,11 +563,11 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
     __syncthreads();
     // four values of d per thread and eight slices in flight at once: the merge is a chain of
     // L2 round trips on one block while the rest of the GPU waits, so it is kept short
-    constexpr int D4 = D / 4;
+    constexpr int D4 = DV / 4;
     for (int idx = threadIdx.x; idx < nheads * D4; idx += DEC_WARPS * 32) {
         const int row = idx / D4, d4 = idx - row * D4;
         const float* f = fac + row * nsplit;
-        const float4* po = reinterpret_cast<const float4*>(partial_o + (group_base + (size_t)row * nsplit) * D) + d4;
+        const float4* po = reinterpret_cast<const float4*>(partial_o + (group_base + (size_t)row * nsplit) * DV) + d4;
         float L = 0.f;
         for (int i = 0; i < nsplit; ++i) L += lsum[row * nsplit + i];
         if (terms.sink) L += exp2f(__ldg(terms.sink + kvh * G + h0 + row) * LOG2E - s_row_max[row]);
@@ -571,11 +588,11 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
             const float fj = f[i];
             o.x += v.x * fj; o.y += v.y * fj; o.z += v.z * fj; o.w += v.w * fj;
         }
-        const float inv = L > 0.f ? 1.f / L : 0.f;
+        const float inv = L > 0.f ? head_gate(terms.gate, n, Hq, kvh * G + h0 + row) / L : 0.f;
         uint2 packed;
         packed.x = pack_bf16(o.x * inv, o.y * inv);
         packed.y = pack_bf16(o.z * inv, o.w * inv);
-        *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * D + 4 * d4) = packed;
+        *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * DV + 4 * d4) = packed;
     }
 }
 
@@ -583,17 +600,17 @@ attn_decode_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restric
 // prefill
 // ---------------------------------------------------------------------------------------
 constexpr int PF_WARPS = 4;
-constexpr int PF_MT = D <= 128 ? 2 : 1;                       // 16-row tiles per warp (the accumulators must fit the registers)
+constexpr int PF_MT = DMAX <= 128 ? 2 : 1;                       // 16-row tiles per warp (the accumulators must fit the registers)
 constexpr int PF_BM = 16 * PF_MT * PF_WARPS;                  // rows (token, head) per block
 constexpr int PF_BN = 64;                                     // keys per iteration
-constexpr int PF_STAGE = 2 * PF_BN * DP;                      // K then V
+constexpr int PF_STAGE = PF_BN * (DP + VP);                   // K then V
 constexpr int PF_Q_ELEMS = PF_BM * DP;
 constexpr int PF_SMEM = PF_Q_ELEMS * 2 + 2 * PF_STAGE * 2 + 2 * PF_BN * 8;
 
 // TERMS: the softmax has a distance table, a sink, or values that are the keys (then v_cache == k_cache, a tile is
 // copied once and both products read it).
 template <bool TERMS>
-__global__ void __launch_bounds__(PF_WARPS * 32, (D <= 128 ? 2 : 1))
+__global__ void __launch_bounds__(PF_WARPS * 32, (DMAX <= 128 ? 2 : 1))
 attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restrict__ q, int q_stride,
                     const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                     const int* __restrict__ seq_kv_len, const int* __restrict__ seq_slot,
@@ -602,7 +619,7 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
                     float scale_log2e, int skip_single, int* status, const ScoreTerms terms) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
     TW_TIMELINE_SCOPE(TW_K_ATTN_PREFILL);
-    const bool values_are_keys = TERMS && v_cache == k_cache;
+    const bool values_are_keys = TERMS && SAME_DIMS && v_cache == k_cache;
     tw_grid_wait();
     TW_TIMELINE_MARK();
     tw_grid_launch_dependents();
@@ -646,7 +663,7 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
             const int r = wbase + 16 * mt + g + 8 * h;
             rvalid[mt][h] = r < rows_total;
             rpos[mt][h] = pos0 + r / G;
-            rlo[mt][h] = (window > 0 && rpos[mt][h] - window + 1 > 0) ? rpos[mt][h] - window + 1 : 0;
+            rlo[mt][h] = tw_first_key(rpos[mt][h], window);
         }
     }
     const float* brow[TERMS ? PF_MT : 1][2];        // the distance table's row of each of this thread's heads
@@ -672,20 +689,20 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
     const int t_last = min(q_len - 1, (row0 + PF_BM - 1) / G);
     const int key_end = pos0 + t_last + 1;
     const int t_first = row0 / G;
-    const int lo_block = (window > 0 && pos0 + t_first - window + 1 > 0) ? pos0 + t_first - window + 1 : 0;
+    const int lo_block = tw_first_key(pos0 + t_first, window);
     const int key_begin = lo_block / PF_BN * PF_BN;
     const int ntiles = (key_end - key_begin + PF_BN - 1) / PF_BN;
     // warp-level bounds, to skip tiles no row of the warp can see
     const int wr1 = min(rows_total - 1, wbase + 16 * PF_MT - 1);
     const int warp_hi = pos0 + wr1 / G;
-    const int warp_lo = (window > 0 && pos0 + wbase / G - window + 1 > 0) ? pos0 + wbase / G - window + 1 : 0;
+    const int warp_lo = tw_first_key(pos0 + wbase / G, window);
 
     auto load_tile = [&](int t, int st) {
         const int kb = key_begin + t * PF_BN;
         long long* offs = offs_all + st * PF_BN;
         if (threadIdx.x < PF_BN)
-            offs[threadIdx.x] = key_offset(kb + threadIdx.x, lo_block, key_end, table, table_stride, page_size, num_pages,
-                                           Hkv, kvh, status);
+            offs[threadIdx.x] = key_row(kb + threadIdx.x, lo_block, key_end, table, table_stride, page_size, num_pages,
+                                        Hkv, kvh, status);
         __syncthreads();
         bf16* ks_ = stages + st * PF_STAGE;
         bf16* vs_ = ks_ + PF_BN * DP;
@@ -693,9 +710,16 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
             const int row = i / CHUNKS, col = i - row * CHUNKS;
             const long long off = offs[row];
             const int bytes = off >= 0 ? 16 : 0;
-            const long long src = off >= 0 ? off + col * 8 : 0;
+            const long long src = off >= 0 ? off * D + col * 8 : 0;
             cp_async16(ks_ + row * DP + col * 8, k_cache + src, bytes);
-            if (!values_are_keys) cp_async16(vs_ + row * DP + col * 8, v_cache + src, bytes);
+            if (SAME_DIMS && !values_are_keys) cp_async16(vs_ + row * VP + col * 8, v_cache + src, bytes);
+        }
+        if constexpr (!SAME_DIMS) {
+            for (int i = threadIdx.x; i < PF_BN * VCHUNKS; i += PF_WARPS * 32) {
+                const int row = i / VCHUNKS, col = i - row * VCHUNKS;
+                const long long off = offs[row];
+                cp_async16(vs_ + row * VP + col * 8, v_cache + (off >= 0 ? off * DV + col * 8 : 0), off >= 0 ? 16 : 0);
+            }
         }
         cp_async_commit();
     };
@@ -798,7 +822,7 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
 #pragma unroll
                 for (int nt2 = 0; nt2 < NT_O / 2; ++nt2) {
                     uint32_t b[4];
-                    ldmatrix_x4_trans(b, vs_ + (kk * 16 + (j & 1) * 8 + r8) * DP + nt2 * 16 + (j >> 1) * 8);
+                    ldmatrix_x4_trans(b, vs_ + (kk * 16 + (j & 1) * 8 + r8) * VP + nt2 * 16 + (j >> 1) * 8);
 #pragma unroll
                     for (int mt = 0; mt < PF_MT; ++mt) {
                         mma_bf16(oacc[mt][2 * nt2], pfrag[mt][kk], b[0], b[1]);
@@ -824,9 +848,13 @@ attn_prefill_kernel(bf16* __restrict__ out, int out_stride, const bf16* __restri
                 l1 += exp2f(__ldg(terms.sink + kvh * G + rb - tb * G) * LOG2E - mrow[mt][1]);
             }
         }
-        const float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
-        bf16* oa = out + (size_t)(n0 + ta) * out_stride + (size_t)(kvh * G + ra - ta * G) * D;
-        bf16* ob = out + (size_t)(n0 + tb) * out_stride + (size_t)(kvh * G + rb - tb * G) * D;
+        float i0 = l0 > 0.f ? 1.f / l0 : 0.f, i1 = l1 > 0.f ? 1.f / l1 : 0.f;
+        if (terms.gate) {
+            if (rvalid[mt][0]) i0 *= head_gate(terms.gate, n0 + ta, Hq, kvh * G + ra - ta * G);
+            if (rvalid[mt][1]) i1 *= head_gate(terms.gate, n0 + tb, Hq, kvh * G + rb - tb * G);
+        }
+        bf16* oa = out + (size_t)(n0 + ta) * out_stride + (size_t)(kvh * G + ra - ta * G) * DV;
+        bf16* ob = out + (size_t)(n0 + tb) * out_stride + (size_t)(kvh * G + rb - tb * G) * DV;
 #pragma unroll
         for (int nt = 0; nt < NT_O; ++nt) {
             const int d = nt * 8 + 2 * c;
@@ -846,12 +874,14 @@ int set_attrs() {
     if (e != cudaSuccess) return (int)e;
     e = cudaFuncSetAttribute(attn_decode_kernel<true, false>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (e != cudaSuccess) return (int)e;
+#if TW_V_DIM == TW_HEAD_DIM
     e = cudaFuncSetAttribute(attn_decode_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DEC_SMEM);
     if (e != cudaSuccess) return (int)e;
     e = cudaFuncSetAttribute(attn_decode_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DEC_SMEM);
     if (e != cudaSuccess) return (int)e;
     e = cudaFuncSetAttribute(attn_decode_kernel<true, true>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
     if (e != cudaSuccess) return (int)e;
+#endif
     e = cudaFuncSetAttribute(attn_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
     if (e != cudaSuccess) return (int)e;
     e = cudaFuncSetAttribute(attn_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, PF_SMEM);
@@ -888,6 +918,7 @@ bool decode_cluster_ok(int size) {
 }  // namespace
 
 TW_EXPORT int tw_attn_head_dim() { return D; }
+TW_EXPORT int tw_attn_v_dim() { return DV; }
 
 #ifdef TW_TRACE
 TW_EXPORT int tw_attn_decode_trace_ptr(void** ptr, int* blocks, int* slots) {
@@ -903,7 +934,7 @@ TW_EXPORT int tw_attn_decode_cluster_slices() { return DEC_MAX_CLUSTER; }
 // Beside them it needs one int32 counter per (request, key/value head, tile of 8 heads), zero before the
 // first launch; the kernel leaves them zero.
 TW_EXPORT long long tw_attn_decode_scratch_floats(int n_seqs, int Hq, int nsplit) {
-    return (long long)n_seqs * Hq * nsplit * (D + 2);
+    return (long long)n_seqs * Hq * nsplit * (DV + 2);
 }
 
 // Most slices a request's keys may be cut into.  The merge through scratch memory keeps two floats per
@@ -935,7 +966,7 @@ static int decode_launch(void* out, int out_stride, const void* q, int q_stride,
     if (int e = set_attrs()) return e;
     const int G = Hq / Hkv, htiles = (G + DEC_HEADS - 1) / DEC_HEADS;
     float* partial_o = scratch;
-    float* partial_ml = scratch ? scratch + (size_t)n_seqs * Hq * nsplit * D : nullptr;
+    float* partial_ml = scratch ? scratch + (size_t)n_seqs * Hq * nsplit * DV : nullptr;
     dim3 grid(nsplit * htiles, Hkv, n_seqs);
     if (nsplit > 1 && !(flags & 1) && decode_cluster_ok(nsplit))
         return tw_launch(attn_decode_kernel<true, false>, dim3(grid), dim3(DEC_WARPS * 32), DEC_SMEM, stream, nsplit,
@@ -960,16 +991,16 @@ TW_EXPORT int tw_attn_decode(void* out, int out_stride, const void* q, int q_str
 }
 
 // With a distance table (fp32 [Hq][reach], or null), a sink (fp32 [Hq], or null), and, when v_cache is k_cache,
-// values that are the keys.
+// values that are the keys; and a gate (fp32 [rows][Hq], or null).
 TW_EXPORT int tw_attn_decode_terms(void* out, int out_stride, const void* q, int q_stride, const int* seq_q_start,
                                    const int* seq_q_len, const int* seq_kv_len, const int* seq_slot, const int* block_table,
                                    int table_stride, const void* k_cache, const void* v_cache, int n_seqs, int Hq, int Hkv,
                                    int page_size, int num_pages, int window, float scale, int nsplit, int flags,
                                    float* scratch, int* counters, const float* bias, int reach, const float* sink,
-                                   int* status, cudaStream_t stream) {
+                                   const float* gate, int* status, cudaStream_t stream) {
     return decode_launch(out, out_stride, q, q_stride, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, table_stride,
                          k_cache, v_cache, n_seqs, Hq, Hkv, page_size, num_pages, window, scale, nsplit, flags, scratch,
-                         counters, status, ScoreTerms{bias, reach, sink}, stream);
+                         counters, status, ScoreTerms{bias, reach, sink, gate}, stream);
 }
 
 // The same for a decode-only step whose q/k/v product has not been touched yet: the kernel adds the bias,
@@ -977,6 +1008,7 @@ TW_EXPORT int tw_attn_decode_terms(void* out, int out_stride, const void* q, int
 // needs no kernel between the product and the attention.  The product is given as fp32 slices
 // [nslices][rows][(Hq + 2 Hkv) D] (`partial`) or as bf16 rows (`dense`); `bias` and `inv_freq` may be null;
 // with write_cache 0 the cache is read only (the new position must then be in it already).
+#if TW_V_DIM == TW_HEAD_DIM
 TW_EXPORT int tw_attn_decode_fused(void* out, int out_stride, const float* partial, int nslices, long long slice_stride,
                                    const void* dense, int dense_stride, const float* bias, const float* inv_freq,
                                    int write_cache, const int* seq_q_start, const int* seq_q_len, const int* seq_kv_len,
@@ -1014,14 +1046,17 @@ TW_EXPORT int tw_attn_decode_fused(void* out, int out_stride, const float* parti
     return TW_LAUNCH_CHECK();
 }
 
-// bias, reach, sink: see ScoreTerms; all null and v_cache apart from k_cache: the plain softmax.
+#endif
+
+// bias, reach, sink, gate: see ScoreTerms; all null and v_cache apart from k_cache: the plain softmax.
 TW_EXPORT int tw_attn_prefill(void* out, int out_stride, const void* q, int q_stride, const int* seq_q_start,
                               const int* seq_q_len, const int* seq_kv_len, const int* seq_slot, const int* block_table,
                               int table_stride, const void* k_cache, const void* v_cache, int n_seqs, int max_q_len,
                               int Hq, int Hkv, int page_size, int num_pages, int window, float scale, int skip_single,
-                              const float* bias, int reach, const float* sink, int* status, cudaStream_t stream) {
+                              const float* bias, int reach, const float* sink, const float* gate, int* status,
+                              cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
-    if (Hkv <= 0 || Hq % Hkv || (bias && reach < 1)) return (int)cudaErrorInvalidValue;
+    if (Hkv <= 0 || Hq % Hkv || (bias && reach < 1) || (!SAME_DIMS && v_cache == k_cache)) return (int)cudaErrorInvalidValue;
     if (int e = set_attrs()) return e;
     const int G = Hq / Hkv;
     dim3 grid((max_q_len * G + PF_BM - 1) / PF_BM, Hkv, n_seqs);
@@ -1029,7 +1064,7 @@ TW_EXPORT int tw_attn_prefill(void* out, int out_stride, const void* q, int q_st
     tw_launch(with_terms ? attn_prefill_kernel<true> : attn_prefill_kernel<false>, dim3(grid), dim3(PF_WARPS * 32), PF_SMEM,
         stream, 1, (bf16*)out, out_stride, (const bf16*)q, q_stride, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table,
         table_stride, (const bf16*)k_cache, (const bf16*)v_cache, Hq, Hkv, page_size, num_pages, window,
-        scale * 1.4426950408889634f, skip_single, status, ScoreTerms{bias, reach, sink});
+        scale * 1.4426950408889634f, skip_single, status, ScoreTerms{bias, reach, sink, gate});
     return TW_LAUNCH_CHECK();
 }
 
@@ -1068,7 +1103,7 @@ TW_EXPORT int tw_attn_decode_static(void* out, int out_stride, const void* q, in
         return r;
     }
     const int G = Hq / Hkv, htiles = (G + DEC_HEADS - 1) / DEC_HEADS;
-    const size_t partial_bytes = sizeof(float) * (size_t)n_seqs * Hq * nsplit * (D + 2);
+    const size_t partial_bytes = sizeof(float) * (size_t)n_seqs * Hq * nsplit * (DV + 2);
     const size_t counter_bytes = sizeof(int) * (size_t)n_seqs * Hkv * htiles;
     if (counter_bytes > TW_ATTN_STATIC_COUNTER_BYTES ||
         partial_bytes > TW_ATTN_STATIC_SCRATCH_BYTES - TW_ATTN_STATIC_COUNTER_BYTES) {
@@ -1098,7 +1133,7 @@ TW_EXPORT int tw_attn_decode_static(void* out, int out_stride, const void* q, in
     unsigned char* base = g_static_scratch_ptr[device];
     int* counters = reinterpret_cast<int*>(base);
     float* partial_o = reinterpret_cast<float*>(base + TW_ATTN_STATIC_COUNTER_BYTES);
-    float* partial_ml = partial_o + (size_t)n_seqs * Hq * nsplit * D;
+    float* partial_ml = partial_o + (size_t)n_seqs * Hq * nsplit * DV;
     if (int a = set_attrs()) return a;
     // the array keeps what the last call left; only the counters need a defined start
     e = cudaMemsetAsync(counters, 0, counter_bytes, stream);

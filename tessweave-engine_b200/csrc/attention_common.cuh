@@ -73,11 +73,16 @@ struct FusedQkv {
 // What a softmax may have beside the scaled dot products; every member optional (null = absent).
 //   bias: fp32 [Hq][reach]; entry min(position - key position, reach - 1) of head h is added to h's scaled score.
 //   sink: fp32 [Hq]; exp(sink[h]) joins head h's denominator once (no key, no value, not scaled, no bias).
+//   gate: fp32 [rows][Hq]; head h's output of a row is multiplied by its entry (not part of the softmax).
 struct ScoreTerms {
     const float* bias;
     int reach;
     const float* sink;
+    const float* gate;
 };
+__device__ __forceinline__ float head_gate(const float* gate, size_t row, int Hq, int head) {
+    return gate ? __ldg(gate + row * Hq + head) : 1.f;
+}
 constexpr float LOG2E = 1.4426950408889634f;
 
 // fp32 values of NC columns of one row of the q/k/v product, bias included.  The slices of a split product are

@@ -1,5 +1,5 @@
 // Paged split-KV decode attention in bfloat16 with keys and values brought in by TMA, for head sizes
-// that are multiples of 64 (compile with -DTW_HEAD_DIM=64, 128, 192 or 256).
+// that are multiples of 64 (compile with -DTW_HEAD_DIM=64, 128, 192 or 256; values of another such size: -DTW_V_DIM).
 //
 // A block serves one (request, key/value head, slice of the request's keys) for requests that bring ONE
 // token; the up to 8 query heads of the group are the columns of one MMA tile, so keys and values are read
@@ -22,7 +22,8 @@
 // the shared memory of the block that merges those values), or -- when there are more slices than a cluster
 // can hold -- through scratch memory in the block that finishes last.
 //
-//   score = (q . k) * scale,  visible iff  position - window < p <= position
+//   score = (q . k) * scale,  visible iff  tw_first_key(position, window) <= p <= position
+//   (`gate`: fp32 [rows][Hq] or null; head h's output is multiplied by its entry)
 // Reference: flow_engine/model.py:193-200 and flow_engine/kernels/paged_decode.py:13-43.
 //
 // Every wait on an mbarrier is bounded; a wait that runs out sets TW_ERR_WAIT in the status word, every role
@@ -35,6 +36,9 @@ namespace cg = cooperative_groups;
 
 #ifndef TW_HEAD_DIM
 #define TW_HEAD_DIM 128
+#endif
+#ifndef TW_V_DIM
+#define TW_V_DIM TW_HEAD_DIM
 #endif
 
 namespace {
@@ -56,20 +60,24 @@ using tw_attn::product_cols;
 
 constexpr int D = TW_HEAD_DIM;
 static_assert(D % 64 == 0 && D >= 64 && D <= 256, "the TMA decode attention takes head sizes 64, 128, 192 and 256");
-constexpr int KB = D / 64;                         // 64-column blocks of a row of k or v
+constexpr int DV = TW_V_DIM;                       // size of a value, and of a head of the output
+static_assert(DV % 64 == 0 && DV >= 64 && DV <= 256, "the TMA decode attention takes value sizes 64, 128, 192 and 256");
+constexpr bool SAME_DIMS = D == DV;
+constexpr int KB = D / 64;                         // 64-column blocks of a row of k
+constexpr int VB = DV / 64;                        // 64-column blocks of a row of v
 constexpr int TILE = 64;                           // keys per stage
 constexpr int CWARPS = 4;                          // consumer warps: warp w owns keys 16 w .. 16 w + 15 of a tile
 constexpr int CTHREADS = CWARPS * 32;
 constexpr int THREADS = CTHREADS + 32;             // plus the producer warp
 constexpr int HEADS = 8;                           // query heads per block (columns of the MMA)
 constexpr int BLKB = TILE * 128;                   // bytes of a [64 keys][64 values of d] swizzled block
-constexpr int STAGE_BYTES = 2 * KB * BLKB;         // K, then V
+constexpr int STAGE_BYTES = (KB + VB) * BLKB;      // K, then V
 constexpr int MAX_STAGES = 8;
-constexpr int STATIC_SMEM_ROOM = 9 * 1024 + HEADS * D * 4;   // barriers, block-table entries, query heads, the cluster's merge, alignment slack
+constexpr int STATIC_SMEM_ROOM = 9 * 1024 + HEADS * (D > DV ? D : DV) * 4;   // barriers, block-table entries, query heads, the cluster's merge, alignment slack
 constexpr int DEEPEST = (227 * 1024 - STATIC_SMEM_ROOM) / STAGE_BYTES < MAX_STAGES ? (227 * 1024 - STATIC_SMEM_ROOM) / STAGE_BYTES : MAX_STAGES;
 constexpr int PAGE_CACHE = 512;                    // block-table entries kept in shared memory
 constexpr int KSTEPS = D / 16;
-constexpr int MT_O = D / 16;                       // m-tiles of O^T
+constexpr int MT_O = DV / 16;                      // m-tiles of O^T
 constexpr int MAX_CLUSTER = 16;
 
 // -DTW_TRACE: the first consumer thread and the producer of every block record the global timer (ns) at
@@ -92,7 +100,7 @@ __device__ long long g_trace[TRACE_BLOCKS * TRACE_SLOTS];
 #endif
 constexpr float NEG_INF = -INFINITY;
 // after the last tile the ring holds the warps' partial results
-constexpr int MERGE_BYTES = CWARPS * HEADS * (D + 2) * 4;
+constexpr int MERGE_BYTES = CWARPS * HEADS * (DV + 2) * 4;
 constexpr int MIN_STAGES = (MERGE_BYTES + STAGE_BYTES - 1) / STAGE_BYTES < 2 ? 2 : (MERGE_BYTES + STAGE_BYTES - 1) / STAGE_BYTES;
 
 // byte offset of (key row, 16-byte chunk of d) inside a K or V tile of a stage
@@ -111,19 +119,20 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                        const int* __restrict__ block_table, int table_stride, int Hq, int Hkv, int page_size,
                        int num_pages, int window, float scale_log2e, int nsplit, int nstages,
                        float* __restrict__ partial_o, float* __restrict__ partial_ml, int* __restrict__ counters,
-                       int* status, const FusedQkv fq) {
+                       int* status, const FusedQkv fq, const float* __restrict__ gate) {
+    static_assert(!FUSED || SAME_DIMS, "the fused form packs q, k and v as heads of one size");
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t full[MAX_STAGES];
     __shared__ __align__(8) uint64_t empty[MAX_STAGES];
     __shared__ int page_cache[PAGE_CACHE];
     __shared__ __align__(16) bf16 s_q[HEADS * D];                 // the block's query heads (zero beyond the group)
-    __shared__ __align__(16) bf16 s_fresh[2 * D];                 // the newest position's key and value, when this block made them
+    __shared__ __align__(16) bf16 s_fresh[FUSED ? 2 * D : 8];                 // the newest position's key and value, when this block made them
     __shared__ int s_is_last, s_aborted;
     __shared__ float s_row_max[HEADS];
     __shared__ float2 s_row_ml[HEADS];                            // this block's (maximum, sum) per head, warps merged
     // what the other blocks of the cluster send this one to merge: their slices of the groups of four values it
     // owns, and their maxima and sums.  Of its own, not in the ring: a neighbour may be done before this block is.
-    __shared__ __align__(16) float4 s_recv_o[HEADS * D / 4 + MAX_CLUSTER];
+    __shared__ __align__(16) float4 s_recv_o[HEADS * DV / 4 + MAX_CLUSTER];
     __shared__ float2 s_recv_ml[MAX_CLUSTER][HEADS];
 
     const int s = blockIdx.z, kvh = blockIdx.y;
@@ -139,7 +148,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int nheads = min(HEADS, G - h0);
     const int n = seq_q_start[s];
     const int pos = seq_kv_len[s] - 1;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = tw_first_key(pos, window);
     // tiles start at multiples of 64 keys, so that a tile is a whole number of pages (or a part of one)
     const int base = (lo / TILE) * TILE;
     const int per = (((pos + 1 - base) + nsplit - 1) / nsplit + TILE - 1) / TILE * TILE;
@@ -195,7 +204,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                     else row_coord = (page * Hkv + kvh) * page_size + (key0 - blk * page_size);
                 }
             }
-            const uint32_t bytes = (uint32_t)__popc(__ballot_sync(0xffffffffu, row_coord >= 0)) * (2 * KB * box_rows * 128);
+            const uint32_t bytes = (uint32_t)__popc(__ballot_sync(0xffffffffu, row_coord >= 0)) * ((KB + VB) * box_rows * 128);
             int ok = 1;
             if (lane == 0) {
                 ok = (!*aborted && mbar_wait(&empty[st], parity ^ 1, status)) ? 1 : 0;
@@ -206,10 +215,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             if (row_coord >= 0) {
                 unsigned char* dst = ring + st * STAGE_BYTES + lane * box_rows * 128;
 #pragma unroll
-                for (int kb = 0; kb < KB; ++kb) {
-                    tma_load_2d(dst + kb * BLKB, &map_k, &full[st], kb * 64, row_coord);
-                    tma_load_2d(dst + (KB + kb) * BLKB, &map_v, &full[st], kb * 64, row_coord);
-                }
+                for (int kb = 0; kb < KB; ++kb) tma_load_2d(dst + kb * BLKB, &map_k, &full[st], kb * 64, row_coord);
+#pragma unroll
+                for (int vb = 0; vb < VB; ++vb) tma_load_2d(dst + (KB + vb) * BLKB, &map_v, &full[st], vb * 64, row_coord);
             }
             issued = i + 1;
         }
@@ -326,8 +334,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 // Value rows of keys this block must not see -- beyond the request's last key, before the window,
                 // or of a page that was never copied -- hold whatever was there: zero them (0 x NaN is NaN).
                 if (key0 < first_key || key0 + 16 > k_end) {
-                    for (int idx = lane; idx < 16 * (D / 8); idx += 32) {
-                        const int r = idx / (D / 8), ch = idx - r * (D / 8);
+                    for (int idx = lane; idx < 16 * (DV / 8); idx += 32) {
+                        const int r = idx / (DV / 8), ch = idx - r * (DV / 8);
                         if (key0 + r < first_key || key0 + r >= k_end)
                             *reinterpret_cast<uint4*>(vs_ + tile_offset(warp * 16 + r, ch)) = make_uint4(0u, 0u, 0u, 0u);
                     }
@@ -413,8 +421,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     // Only the consumer warps are here: the producer has left (see above), so every barrier below is theirs.
     consumer_sync();
     const bool failed = *aborted != 0;
-    float* mo = reinterpret_cast<float*>(ring);                  // [warps][heads][D]
-    float* wml = mo + CWARPS * HEADS * D;                        // [warps][heads][2]
+    float* mo = reinterpret_cast<float*>(ring);                  // [warps][heads][DV]
+    float* wml = mo + CWARPS * HEADS * DV;                       // [warps][heads][2]
     if (g == 0) {
         wml[(warp * HEADS + 2 * c) * 2] = m0; wml[(warp * HEADS + 2 * c) * 2 + 1] = l0;
         wml[(warp * HEADS + 2 * c + 1) * 2] = m1; wml[(warp * HEADS + 2 * c + 1) * 2 + 1] = l1;
@@ -430,8 +438,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         if (failed) M0 = M1 = NEG_INF;
         const float f0 = (m0 == NEG_INF || M0 == NEG_INF) ? 0.f : exp2f(m0 - M0);
         const float f1 = (m1 == NEG_INF || M1 == NEG_INF) ? 0.f : exp2f(m1 - M1);
-        float* p0 = mo + (warp * HEADS + 2 * c) * D;
-        float* p1 = p0 + D;
+        float* p0 = mo + (warp * HEADS + 2 * c) * DV;
+        float* p1 = p0 + DV;
 #pragma unroll
         for (int mt = 0; mt < MT_O; ++mt) {
             const int d = mt * 16 + g;
@@ -453,7 +461,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     consumer_sync();
     // Four values of d at a time: the block's slice of (head, d .. d + 3).  It goes to the output (one slice), to
     // the block of the cluster that merges these four values (see below), or to scratch memory.
-    constexpr int D4 = D / 4;
+    constexpr int D4 = DV / 4;
     const int n4 = nheads * D4;
     const int own4 = (n4 + nsplit - 1) / nsplit;                 // groups of four a block of the cluster merges
     const float4* mo4 = reinterpret_cast<const float4*>(mo);
@@ -468,17 +476,17 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const int head = kvh * G + h0 + row;
         if (nsplit == 1) {
             const float L = s_row_ml[row].y;
-            const float inv = L > 0.f ? 1.f / L : 0.f;
+            const float inv = L > 0.f ? tw_attn::head_gate(gate, n, Hq, head) / L : 0.f;
             uint2 packed;
             packed.x = pack_bf16(o.x * inv, o.y * inv);
             packed.y = pack_bf16(o.z * inv, o.w * inv);
-            *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)head * D + 4 * d4) = packed;
+            *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)head * DV + 4 * d4) = packed;
         } else if (CLUSTER) {
             cg::cluster_group cluster = cg::this_cluster();
             *cluster.map_shared_rank(s_recv_o + split * own4 + j / nsplit, j % nsplit) = o;
         } else {
             const size_t at = ((size_t)s * Hq + head) * nsplit + split;
-            *reinterpret_cast<float4*>(partial_o + at * D + 4 * d4) = o;
+            *reinterpret_cast<float4*>(partial_o + at * DV + 4 * d4) = o;
             if (d4 == 0) { partial_ml[at * 2] = s_row_ml[row].x; partial_ml[at * 2 + 1] = s_row_ml[row].y; }
         }
     }
@@ -514,7 +522,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 L += ml.y * f;
                 o += mine[(i * own4 + jj) * 4] * f;
             }
-            out[(size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * D + d] = __float2bfloat16_rn(L > 0.f ? o / L : 0.f);
+            out[(size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * DV + d] =
+                __float2bfloat16_rn(L > 0.f ? o / L * tw_attn::head_gate(gate, n, Hq, kvh * G + h0 + row) : 0.f);
         }
         if (warp == 0) TW_TTRACE(7);
         return;
@@ -558,7 +567,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     for (int idx = threadIdx.x; idx < nheads * D4; idx += CTHREADS) {
         const int row = idx / D4, d4 = idx - row * D4;
         const float* f = fac + row * nsplit;
-        const float4* po = reinterpret_cast<const float4*>(partial_o + (group_base + (size_t)row * nsplit) * D) + d4;
+        const float4* po = reinterpret_cast<const float4*>(partial_o + (group_base + (size_t)row * nsplit) * DV) + d4;
         float L = 0.f;
         for (int i = 0; i < nsplit; ++i) L += lsum[row * nsplit + i];
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -578,11 +587,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             const float fj = f[i];
             o.x += v.x * fj; o.y += v.y * fj; o.z += v.z * fj; o.w += v.w * fj;
         }
-        const float inv = L > 0.f ? 1.f / L : 0.f;
+        const float inv = L > 0.f ? tw_attn::head_gate(gate, n, Hq, kvh * G + h0 + row) / L : 0.f;
         uint2 packed;
         packed.x = pack_bf16(o.x * inv, o.y * inv);
         packed.y = pack_bf16(o.z * inv, o.w * inv);
-        *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * D + 4 * d4) = packed;
+        *reinterpret_cast<uint2*>(out + (size_t)n * out_stride + (size_t)(kvh * G + h0 + row) * DV + 4 * d4) = packed;
     }
 }
 
@@ -661,15 +670,18 @@ TW_EXPORT int tw_attn_decode_tma_supported(int page_size) {
 // duty to store the new key and value.  `nstages` is the depth of the ring (0: as deep as one block per SM
 // allows while the launch has no more blocks than SMs, else half of that so that two blocks share an SM).
 // `scratch` and `counters` as for tw_attn_decode; they are used when the slices do not fit a cluster.
+// `gate` (fp32 [rows][Hq] or null): head h's output of a row is multiplied by its entry.
 TW_EXPORT int tw_attn_decode_tma(void* out, int out_stride, const void* q, int q_stride, const float* partial, int nslices,
                                  long long slice_stride, const void* dense, int dense_stride, const float* bias,
                                  const float* inv_freq, int write_cache, const int* seq_q_start, const int* seq_q_len,
                                  const int* seq_kv_len, const int* seq_slot, const int* block_table, int table_stride,
                                  void* k_cache, void* v_cache, int n_seqs, int Hq, int Hkv, int page_size, int num_pages,
                                  int window, float scale, int nsplit, int nstages, int flags, float* scratch, int* counters,
-                                 int* status, const void* next_weights, long long next_bytes, cudaStream_t stream) {
+                                 int* status, const void* next_weights, long long next_bytes, const float* gate,
+                                 cudaStream_t stream) {
     if (n_seqs <= 0) return 0;
     const bool fused = partial || dense;
+    if (fused && !SAME_DIMS) return (int)cudaErrorInvalidValue;
     if (Hkv <= 0 || Hq % Hkv || nsplit < 1 || nsplit > DEC_MAX_SPLITS || !tw_attn_decode_tma_supported(page_size) ||
         (!fused && !q) || (partial && nslices < 1) || (nsplit > 1 && (!scratch || !counters)))
         return (int)cudaErrorInvalidValue;
@@ -692,9 +704,9 @@ TW_EXPORT int tw_attn_decode_tma(void* out, int out_stride, const void* q, int q
     const int box_rows = page_size < TILE ? page_size : TILE;
     CUtensorMap mk, mv;
     if (int e = tc5::get_map(k_cache, rows, D, box_rows, &mk)) return e;
-    if (int e = tc5::get_map(v_cache, rows, D, box_rows, &mv)) return e;
+    if (int e = tc5::get_map(v_cache, rows, DV, box_rows, &mv)) return e;
     float* partial_o = scratch;
-    float* partial_ml = scratch ? scratch + (size_t)n_seqs * Hq * nsplit * D : nullptr;
+    float* partial_ml = scratch ? scratch + (size_t)n_seqs * Hq * nsplit * DV : nullptr;
     FusedQkv fq = {};
     if (fused) {
         fq.partial = partial; fq.nslices = nslices; fq.slice_stride = slice_stride;
@@ -713,11 +725,13 @@ TW_EXPORT int tw_attn_decode_tma(void* out, int out_stride, const void* q, int q
         return tw_launch(attn_decode_tma_kernel<CL, FU>, grid, dim3(THREADS), smem, stream, CL ? nsplit : 1, mk, mv,    \
                          (bf16*)out, out_stride, (const bf16*)q, q_stride, seq_q_start, seq_q_len, seq_kv_len, seq_slot, \
                          block_table, table_stride, Hq, Hkv, page_size, num_pages, window, scale_log2e, nsplit, nstages, \
-                         partial_o, partial_ml, counters, status, fq);                                                 \
+                         partial_o, partial_ml, counters, status, fq, gate);                                              \
     } while (0)
-    if (cluster && fused) TW_DECODE_TMA_LAUNCH(true, true);
+    if constexpr (SAME_DIMS) {
+        if (cluster && fused) TW_DECODE_TMA_LAUNCH(true, SAME_DIMS);
+        if (fused) TW_DECODE_TMA_LAUNCH(false, SAME_DIMS);
+    }
     if (cluster) TW_DECODE_TMA_LAUNCH(true, false);
-    if (fused) TW_DECODE_TMA_LAUNCH(false, true);
     TW_DECODE_TMA_LAUNCH(false, false);
 #undef TW_DECODE_TMA_LAUNCH
 }

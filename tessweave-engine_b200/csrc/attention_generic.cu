@@ -3,15 +3,16 @@
 // This is the exact-arithmetic kernel: fp32 scores, fp32 online softmax, fp32
 // accumulation, any head size up to 1024 (keys and values may differ in size:
 // D for queries and keys, Dv for values and the output), any number of heads
-// and groups, an optional window.  It serves the whole float32 path and any bfloat16 shape
+// and groups, an optional window or chunks (`window`: see tw_first_key).  It serves the whole float32 path and any bfloat16 shape
 // that the tensor-core kernels refuse.  Prompt portions and single decoded
 // tokens are the same case here: each token row attends to the keys
 // lo..position of its own request through that request's block table.
 //
 //   kv_head = head / (Hq / Hkv)
 //   score_p = (q . k_p) * scale [+ bias[min(position - p, bias_rows - 1), head]]
-//                                          p in [lo, position], lo = max(0, position - window + 1)
+//                                          p in [lo, position], lo = tw_first_key(position, window)
 //   out     = softmax(score) @ v           [the denominator also holds exp(sink[head]): a term without key or value]
+//             [* gate[row, head], a number per head and row]
 // Reference: flow_engine/model.py:193-200 (mask p <= position), flow_engine/
 // kernels/paged_decode.py:13-43 (online softmax in fp32, GQA head map).
 //
@@ -30,7 +31,7 @@ __global__ void attn_generic_kernel(T* __restrict__ out, int out_stride, const T
                                     int table_stride, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                                     int Hq, int Hkv, int D, int Dv, int page_size, int num_pages, int window, float scale,
                                     const float* __restrict__ dist_bias, int bias_rows, const float* __restrict__ sink,
-                                    int* status) {
+                                    const float* __restrict__ gate, int* status) {
     extern __shared__ float smem[];  // TW_ATTN_WARPS * (Dv + 2)
     tw_grid_wait();
     tw_grid_launch_dependents();
@@ -51,7 +52,7 @@ __global__ void attn_generic_kernel(T* __restrict__ out, int out_stride, const T
         acc[j] = 0.f;
     }
     float m = -INFINITY, l = 0.f;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = tw_first_key(pos, window);
     int p = lo + ((warp - lo) % TW_ATTN_WARPS + TW_ATTN_WARPS) % TW_ATTN_WARPS;
     for (; p <= pos; p += TW_ATTN_WARPS) {
         const int blk = p / page_size;
@@ -106,11 +107,12 @@ __global__ void attn_generic_kernel(T* __restrict__ out, int out_stride, const T
         L += smem[w * (Dv + 2) + Dv + 1] * f[w];
     }
     T* orow = out + (size_t)n * out_stride + head * Dv;
+    const float scale_out = gate ? gate[(size_t)n * gridDim.y + head] : 1.f;
     for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
         float o = 0.f;
 #pragma unroll
         for (int w = 0; w < TW_ATTN_WARPS; ++w) o += smem[w * (Dv + 2) + d] * f[w];
-        orow[d] = tw_from_float<T>(L > 0.f ? o / L : 0.f);
+        orow[d] = tw_from_float<T>(L > 0.f ? o / L * scale_out : 0.f);
     }
 }
 
@@ -118,7 +120,8 @@ TW_EXPORT int tw_attn_generic(void* out, int out_stride, const void* q, int q_st
                               const int* seq_of_token, const int* seq_slot, const int* block_table, int table_stride,
                               const void* k_cache, const void* v_cache, int n_tokens, int Hq, int Hkv, int D,
                               int Dv, int page_size, int num_pages, int window, float scale, const float* dist_bias,
-                              int bias_rows, const float* sink, int dtype, int* status, cudaStream_t stream) {
+                              int bias_rows, const float* sink, const float* gate, int dtype, int* status,
+                              cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (dist_bias && bias_rows <= 0) return (int)cudaErrorInvalidValue;
     if (D <= 0 || D > 1024 || Dv <= 0 || Dv > 1024 || Hkv <= 0 || Hq % Hkv) return (int)cudaErrorInvalidValue;
@@ -130,13 +133,13 @@ TW_EXPORT int tw_attn_generic(void* out, int out_stride, const void* q, int q_st
         tw_launch(kernel, dim3(grid), dim3(32 * TW_ATTN_WARPS), smem, stream, 1,
             (float*)out, out_stride, (const float*)q, q_stride, positions, seq_of_token, seq_slot, block_table,
             table_stride, (const float*)k_cache, (const float*)v_cache, Hq, Hkv, D, Dv, page_size, num_pages, window, scale,
-            dist_bias, bias_rows, sink, status);
+            dist_bias, bias_rows, sink, gate, status);
     } else {
         auto kernel = wide ? attn_generic_kernel<__nv_bfloat16, 32> : attn_generic_kernel<__nv_bfloat16, 8>;
         tw_launch(kernel, dim3(grid), dim3(32 * TW_ATTN_WARPS), smem, stream, 1,
             (__nv_bfloat16*)out, out_stride, (const __nv_bfloat16*)q, q_stride, positions, seq_of_token, seq_slot,
             block_table, table_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, Hq, Hkv, D, Dv,
-            page_size, num_pages, window, scale, dist_bias, bias_rows, sink, status);
+            page_size, num_pages, window, scale, dist_bias, bias_rows, sink, gate, status);
     }
     return TW_LAUNCH_CHECK();
 }

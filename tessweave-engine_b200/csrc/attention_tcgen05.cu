@@ -1,5 +1,5 @@
 // Paged causal attention for prompt portions on the 5th-generation tensor cores, for one head
-// size (compile with -DTW_HEAD_DIM=64 or 128).
+// size (compile with -DTW_HEAD_DIM=64 or 128; values of the other size: -DTW_V_DIM).
 //
 // A block serves up to 256 rows of one (request, key/value head), a row being a (token, query
 // head of the group) pair, as two tiles of 128 rows, and walks the request's keys in tiles of
@@ -17,9 +17,12 @@
 //
 // O is only rescaled when a row's maximum grows by more than 2^8 (the sums carry the same
 // stale maximum, so the quotient is exact); rows of values beyond the request's last key are
-// zeroed in shared memory, so stale page contents cannot reach a product.
+// zeroed in shared memory, so stale page contents cannot reach a product.  Pages that lie wholly before the first key
+// any row of the block sees (a window or a chunk has moved on, and the pages may have been given back) are not read:
+// their boxes are asked for beyond the end of the cache, which the copy engine answers with zeros.
 //
-//   score = (q . k) * scale,  visible iff  position - window < p <= position
+//   score = (q . k) * scale,  visible iff  tw_first_key(position, window) <= p <= position
+//   (`gate`: fp32 [rows][Hq] or null; head h's output is multiplied by its entry)
 // Reference: flow_engine/model.py:193-200 (the reference calls a library's attention here).
 //
 // Every wait on an mbarrier is bounded; a wait that runs out sets TW_ERR_WAIT in the status
@@ -29,6 +32,9 @@
 
 #ifndef TW_HEAD_DIM
 #define TW_HEAD_DIM 128
+#endif
+#ifndef TW_V_DIM
+#define TW_V_DIM TW_HEAD_DIM
 #endif
 
 namespace {
@@ -41,15 +47,18 @@ static_assert(D == 64 || D == 128, "the tcgen05 attention is built for head size
 constexpr int BM = 128;                       // rows of a query tile = TMEM lanes
 constexpr int NQ = 2;                         // query tiles per block
 constexpr int BN = 128;                       // keys per tile
-constexpr int KB = D / 64;                    // 64-column blocks of a row of q, k or v
+constexpr int DV = TW_V_DIM;
+static_assert(DV == 64 || DV == 128, "the tcgen05 attention is built for value sizes 64 and 128");
+constexpr int KB = D / 64;                    // 64-column blocks of a row of q or k
+constexpr int VB = DV / 64;                   // 64-column blocks of a row of v
 constexpr int BLK = 128 * 128;                // bytes of a [128 rows][64 columns] swizzled block
-constexpr int KV_STAGES = D == 128 ? 2 : 4;   // K and V have rings of their own
+constexpr int KV_STAGES = D == 64 && DV == 64 ? 4 : 2;   // K and V have rings of their own
 constexpr int Q_BYTES = NQ * KB * BLK;
-constexpr int KV_STAGE_BYTES = KB * BLK;
-constexpr int SMEM_TILES = Q_BYTES + 2 * KV_STAGES * KV_STAGE_BYTES;
+constexpr int K_STAGE_BYTES = KB * BLK, V_STAGE_BYTES = VB * BLK;
+constexpr int SMEM_TILES = Q_BYTES + KV_STAGES * (K_STAGE_BYTES + V_STAGE_BYTES);
 constexpr int SMEM = SMEM_TILES + 1024 /* alignment slack */ + 256 /* barriers */;
 constexpr int THREADS = 320;                  // warp 0: TMA, warp 1: MMA, warps 2-5 / 6-9: softmax of tile 0 / 1
-constexpr int TMEM_COLS = 512;                // S of both tiles (2 x 128 columns; P over its first 64), O of both tiles (2 x D)
+constexpr int TMEM_COLS = 512;                // S of both tiles (2 x 128 columns; P over its first 64), O of both tiles (2 x DV)
 constexpr int O_COL = 256;
 constexpr float RESCALE_THRESHOLD = 8.f;      // log2 units
 #define NEG_INF (-INFINITY)
@@ -108,7 +117,8 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                         const int* __restrict__ seq_kv_len, const int* __restrict__ seq_slot,
                         const int* __restrict__ block_table, int table_stride, int Hq, int Hkv, int page_size,
-                        int num_pages, int window, float scale_log2e, int skip_single, int* status) {
+                        int num_pages, int window, float scale_log2e, int skip_single, const float* __restrict__ gate,
+                        int* status) {
     extern __shared__ unsigned char smem_raw[];
     TW_TIMELINE_SCOPE(TW_K_ATTN_PREFILL);
     if (threadIdx.x == 0) TW_TRACE_AT(0, 0, 5);
@@ -133,14 +143,15 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int row_end = min(rows_total, row0 + NQ * BM);
     const int nq = row_end - row0 > BM ? 2 : 1;
     const int pos_first = pos0 + row0 / G, pos_last = pos0 + (row_end - 1) / G;
-    const int j_begin = (window > 0 && pos_first - window + 1 > 0) ? (pos_first - window + 1) / BN : 0;
+    const int lo_block = tw_first_key(pos_first, window);             // no row of the block sees a key before this one
+    const int j_begin = lo_block / BN;
     const int ntiles = pos_last / BN + 1 - j_begin;
     const int tail_rows = max(0, (j_begin + ntiles) * BN - kv_len);  // rows of the last tile that hold no key
 
     unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     unsigned char* q_s = tiles;                                      // [NQ][KB][128 rows][128 B]
     unsigned char* k_s = q_s + Q_BYTES;                              // [KV_STAGES][KB][128 keys][128 B]
-    unsigned char* v_s = k_s + KV_STAGES * KV_STAGE_BYTES;           // [KV_STAGES][KB][128 keys][128 B]
+    unsigned char* v_s = k_s + KV_STAGES * K_STAGE_BYTES;            // [KV_STAGES][VB][128 keys][128 B]
     uint64_t* k_full = reinterpret_cast<uint64_t*>(tiles + SMEM_TILES);
     uint64_t* k_empty = k_full + KV_STAGES;
     uint64_t* v_full = k_empty + KV_STAGES;
@@ -173,18 +184,20 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         int row_coord = -1;
         if (lane < boxes) {
             const int key0 = (j_begin + i) * BN + lane * box_rows;
-            if (key0 < kv_len) {
+            if (key0 < kv_len && key0 + box_rows <= lo_block) {
+                row_coord = num_pages * Hkv * page_size;              // beyond the cache: zeros
+            } else if (key0 < kv_len) {
                 const int blk = key0 / page_size;
                 const int page = blk < table_stride ? table[blk] : -1;
                 if (page < 0 || page >= num_pages) atomicOr(status, TW_ERR_PAGE);
                 else row_coord = (page * Hkv + kvh) * page_size + (key0 - blk * page_size);
             }
         }
-        const uint32_t bytes = (uint32_t)__popc(__ballot_sync(0xffffffffu, row_coord >= 0)) * KB * box_rows * 128;
+        const uint32_t box_bytes = (uint32_t)__popc(__ballot_sync(0xffffffffu, row_coord >= 0)) * box_rows * 128;
         int ok = 1;
         if (lane == 0) {
             ok = (!*aborted && mbar_wait(&k_empty[st], parity ^ 1, status)) ? 1 : 0;
-            if (ok) mbar_expect_tx(&k_full[st], bytes); else *aborted = 1;
+            if (ok) mbar_expect_tx(&k_full[st], box_bytes * KB); else *aborted = 1;
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);
         if (!ok) return false;
@@ -192,11 +205,11 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         if (row_coord >= 0) {
 #pragma unroll
             for (int kb = 0; kb < KB; ++kb)
-                tma_load_2d(k_s + st * KV_STAGE_BYTES + kb * BLK + lane * box_rows * 128, &map_k, &k_full[st], kb * 64, row_coord);
+                tma_load_2d(k_s + st * K_STAGE_BYTES + kb * BLK + lane * box_rows * 128, &map_k, &k_full[st], kb * 64, row_coord);
         }
         if (lane == 0) {
             ok = (!*aborted && mbar_wait(&v_empty[st], parity ^ 1, status)) ? 1 : 0;
-            if (ok) mbar_expect_tx(&v_full[st], bytes); else *aborted = 1;
+            if (ok) mbar_expect_tx(&v_full[st], box_bytes * VB); else *aborted = 1;
         }
         ok = __shfl_sync(0xffffffffu, ok, 0);
         if (!ok) {                                   // K of this tile is in flight: let it land
@@ -206,8 +219,8 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         if (lane == 0) TW_TRACE_AT(1, i, 2);
         if (row_coord >= 0) {
 #pragma unroll
-            for (int kb = 0; kb < KB; ++kb)
-                tma_load_2d(v_s + st * KV_STAGE_BYTES + kb * BLK + lane * box_rows * 128, &map_v, &v_full[st], kb * 64, row_coord);
+            for (int vb = 0; vb < VB; ++vb)
+                tma_load_2d(v_s + st * V_STAGE_BYTES + vb * BLK + lane * box_rows * 128, &map_v, &v_full[st], vb * 64, row_coord);
         }
         return true;
     };
@@ -265,9 +278,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             // zero them once the copies have landed, then tell the MMA thread.
             const int last = ntiles - 1;
             if (mbar_wait(&v_full[last % KV_STAGES], (last / KV_STAGES) & 1, status)) {
-                unsigned char* vt = v_s + (last % KV_STAGES) * KV_STAGE_BYTES;
-                for (int idx = lane; idx < tail_rows * KB * 8; idx += 32) {
-                    const int r = BN - tail_rows + idx / (KB * 8), rest = idx % (KB * 8);
+                unsigned char* vt = v_s + (last % KV_STAGES) * V_STAGE_BYTES;
+                for (int idx = lane; idx < tail_rows * VB * 8; idx += 32) {
+                    const int r = BN - tail_rows + idx / (VB * 8), rest = idx % (VB * 8);
                     *reinterpret_cast<uint4*>(vt + (rest >> 3) * BLK + r * 128 + ((rest & 7) << 4)) = make_uint4(0u, 0u, 0u, 0u);
                 }
                 fence_proxy_async();
@@ -289,12 +302,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         // this thread does anything else, so whatever a group of MMAs needs beside P (V of the tile, K of
         // the next one) is waited for before P, and the groups follow one another without a break.
         if (lane == 0 && ntiles > 0) {
-            const uint32_t idesc_s = instr_desc(BN), idesc_o = instr_desc(D, true);
+            const uint32_t idesc_s = instr_desc(BN), idesc_o = instr_desc(DV, true);
             // Descriptors are built once; per MMA only a constant is added to the address field (a thread
             // that computes a descriptor from scratch before each MMA issues them slower than they execute).
             const uint64_t q_desc = smem_desc(q_s, 0), k_desc = smem_desc(k_s, 0), v_desc = smem_desc_mn_major(v_s, BLK);
             auto issue_s = [&](int x, int i) {
-                const uint64_t kd = k_desc + (uint64_t)((i % KV_STAGES) * (KV_STAGE_BYTES >> 4));
+                const uint64_t kd = k_desc + (uint64_t)((i % KV_STAGES) * (K_STAGE_BYTES >> 4));
                 const uint64_t qd = q_desc + (uint64_t)(x * KB * (BLK >> 4));
 #pragma unroll
                 for (int kb = 0; kb < KB; ++kb)
@@ -305,10 +318,10 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 umma_commit(&s_full[x]);
             };
             auto issue_o = [&](int x, int i) {
-                const uint64_t vd = v_desc + (uint64_t)((i % KV_STAGES) * (KV_STAGE_BYTES >> 4));
+                const uint64_t vd = v_desc + (uint64_t)((i % KV_STAGES) * (V_STAGE_BYTES >> 4));
 #pragma unroll
                 for (int k = 0; k < BN / 16; ++k)
-                    umma_bf16_ts(tmem_base + O_COL + x * D, tmem_base + x * BN + k * 8, vd + (uint64_t)(k * (2048 >> 4)),
+                    umma_bf16_ts(tmem_base + O_COL + x * DV, tmem_base + x * BN + k * 8, vd + (uint64_t)(k * (2048 >> 4)),
                                  idesc_o, (i > 0 || k > 0) ? 1u : 0u);
                 umma_commit(&o_done[x]);
             };
@@ -355,9 +368,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         const bool valid = r < rows_total;
         const int t = valid ? r / G : (rows_total - 1) / G;
         const int pos = pos0 + t;
-        const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+        const int lo = tw_first_key(pos, window);
         const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
-        const uint32_t s_addr = lane_addr + x * BN, o_addr = lane_addr + O_COL + x * D;
+        const uint32_t s_addr = lane_addr + x * BN, o_addr = lane_addr + O_COL + x * DV;
         float m_used = NEG_INF, l = 0.f;
         bool ok = true;
         for (int i = 0; i < ntiles; ++i) {
@@ -417,7 +430,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 tc_fence_after();
                 {
 #pragma unroll
-                    for (int c = 0; c < D; c += 32) {
+                    for (int c = 0; c < DV; c += 32) {
                         uint32_t o[32];
                         tmem_ld32_nowait(o_addr + c, o);
                         tmem_wait_ld();
@@ -444,10 +457,11 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             *aborted = 1;
         } else if (ntiles > 0) {
             tc_fence_after();
-            const float inv = l > 0.f ? 1.f / l : 0.f;
-            bf16* orow = out + (size_t)(n0 + t) * out_stride + (size_t)(kvh * G + (r - t * G)) * D;
+            float inv = l > 0.f ? 1.f / l : 0.f;
+            if (gate && valid) inv *= __ldg(gate + (size_t)(n0 + t) * Hq + kvh * G + (r - t * G));
+            bf16* orow = out + (size_t)(n0 + t) * out_stride + (size_t)(kvh * G + (r - t * G)) * DV;
 #pragma unroll
-            for (int c = 0; c < D; c += 32) {
+            for (int c = 0; c < DV; c += 32) {
                 uint32_t o[32];
                 tmem_ld32_nowait(o_addr + c, o);
                 tmem_wait_ld();
@@ -493,12 +507,12 @@ TW_EXPORT int tw_attn_prefill_tc5_supported(int page_size) {
 
 // Attention for the requests of the batch that bring several tokens (with skip_single, requests
 // with one token are left to the decode kernel).  q [tokens, Hq * D] and out [tokens, Hq * D] are
-// bf16 with 16-byte aligned rows; the cache is [pages, Hkv, page_size, D] bf16.
+// bf16 with 16-byte aligned rows; the cache is [pages, Hkv, page_size, D] bf16 (values and out: heads of DV).
 TW_EXPORT int tw_attn_prefill_tc5(void* out, int out_stride, const void* q, int q_stride, const int* seq_q_start,
                                   const int* seq_q_len, const int* seq_kv_len, const int* seq_slot,
                                   const int* block_table, int table_stride, const void* k_cache, const void* v_cache,
                                   int n_seqs, int max_q_len, int Hq, int Hkv, int page_size, int num_pages, int window,
-                                  float scale, int skip_single, int* status, cudaStream_t stream) {
+                                  float scale, int skip_single, const float* gate, int* status, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
     if (Hkv <= 0 || Hq % Hkv || !tw_attn_prefill_tc5_supported(page_size) || scale <= 0.f) return (int)cudaErrorInvalidValue;
     if ((reinterpret_cast<uintptr_t>(out) & 15) || (reinterpret_cast<uintptr_t>(q) & 15) || (out_stride & 7) || (q_stride & 7) ||
@@ -512,13 +526,13 @@ TW_EXPORT int tw_attn_prefill_tc5(void* out, int out_stride, const void* q, int 
     }
     const int box_rows = page_size < BN ? page_size : BN;
     const long long rows = (long long)num_pages * Hkv * page_size;
-    if (rows >= (1ll << 31)) return (int)cudaErrorInvalidValue;
+    if (rows >= (1ll << 31) - 1) return (int)cudaErrorInvalidValue;
     CUtensorMap mk, mv;
     if (int e = get_map(k_cache, rows, D, box_rows, &mk)) return e;
-    if (int e = get_map(v_cache, rows, D, box_rows, &mv)) return e;
+    if (int e = get_map(v_cache, rows, DV, box_rows, &mv)) return e;
     const int G = Hq / Hkv;
     dim3 grid(((max_q_len * G + NQ * BM - 1) / (NQ * BM)) * Hkv, n_seqs);
     return tw_launch(attn_prefill_tc5_kernel, grid, dim3(THREADS), (size_t)SMEM, stream, 1, mk, mv, (bf16*)out, out_stride,
                      (const bf16*)q, q_stride, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, table_stride,
-                     Hq, Hkv, page_size, num_pages, window, scale * 1.4426950408889634f, skip_single, status);
+                     Hq, Hkv, page_size, num_pages, window, scale * 1.4426950408889634f, skip_single, gate, status);
 }

@@ -75,6 +75,33 @@ __device__ __forceinline__ float tw_block_max(float v, float* scratch) {
     return scratch[32];
 }
 
+// What stands between two matrix products of a feed-forward, in fp32.
+enum : int { TW_ACT_NONE = 0, TW_ACT_SILU = 1, TW_ACT_GELU_TANH = 2, TW_ACT_RELU_SQUARED = 3 };
+__device__ __forceinline__ float tw_activate(float z, int act) {
+    if (act == TW_ACT_SILU) return z / (1.0f + expf(-z));
+    if (act == TW_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    if (act == TW_ACT_RELU_SQUARED) { z = fmaxf(z, 0.f); return z * z; }
+    return z;
+}
+// What a matrix product does to its sums before it stores them: add a bias (one per weight row; may be null), then
+// apply the activation -- to every value, or, where the rows alternate between gates and ups, to the gate alone.  Of a
+// product split over k the first slice gets the bias and no slice an activation.
+struct TwEpilogue {
+    const __nv_bfloat16* bias;
+    int act;
+};
+__device__ __forceinline__ float tw_biased(const TwEpilogue& ep, float v, int row) {
+    return ep.bias ? v + __bfloat162float(ep.bias[row]) : v;
+}
+
+// The first key position that a query at position `pos` sees.  reach > 0: a sliding window of that many keys, the
+// query's own position included; reach < 0: chunks of -reach positions, counted from position 0 of the request, of
+// which a query sees its own; 0: every key.  Never falls as `pos` grows, so a block of rows may stop at its first row's.
+__device__ __forceinline__ int tw_first_key(int pos, int reach) {
+    if (reach > 0) return max(pos - reach + 1, 0);
+    return reach < 0 ? pos - pos % -reach : 0;
+}
+
 #define TW_LAUNCH_CHECK() (int)cudaGetLastError()
 
 // ---------------------------------------------------------------------------------------

@@ -868,15 +868,16 @@ TW_EXPORT int tw_softcap(float* x, long long total, float cap, cudaStream_t stre
 }
 
 // ---------------------------------------------------------------------------
-// SwiGLU activation: out[n, i] = silu(gate[n, i]) * up[n, i], silu(z) = z / (1 + exp(-z)),
-// with gate = gate_up[n, i] and up = gate_up[n, I + i] (rows packed [gate; up]).
+// Gated activation: out[n, i] = act(gate[n, i]) * up[n, i] (act: silu, the tanh form of gelu, the square of relu),
+// with gate = gate_up[n, i] and up = gate_up[n, I + i] (rows packed [gate; up]); `bias` (2 I values in the order of the
+// columns, of the rows' type, or null) is added to both first, in fp32.
 // Reference: flow_engine/model.py:76-80.
 // ---------------------------------------------------------------------------
 // With `interleaved` the columns come in groups of 16: eight gates, then their eight ups
 // (the packing the fused small-batch kernel wants); otherwise all gates, then all ups.
 template <typename T>
 __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_up, int inter, long total,
-                                int interleaved) {
+                                int interleaved, int act, const T* __restrict__ bias) {
     TW_TIMELINE_SCOPE(TW_K_SILU_MUL);
     tw_grid_wait();
     TW_TIMELINE_MARK();
@@ -888,16 +889,17 @@ __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_
         const int i = (int)(idx - n * inter);
         const int gcol = interleaved ? ((i >> 3) << 4) + (i & 7) : i;
         const int ucol = interleaved ? gcol + 8 : inter + i;
-        const float g = tw_to_float(gate_up[n * 2 * inter + gcol]);
-        const float u = tw_to_float(gate_up[n * 2 * inter + ucol]);
-        const float act = g / (1.0f + expf(-g));
-        out[idx] = tw_from_float<T>(act * u);
+        float g = tw_to_float(gate_up[n * 2 * inter + gcol]);
+        float u = tw_to_float(gate_up[n * 2 * inter + ucol]);
+        if (bias) { g += tw_to_float(bias[gcol]); u += tw_to_float(bias[ucol]); }
+        out[idx] = tw_from_float<T>(tw_activate(g, act) * u);
     }
 }
 
 // bf16 with the intermediate size a multiple of 8: a thread handles 8 outputs with 16-byte accesses.
 __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate_up,
-                                       int inter, long total8, int interleaved) {
+                                       int inter, long total8, int interleaved, int act,
+                                       const __nv_bfloat16* __restrict__ bias) {
     TW_TIMELINE_SCOPE(TW_K_SILU_MUL);
     tw_grid_wait();
     TW_TIMELINE_MARK();
@@ -917,8 +919,13 @@ __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __
         __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float2 g = __bfloat1622float2(g2[e]), u = __bfloat1622float2(u2[e]);
-            o2[e] = __floats2bfloat162_rn(g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y);
+            float2 g = __bfloat1622float2(g2[e]), u = __bfloat1622float2(u2[e]);
+            if (bias) {
+                const float2 bg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(bias + (interleaved ? j * 16 : j * 8) + 2 * e));
+                const float2 bu = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(bias + (interleaved ? j * 16 + 8 : inter + j * 8) + 2 * e));
+                g.x += bg.x; g.y += bg.y; u.x += bu.x; u.y += bu.y;
+            }
+            o2[e] = __floats2bfloat162_rn(tw_activate(g.x, act) * u.x, tw_activate(g.y, act) * u.y);
         }
         *reinterpret_cast<uint4*>(out + n * (long)inter + j * 8) = ov;
     }
@@ -949,7 +956,8 @@ __device__ __forceinline__ float4 tw_sum_slices4(const float* p, int nsplit, siz
 }
 
 __global__ void silu_mul_slices_kernel(__nv_bfloat16* __restrict__ out, const float* __restrict__ partial, int nsplit,
-                                       size_t split_stride, int inter, long total4, int interleaved) {
+                                       size_t split_stride, int inter, long total4, int interleaved, int act,
+                                       const __nv_bfloat16* __restrict__ bias) {
     TW_TIMELINE_SCOPE(TW_K_SILU_MUL);
     tw_grid_wait();
     TW_TIMELINE_MARK();
@@ -963,19 +971,23 @@ __global__ void silu_mul_slices_kernel(__nv_bfloat16* __restrict__ out, const fl
         const int gcol = interleaved ? ((i >> 3) << 4) + (i & 7) : i;
         const int ucol = interleaved ? gcol + 8 : inter + i;
         const float* row = partial + (size_t)n * 2 * inter;
-        const float4 g = tw_sum_slices4(row + gcol, nsplit, split_stride);
-        const float4 u = tw_sum_slices4(row + ucol, nsplit, split_stride);
+        float4 g = tw_sum_slices4(row + gcol, nsplit, split_stride);
+        float4 u = tw_sum_slices4(row + ucol, nsplit, split_stride);
+        if (bias) {
+            g.x += tw_to_float(bias[gcol]); g.y += tw_to_float(bias[gcol + 1]); g.z += tw_to_float(bias[gcol + 2]); g.w += tw_to_float(bias[gcol + 3]);
+            u.x += tw_to_float(bias[ucol]); u.y += tw_to_float(bias[ucol + 1]); u.z += tw_to_float(bias[ucol + 2]); u.w += tw_to_float(bias[ucol + 3]);
+        }
         uint2 packed;
         *reinterpret_cast<__nv_bfloat162*>(&packed.x) =
-            __floats2bfloat162_rn(g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y);
+            __floats2bfloat162_rn(tw_activate(g.x, act) * u.x, tw_activate(g.y, act) * u.y);
         *reinterpret_cast<__nv_bfloat162*>(&packed.y) =
-            __floats2bfloat162_rn(g.z / (1.0f + expf(-g.z)) * u.z, g.w / (1.0f + expf(-g.w)) * u.w);
+            __floats2bfloat162_rn(tw_activate(g.z, act) * u.z, tw_activate(g.w, act) * u.w);
         *reinterpret_cast<uint2*>(out + n * (long)inter + i) = packed;
     }
 }
 
 TW_EXPORT int tw_silu_mul_slices(void* out, const float* partial, int nsplit, long split_stride, int n_rows, int inter,
-                                 int interleaved, cudaStream_t stream) {
+                                 int interleaved, int act, const void* bias, cudaStream_t stream) {
     if (n_rows <= 0 || inter <= 0) return 0;
     if (nsplit < 1 || (inter & 3) || (interleaved && (inter & 7)) || (split_stride & 3) ||
         ((uintptr_t)partial & 15) || ((uintptr_t)out & 7))
@@ -983,32 +995,79 @@ TW_EXPORT int tw_silu_mul_slices(void* out, const float* partial, int nsplit, lo
     const long total4 = (long)n_rows * (inter >> 2);
     const long blocks = (total4 + 255) / 256;
     tw_launch(silu_mul_slices_kernel, dim3((int)(blocks > 4096 ? 4096 : blocks)), dim3(256), 0, stream, 1, (__nv_bfloat16*)out,
-              partial, nsplit, (size_t)split_stride, inter, total4, interleaved);
+              partial, nsplit, (size_t)split_stride, inter, total4, interleaved, act, (const __nv_bfloat16*)bias);
     return TW_LAUNCH_CHECK();
 }
 
-TW_EXPORT int tw_silu_mul(void* out, const void* gate_up, int n_rows, int inter, int interleaved, int dtype,
-                          cudaStream_t stream) {
+TW_EXPORT int tw_silu_mul(void* out, const void* gate_up, int n_rows, int inter, int interleaved, int act, const void* bias,
+                          int dtype, cudaStream_t stream) {
     const long total = (long)n_rows * inter;
     if (total <= 0) return 0;
     long blocks = (total + 255) / 256;
     if (blocks > 148L * 16) blocks = 148L * 16;
-    if (dtype == TW_BF16 && (inter & 7) == 0) {
+    if (dtype == TW_BF16 && (inter & 7) == 0 && ((uintptr_t)bias & 3) == 0) {
         const long total8 = total >> 3;
         long b8 = (total8 + 255) / 256;
         if (b8 > 148L * 16) b8 = 148L * 16;
         tw_launch(silu_mul_bf16x8_kernel, dim3((int)b8), dim3(256), 0, stream, 1, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate_up, inter,
-                                                            total8, interleaved);
+                                                            total8, interleaved, act, (const __nv_bfloat16*)bias);
         return TW_LAUNCH_CHECK();
     }
     if (dtype == TW_F32)
         tw_launch(silu_mul_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, 1, (float*)out, (const float*)gate_up, inter, total,
-                                                                interleaved);
+                                                                interleaved, act, (const float*)bias);
     else
         tw_launch(silu_mul_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(256), 0, stream, 1, (__nv_bfloat16*)out,
                                                                         (const __nv_bfloat16*)gate_up, inter, total,
-                                                                        interleaved);
+                                                                        interleaved, act, (const __nv_bfloat16*)bias);
     return TW_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------------------
+// x[i] = act(x[i] + bias[i mod cols]) in place on contiguous rows: the activation of a feed-forward without a gate.
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void activate_kernel(T* __restrict__ x, const T* __restrict__ bias, int cols, long total, int act) {
+    tw_grid_wait();
+    tw_grid_launch_dependents();
+    const long step = (long)gridDim.x * blockDim.x;
+    for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += step) {
+        float v = tw_to_float(x[i]);
+        if (bias) v += tw_to_float(bias[i % cols]);
+        x[i] = tw_from_float<T>(tw_activate(v, act));
+    }
+}
+// bf16, eight values per access (the row length a multiple of 8)
+__global__ void activate_bf16x8_kernel(uint4* __restrict__ x, const uint4* __restrict__ bias, int cols8, long total8, int act) {
+    tw_grid_wait();
+    tw_grid_launch_dependents();
+    const long step = (long)gridDim.x * blockDim.x;
+    for (long i = (long)blockIdx.x * blockDim.x + threadIdx.x; i < total8; i += step) {
+        uint4 raw = x[i];
+        const uint4 braw = bias ? bias[i % cols8] : make_uint4(0u, 0u, 0u, 0u);
+        __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&raw);
+        const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&braw);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(p[e]), g = __bfloat1622float2(b[e]);
+            p[e] = __floats2bfloat162_rn(tw_activate(f.x + g.x, act), tw_activate(f.y + g.y, act));
+        }
+        x[i] = raw;
+    }
+}
+
+TW_EXPORT int tw_activate_rows(void* x, const void* bias, int n_rows, int cols, int act, int dtype, cudaStream_t stream) {
+    if (n_rows <= 0 || cols <= 0) return 0;
+    const bool vec = dtype == TW_BF16 && (cols & 7) == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)bias & 15) == 0;
+    const long total = (long)n_rows * cols / (vec ? 8 : 1);
+    const long want = (total + 255) / 256;
+    const dim3 blocks((unsigned)(want < 148L * 16 ? want : 148L * 16));
+    if (vec)
+        return tw_launch(activate_bf16x8_kernel, blocks, dim3(256), 0, stream, 1, (uint4*)x, (const uint4*)bias, cols / 8, total, act);
+    if (dtype == TW_F32)
+        return tw_launch(activate_kernel<float>, blocks, dim3(256), 0, stream, 1, (float*)x, (const float*)bias, cols, total, act);
+    return tw_launch(activate_kernel<__nv_bfloat16>, blocks, dim3(256), 0, stream, 1, (__nv_bfloat16*)x, (const __nv_bfloat16*)bias,
+                     cols, total, act);
 }
 
 // ---------------------------------------------------------------------------

@@ -49,7 +49,7 @@ constexpr int WARPS = TW_GEMM_WARPS;
 constexpr int ROWS_PER_BLOCK = WARPS * 16;
 constexpr int CHUNK = 64;      // values of k per step: a thread reads 32 contiguous bytes of each of its rows
 
-enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_PARTIAL = 2, OUT_SILU_MUL = 3, OUT_EARLY_DEPENDENTS = 16 /* flag, or-ed in */ };
+enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_PARTIAL = 2, OUT_GATED = 3, OUT_EARLY_DEPENDENTS = 16 /* flag, or-ed in */ };
 
 struct Frag {          // 16 consecutive values of k of one row
     uint4 lo, hi;
@@ -59,10 +59,13 @@ struct Frag {          // 16 consecutive values of k of one row
 // share its values of k and add their sums through shared memory: twice the warps for a matrix with few
 // row tiles whose k cannot be split over blocks (the SiLU.mul output needs whole sums): 27,648 x 5,120
 // at 8 rows 52 -> 45 us.
-template <int NT, int KS>
+// EPI: the sums get a bias or an activation other than SiLU on gates (kept apart, since it takes registers from the
+// stream of the plain form).
+template <int NT, int KS, bool EPI>
 __global__ void __launch_bounds__(WARPS * 32, (NT == 1 ? 5 : 0))
 gemm_smallm_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x, int M, int N, int K, int kper,
-                   void* __restrict__ out, int out_mode, int out_stride, const void* next_weights, long long next_bytes) {
+                   void* __restrict__ out, int out_mode, int out_stride, const TwEpilogue ep, const void* next_weights,
+                   long long next_bytes) {
     constexpr int TILES = WARPS / KS;                  // 16-row tiles of a block
     __shared__ float s_part[KS > 1 ? TILES * 32 * NT * 4 : 1];
     TW_TIMELINE_SCOPE(TW_K_GEMM_SMALLM);
@@ -172,23 +175,34 @@ gemm_smallm_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x, int M
         for (int e = 0; e < 2; ++e) {
             const int tok = t * 8 + 2 * c + e;
             if (tok >= M) continue;
-            if (out_mode == OUT_SILU_MUL) {
+            if (out_mode == OUT_GATED) {
                 // weight rows come in groups of 16: eight gate rows, then the eight up rows that belong to
-                // them, so row ra is a gate and row rb its up: out[tok, r0 / 2 + g] = silu(gate) * up
+                // them, so row ra is a gate and row rb its up: out[tok, r0 / 2 + g] = act(gate) * up
                 if (wb_ok) {
-                    const float gt = acc[t][e], up = acc[t][2 + e];
+                    float gt = acc[t][e], up = acc[t][2 + e];
+                    if constexpr (EPI) { gt = tw_biased(ep, gt, ra); up = tw_biased(ep, up, rb); }
                     reinterpret_cast<bf16*>(out)[(size_t)tok * out_stride + (r0 >> 1) + g] =
-                        __float2bfloat16_rn(gt / (1.0f + expf(-gt)) * up);
+                        __float2bfloat16_rn(tw_activate(gt, EPI ? ep.act : (int)TW_ACT_SILU) * up);
                 }
-            } else if (out_mode == OUT_BF16) {
+                continue;
+            }
+            float xa = acc[t][e], xb = acc[t][2 + e];
+            if constexpr (EPI) {
+                if (blockIdx.y == 0) {
+                    if (wa_ok) xa = tw_biased(ep, xa, ra);
+                    if (wb_ok) xb = tw_biased(ep, xb, rb);
+                }
+                if (out_mode != OUT_PARTIAL) { xa = tw_activate(xa, ep.act); xb = tw_activate(xb, ep.act); }
+            }
+            if (out_mode == OUT_BF16) {
                 bf16* o = reinterpret_cast<bf16*>(out) + (size_t)tok * out_stride;
-                if (wa_ok) o[ra] = __float2bfloat16_rn(acc[t][e]);
-                if (wb_ok) o[rb] = __float2bfloat16_rn(acc[t][2 + e]);
+                if (wa_ok) o[ra] = __float2bfloat16_rn(xa);
+                if (wb_ok) o[rb] = __float2bfloat16_rn(xb);
             } else {
                 float* o = reinterpret_cast<float*>(out) +
                            (out_mode == OUT_PARTIAL ? ((size_t)blockIdx.y * M + tok) * out_stride : (size_t)tok * out_stride);
-                if (wa_ok) o[ra] = acc[t][e];
-                if (wb_ok) o[rb] = acc[t][2 + e];
+                if (wa_ok) o[ra] = xa;
+                if (wb_ok) o[rb] = xb;
             }
         }
     }
@@ -218,18 +232,22 @@ __global__ void reduce_partial_kernel(T* __restrict__ out, const float* __restri
 }  // namespace
 
 // out_mode 0: bf16 [M, out_stride]; 1: fp32 [M, out_stride]; 2: fp32 partial sums [ksplit, M, out_stride]
-// (then kper < K); 3: bf16 [M, out_stride] = silu(gate) * up for weights whose rows alternate between eight
+// (then kper < K); 3: bf16 [M, out_stride] = act(gate) * up for weights whose rows alternate between eight
 // gate rows and their eight up rows (N a multiple of 16, no split).  K must be a multiple of 8; kper of 32.
+// `bias` (bf16 [N], in the order of the rows, or null) and `act`: see TwEpilogue.
 TW_EXPORT int tw_gemm_smallm(const void* w, const void* x, int M, int N, int K, int kper, void* out, int out_mode,
-                             int out_stride, const void* next_weights, long long next_bytes, cudaStream_t stream) {
+                             int out_stride, const void* bias, int act, const void* next_weights, long long next_bytes,
+                             cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if ((uintptr_t)next_weights & 15) return (int)cudaErrorMisalignedAddress;
     if (!next_weights || next_bytes < 0) next_bytes = 0;
-    if (M > 64 || K <= 0 || (K & 7) || kper <= 0 || (kper & 31) || (out_mode & ~OUT_EARLY_DEPENDENTS) < 0 || (out_mode & ~OUT_EARLY_DEPENDENTS) > 3 || ((out_mode & ~OUT_EARLY_DEPENDENTS) == OUT_SILU_MUL && (N & 15)))
+    if (M > 64 || K <= 0 || (K & 7) || kper <= 0 || (kper & 31) || (out_mode & ~OUT_EARLY_DEPENDENTS) < 0 || (out_mode & ~OUT_EARLY_DEPENDENTS) > 3 || ((out_mode & ~OUT_EARLY_DEPENDENTS) == OUT_GATED && (N & 15)) ||
+        act < TW_ACT_NONE || act > TW_ACT_RELU_SQUARED || (act != TW_ACT_NONE && (out_mode & ~OUT_EARLY_DEPENDENTS) == OUT_PARTIAL))
         return (int)cudaErrorInvalidValue;
     const int ksplit = (K + kper - 1) / kper;
     if (ksplit > 1 && (out_mode & ~OUT_EARLY_DEPENDENTS) != OUT_PARTIAL) return (int)cudaErrorInvalidValue;
     dim3 grid((N + ROWS_PER_BLOCK - 1) / ROWS_PER_BLOCK, ksplit);
+    const TwEpilogue ep{(const bf16*)bias, act};
     const bf16* wp = (const bf16*)w;
     const bf16* xp = (const bf16*)x;
     static int sm_count = 0;
@@ -240,22 +258,15 @@ TW_EXPORT int tw_gemm_smallm(const void* w, const void* x, int M, int N, int K, 
     }
     // few blocks for the GPU (under 3.2 per SM, five fit) and enough k for two warps: two warps per row tile
     const bool pair_warps = M <= 8 && (long)grid.x * grid.y * 10 <= (long)sm_count * 32 && kper >= 512;
-    if (pair_warps) {
-        grid.x = (N + (WARPS / 2) * 16 - 1) / ((WARPS / 2) * 16);
-        tw_launch(gemm_smallm_kernel<1, 2>, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride,
-                  next_weights, next_bytes);
-    } else if (M <= 8)
-        tw_launch(gemm_smallm_kernel<1, 1>, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride,
-                  next_weights, next_bytes);
-    else if (M <= 16)
-        tw_launch(gemm_smallm_kernel<2, 1>, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride,
-                  next_weights, next_bytes);
-    else if (M <= 32)
-        tw_launch(gemm_smallm_kernel<4, 1>, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride,
-                  next_weights, next_bytes);
-    else
-        tw_launch(gemm_smallm_kernel<8, 1>, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride,
-                  next_weights, next_bytes);
+    const bool epi = bias || act != ((out_mode & ~OUT_EARLY_DEPENDENTS) == OUT_GATED ? TW_ACT_SILU : TW_ACT_NONE);
+    if (pair_warps) grid.x = (N + (WARPS / 2) * 16 - 1) / ((WARPS / 2) * 16);
+    auto kernel = pair_warps ? (epi ? gemm_smallm_kernel<1, 2, true> : gemm_smallm_kernel<1, 2, false>)
+                : M <= 8     ? (epi ? gemm_smallm_kernel<1, 1, true> : gemm_smallm_kernel<1, 1, false>)
+                : M <= 16    ? (epi ? gemm_smallm_kernel<2, 1, true> : gemm_smallm_kernel<2, 1, false>)
+                : M <= 32    ? (epi ? gemm_smallm_kernel<4, 1, true> : gemm_smallm_kernel<4, 1, false>)
+                             : (epi ? gemm_smallm_kernel<8, 1, true> : gemm_smallm_kernel<8, 1, false>);
+    tw_launch(kernel, dim3(grid), dim3(WARPS * 32), 0, stream, 1, wp, xp, M, N, K, kper, out, out_mode, out_stride, ep,
+              next_weights, next_bytes);
     return TW_LAUNCH_CHECK();
 }
 

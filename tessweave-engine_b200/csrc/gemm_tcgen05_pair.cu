@@ -46,7 +46,7 @@ constexpr int STAGES = 7;
 constexpr int TMEM_COLS = 512;         // two accumulators of 256 columns: the epilogue of a tile overlaps the next tile's MMAs
 constexpr int SMEM = STAGES * STAGE_BYTES + 1024 /* alignment slack */ + 256 /* barriers */;
 
-enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_SILU_MUL = 3 };
+enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_GATED = 3 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
     uint32_t r;
@@ -90,10 +90,29 @@ __device__ __forceinline__ uint32_t instr_desc_pair() {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(256 >> 4) << 24);
 }
 
-// One accumulator row of 16 columns, written the way `out_mode` says.
-__device__ __forceinline__ void store_chunk(const uint32_t (&v)[16], void* out, int out_mode, int out_stride, int row, int col,
-                                            int rows_b) {
-    if (out_mode == OUT_SILU_MUL) {
+// One accumulator row of 16 columns, biased, activated and written the way `ep` and `out_mode` say.
+__device__ __forceinline__ void store_chunk(uint32_t (&v)[16], void* out, int out_mode, int out_stride, int row, int col,
+                                            int rows_b, const TwEpilogue& ep) {
+    if (ep.bias) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j)
+            if (col + j < rows_b) v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(ep.bias[col + j]));
+    }
+    if (out_mode != OUT_GATED && ep.act != TW_ACT_NONE) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(tw_activate(__uint_as_float(v[j]), ep.act));
+    }
+    if (out_mode == OUT_GATED && ep.act != TW_ACT_SILU) {
+        uint4 p;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&p);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            h[j] = __floats2bfloat162_rn(tw_activate(__uint_as_float(v[2 * j]), ep.act) * __uint_as_float(v[8 + 2 * j]),
+                                         tw_activate(__uint_as_float(v[2 * j + 1]), ep.act) * __uint_as_float(v[9 + 2 * j]));
+        *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(out) + (size_t)row * out_stride + (col >> 1)) = p;
+        return;
+    }
+    if (out_mode == OUT_GATED) {
         // columns col .. col + 7 are gates, col + 8 .. col + 15 their ups (rows_b is a multiple of 16)
         uint4 p;
         __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&p);
@@ -133,7 +152,7 @@ __device__ __forceinline__ void store_chunk(const uint32_t (&v)[16], void* out, 
 // and weight rows 256 (t / tiles_m) .., so that the pairs at work at one time share weight tiles.
 __global__ void __launch_bounds__(THREADS)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b, int rows_a,
-                 int rows_b, int K, void* __restrict__ out, int out_mode, int out_stride, int* status) {
+                 int rows_b, int K, void* __restrict__ out, int out_mode, int out_stride, const TwEpilogue ep, int* status) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint64_t* full = reinterpret_cast<uint64_t*>(tiles + STAGES * STAGE_BYTES);     // used in the pair's first block
@@ -237,7 +256,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
             for (int c0 = 0; c0 < BN; c0 += 16) {
                 uint32_t v[16];
                 tmem_ld16(tmem_base + ((uint32_t)(quarter * 32) << 16) + b * BN + c0, v);
-                if (row < rows_a && col0 + c0 < rows_b) store_chunk(v, out, out_mode, out_stride, row, col0 + c0, rows_b);
+                if (row < rows_a && col0 + c0 < rows_b) store_chunk(v, out, out_mode, out_stride, row, col0 + c0, rows_b, ep);
             }
             tc_fence_before();
             __syncwarp();
@@ -256,13 +275,14 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
 
 // out[m, n] = x[m, k] @ w[n, k].T, bf16 operands (k a multiple of 8, both 16-byte aligned), for m of
 // a few hundred rows and more.  out_mode 0: bf16 [m, out_stride]; 1: fp32 [m, out_stride]; 3: bf16
-// [m, out_stride] = silu(gate) * up with n / 2 columns, for w whose rows come in groups of eight
-// gates followed by their eight ups (n a multiple of 16).
+// [m, out_stride] = act(gate) * up with n / 2 columns, for w whose rows come in groups of eight
+// gates followed by their eight ups (n a multiple of 16).  `bias` (bf16 [n], in the order of the rows, or null) and
+// `act`: see TwEpilogue.
 TW_EXPORT int tw_gemm_tcgen05_pair(const void* x, const void* w, int m, int n, int k, void* out, int out_mode,
-                                   int out_stride, int* status, cudaStream_t stream) {
+                                   int out_stride, const void* bias, int act, int* status, cudaStream_t stream) {
     if (m <= 0 || n <= 0) return 0;
-    if (k <= 0 || (k & 7) || (out_mode != OUT_BF16 && out_mode != OUT_F32 && out_mode != OUT_SILU_MUL) ||
-        (out_mode == OUT_SILU_MUL && ((n & 15) || (out_stride & 7) || (reinterpret_cast<uintptr_t>(out) & 15))) ||
+    if (k <= 0 || (k & 7) || act < TW_ACT_NONE || act > TW_ACT_RELU_SQUARED || (out_mode != OUT_BF16 && out_mode != OUT_F32 && out_mode != OUT_GATED) ||
+        (out_mode == OUT_GATED && ((n & 15) || (out_stride & 7) || (reinterpret_cast<uintptr_t>(out) & 15))) ||
         (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
         return (int)cudaErrorInvalidValue;
     static bool attr_set = false;
@@ -285,5 +305,5 @@ TW_EXPORT int tw_gemm_tcgen05_pair(const void* x, const void* w, int m, int n, i
     const int pairs = n_tiles < sm_count / 2 ? n_tiles : sm_count / 2;
     dim3 grid(2 * pairs);
     return tw_launch(gemm_pair_kernel, grid, dim3(THREADS), (size_t)SMEM, stream, 2, ma, mb, m, n, k, out, out_mode,
-                     out_stride, status);
+                     out_stride, TwEpilogue{(const bf16*)bias, act}, status);
 }

@@ -32,7 +32,7 @@ constexpr int EPI_WARPS = 4;
 constexpr int THREADS = 64 + EPI_WARPS * 32;
 constexpr int A_BYTES = BM * BK * 2;
 
-enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_PARTIAL = 2, OUT_SILU_MUL = 3, OUT_EARLY_DEPENDENTS = 16 /* flag, or-ed in */ };
+enum : int { OUT_BF16 = 0, OUT_F32 = 1, OUT_PARTIAL = 2, OUT_GATED = 3, OUT_EARLY_DEPENDENTS = 16 /* flag, or-ed in */ };
 
 template <int BN> struct Config {
     static constexpr int B_BYTES = BN * BK * 2 < 1024 ? 1024 : BN * BK * 2;
@@ -48,7 +48,7 @@ template <int BN>
 __global__ void __launch_bounds__(THREADS)
 gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, int n_rows,
                    int m_tokens, int K, int kper, int ksplit, void* __restrict__ out, int out_mode, int out_stride,
-                   int* status, const void* next_weights, long long next_bytes) {
+                   const TwEpilogue ep, int* status, const void* next_weights, long long next_bytes) {
     using C = Config<BN>;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -152,21 +152,22 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             if (!ok) break;
             tc_fence_after();
             const int row = (item / ksplit) * BM + quarter * 32 + lane;          // weight row = output feature
+            const float row_bias = ep.bias && slice == 0 && row < n_rows ? __bfloat162float(ep.bias[row]) : 0.f;
 #pragma unroll 1
             for (int c0 = 0; c0 < BN; c0 += 16) {
                 if (c0 >= m_tokens) break;
                 uint32_t v[16];
                 tmem_ld16(tmem_base + ((uint32_t)(quarter * 32) << 16) + b * C::ACC_COLS + c0, v);
-                if (out_mode == OUT_SILU_MUL) {
+                if (out_mode == OUT_GATED) {
                     // rows 16 g .. 16 g + 7 are gates, the eight after them their ups: lane l < 8 (mod 16) takes the up from lane l + 8
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        const float up = __shfl_down_sync(0xffffffffu, __uint_as_float(v[j]), 8);
-                        const float gt = __uint_as_float(v[j]);
+                        const float gt = __uint_as_float(v[j]) + row_bias;
+                        const float up = __shfl_down_sync(0xffffffffu, gt, 8);
                         const int tok = c0 + j;
                         if ((lane & 8) == 0 && row < n_rows && tok < m_tokens)
                             reinterpret_cast<bf16*>(out)[(size_t)tok * out_stride + (row >> 4) * 8 + (lane & 7)] =
-                                __float2bfloat16_rn(gt / (1.0f + expf(-gt)) * up);
+                                __float2bfloat16_rn(tw_activate(gt, ep.act) * up);
                     }
                     continue;
                 }
@@ -175,7 +176,8 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                 for (int j = 0; j < 16; ++j) {
                     const int tok = c0 + j;
                     if (tok >= m_tokens) break;
-                    const float f = __uint_as_float(v[j]);
+                    float f = __uint_as_float(v[j]) + row_bias;
+                    if (out_mode != OUT_PARTIAL) f = tw_activate(f, ep.act);
                     if (out_mode == OUT_BF16)
                         reinterpret_cast<bf16*>(out)[(size_t)tok * out_stride + row] = __float2bfloat16_rn(f);
                     else if (out_mode == OUT_F32)
@@ -197,7 +199,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
 
 template <int BN>
 int launch(const void* w, int n, const void* x, int m, int K, int kper, int ksplit, void* out, int out_mode, int out_stride,
-           int* status, int blocks, const void* next_weights, long long next_bytes, cudaStream_t stream) {
+           const TwEpilogue& ep, int* status, int blocks, const void* next_weights, long long next_bytes, cudaStream_t stream) {
     using C = Config<BN>;
     static bool attr_set = false;
     if (!attr_set) {
@@ -209,28 +211,31 @@ int launch(const void* w, int n, const void* x, int m, int K, int kper, int kspl
     if (int e = get_map(w, n, K, BM, &mw)) return e;
     if (int e = get_map(x, m, K, BN, &mx)) return e;
     return tw_launch(gemm_stream_kernel<BN>, dim3(blocks), dim3(THREADS), (size_t)C::SMEM, stream, 1, mw, mx, n, m, K, kper, ksplit,
-                     out, out_mode, out_stride, status, next_weights, next_bytes);
+                     out, out_mode, out_stride, ep, status, next_weights, next_bytes);
 }
 
 }  // namespace
 
 // out[m, n] = x[m, k] @ w[n, k].T for m <= 128 rows, bf16 operands (k a multiple of 8, both 16-byte aligned).
 // kper (a multiple of 64) < k splits k into slices; out is then fp32 [slices, m, n] (out_mode 2).
-// out_mode 0: bf16 [m, out_stride]; 1: fp32 [m, out_stride]; 3: bf16 [m, out_stride] = silu(gate) * up with n / 2
+// out_mode 0: bf16 [m, out_stride]; 1: fp32 [m, out_stride]; 3: bf16 [m, out_stride] = act(gate) * up with n / 2
 // columns, for w whose rows come in groups of eight gates followed by their eight ups (n a multiple of 16, no slices).
+// `bias` (bf16 [n], in the order of the rows, or null) and `act`: see TwEpilogue.
 TW_EXPORT int tw_gemm_tcgen05_stream(const void* x, const void* w, int m, int n, int k, int kper, void* out, int out_mode,
-                                     int out_stride, int* status, const void* next_weights, long long next_bytes,
+                                     int out_stride, const void* bias, int act, int* status, const void* next_weights,
+                                     long long next_bytes,
                                      cudaStream_t stream) {
     if (m <= 0 || n <= 0) return 0;
     if ((uintptr_t)next_weights & 15) return (int)cudaErrorMisalignedAddress;
     if (!next_weights || next_bytes < 0) next_bytes = 0;
     const int mode = out_mode & ~OUT_EARLY_DEPENDENTS;
     if (m > 128 || k <= 0 || (k & 7) || kper <= 0 || (kper & 63) || mode < 0 || mode > 3 ||
+        act < TW_ACT_NONE || act > TW_ACT_RELU_SQUARED || (act != TW_ACT_NONE && mode == OUT_PARTIAL) ||
         (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
         return (int)cudaErrorInvalidValue;
     const int ksplit = (k + kper - 1) / kper;
     if (ksplit > 1 && mode != OUT_PARTIAL) return (int)cudaErrorInvalidValue;
-    if (mode == OUT_SILU_MUL && (n & 15)) return (int)cudaErrorInvalidValue;
+    if (mode == OUT_GATED && (n & 15)) return (int)cudaErrorInvalidValue;
     static int sm_count = 0;
     if (!sm_count) {
         int dev = 0;
@@ -239,10 +244,11 @@ TW_EXPORT int tw_gemm_tcgen05_stream(const void* x, const void* w, int m, int n,
     }
     const long long items = (long long)((n + BM - 1) / BM) * ksplit;
     const int blocks = (int)(items < sm_count ? items : sm_count);
-    if (m <= 16) return launch<16>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, status, blocks, next_weights, next_bytes, stream);
-    if (m <= 32) return launch<32>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, status, blocks, next_weights, next_bytes, stream);
-    if (m <= 64) return launch<64>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, status, blocks, next_weights, next_bytes, stream);
-    return launch<128>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, status, blocks, next_weights, next_bytes, stream);
+    const TwEpilogue ep{(const bf16*)bias, act};
+    if (m <= 16) return launch<16>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, ep, status, blocks, next_weights, next_bytes, stream);
+    if (m <= 32) return launch<32>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, ep, status, blocks, next_weights, next_bytes, stream);
+    if (m <= 64) return launch<64>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, ep, status, blocks, next_weights, next_bytes, stream);
+    return launch<128>(w, n, x, m, k, kper, ksplit, out, out_mode, out_stride, ep, status, blocks, next_weights, next_bytes, stream);
 }
 
 TW_EXPORT int tw_gemm_tcgen05_stream_sm_count() {

@@ -9,6 +9,7 @@
 //                    (not renormalised)
 //   tw_moe_gate_up   act[token, j] = silu(Wg_e h) * (Wu_e h)          e = the j-th expert of the token
 //                    with `act` 1: g = min(Wg_e h, limit), u = clamp(Wu_e h, -limit, limit), g sigmoid(alpha g) (u + 1)
+//   tw_moe_up        act[token, j] = f(Wu_e h) for experts without a gate, f one of the activations of common.cuh
 //   tw_moe_down      out[token] = sum_j weight_j Wd_e act[token, j]  (+ gate * shared[token])
 //
 // The router may have more outputs than there are experts with matrices: outputs E .. E + identity - 1 are identity
@@ -231,6 +232,50 @@ TW_EXPORT int tw_moe_gate_up(void* act, const void* h, int h_stride, const void*
                          h_stride, (const float*)wgu, chosen, width, F, E, top, per, glu, limit, alpha);
     return tw_launch(moe_gate_up_kernel<__nv_bfloat16>, grid, dim3(32 * TW_MOE_WARPS), smem, stream, 1, (__nv_bfloat16*)act,
                      (const __nv_bfloat16*)h, h_stride, (const __nv_bfloat16*)wgu, chosen, width, F, E, top, per, glu, limit, alpha);
+}
+
+// Experts of one matrix before the activation: a warp streams two of its rows side by side.
+template <typename T>
+__global__ void __launch_bounds__(32 * TW_MOE_WARPS)
+moe_up_kernel(T* __restrict__ act, const T* __restrict__ h, int h_stride, const T* __restrict__ wu, const int* __restrict__ chosen,
+              int width, int F, int E, int top, int rows_per_block, int activation) {
+    extern __shared__ float sm[];           // [width]
+    tw_grid_wait();
+    tw_grid_launch_dependents();
+    const int pair = blockIdx.x, row = pair / top;
+    const int e = chosen[pair];
+    if (e < 0 || e >= E) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) sm[c] = tw_to_float(h[(size_t)row * h_stride + c]);
+    __syncthreads();
+    const bool vec = (width & 7) == 0;
+    const T* w = wu + (size_t)e * F * width;
+    const int f0 = blockIdx.y * rows_per_block, f1 = min(F, f0 + rows_per_block);
+    for (int f = f0 + 2 * warp; f < f1; f += 2 * TW_MOE_WARPS) {
+        const int g = f + 1 < f1 ? f + 1 : f;
+        float a, b;
+        tw_dot2<T>(w + (size_t)f * width, w + (size_t)g * width, sm, sm, width, lane, vec, a, b);
+        if (lane == 0) {
+            act[(size_t)pair * F + f] = tw_from_float<T>(tw_activate(a, activation));
+            if (g != f) act[(size_t)pair * F + g] = tw_from_float<T>(tw_activate(b, activation));
+        }
+    }
+}
+
+TW_EXPORT int tw_moe_up(void* act, const void* h, int h_stride, const void* wu, const int* chosen, int rows, int width, int F,
+                        int E, int top, int activation, int dtype, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    const size_t smem = (size_t)width * sizeof(float);
+    if (smem > 48 * 1024 || activation < TW_ACT_NONE || activation > TW_ACT_RELU_SQUARED) return (int)cudaErrorInvalidValue;
+    int per = F;
+    while (per > 2 * TW_MOE_WARPS && (size_t)rows * top * ((F + per - 1) / per) < 592) per = (per + 1) / 2;
+    per = ((per + 2 * TW_MOE_WARPS - 1) / (2 * TW_MOE_WARPS)) * (2 * TW_MOE_WARPS);
+    const dim3 grid(rows * top, (F + per - 1) / per);
+    if (dtype == TW_F32)
+        return tw_launch(moe_up_kernel<float>, grid, dim3(32 * TW_MOE_WARPS), smem, stream, 1, (float*)act, (const float*)h, h_stride,
+                         (const float*)wu, chosen, width, F, E, top, per, activation);
+    return tw_launch(moe_up_kernel<__nv_bfloat16>, grid, dim3(32 * TW_MOE_WARPS), smem, stream, 1, (__nv_bfloat16*)act,
+                     (const __nv_bfloat16*)h, h_stride, (const __nv_bfloat16*)wu, chosen, width, F, E, top, per, activation);
 }
 
 template <typename T>

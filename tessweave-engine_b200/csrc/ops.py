@@ -559,11 +559,24 @@ def softcap(logits: torch.Tensor, cap: float) -> None:
     _check(code, "softcap")
 
 
-def silu_mul(out: torch.Tensor, gate_up, n_rows: int, interleaved: bool = False) -> None:
-    """out[n, i] = silu(gate[n, i]) * up[n, i].  Columns of ``gate_up`` are [all gates | all ups],
+# what stands between two products of a feed-forward (csrc/common.cuh: tw_activate)
+ACT_NONE, ACT_SILU, ACT_GELU_TANH, ACT_RELU_SQUARED = 0, 1, 2, 3
+ACTIVATIONS = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "relu_squared": ACT_RELU_SQUARED}
+
+
+def _bias_check(bias: torch.Tensor | None, n: int, dtype: torch.dtype, what: str) -> None:
+    _need(bias is None or (bias.is_cuda and bias.dtype == dtype and bias.dim() == 1 and bias.numel() == n and bias.is_contiguous()),
+          f"{what}: the bias must be one contiguous value of the activations' type per output")
+
+
+def silu_mul(out: torch.Tensor, gate_up, n_rows: int, interleaved: bool = False, act: int = ACT_SILU,
+             bias: torch.Tensor | None = None) -> None:
+    """out[n, i] = act(gate[n, i]) * up[n, i].  Columns of ``gate_up`` are [all gates | all ups],
     or with ``interleaved`` groups of 16: eight gates followed by their eight ups.  ``gate_up`` may be a
-    ``SplitSum`` (fp32 slices of the product, added here in slice order); ``out`` is then bfloat16."""
+    ``SplitSum`` (fp32 slices of the product, added here in slice order); ``out`` is then bfloat16.  ``bias``
+    (in the order of the columns, of the output's type) is added to gates and ups first."""
     inter = out.shape[1]
+    _bias_check(bias, 2 * inter, out.dtype, "silu_mul")
     if isinstance(gate_up, SplitSum):
         slices = gate_up.slices
         _cuda(out, slices)
@@ -572,7 +585,8 @@ def silu_mul(out: torch.Tensor, gate_up, n_rows: int, interleaved: bool = False)
               and inter % 4 == 0 and (not interleaved or inter % 8 == 0) and out.shape[0] >= n_rows,
               "silu_mul: slices must be fp32 [slices, rows, 2I], the output bf16 [rows, I], I a multiple of 4 (8 interleaved)")
         code = _fn("elementwise", "tw_silu_mul_slices")(_ptr(out), _ptr(slices), c_int(slices.shape[0]), c_long(slices.stride(0)),
-                                                        c_int(n_rows), c_int(inter), c_int(1 if interleaved else 0), _stream())
+                                                        c_int(n_rows), c_int(inter), c_int(1 if interleaved else 0), c_int(act), _ptr(bias),
+                                                        _stream())
         _check(code, "silu_mul_slices")
         return
     _cuda(out, gate_up)
@@ -580,21 +594,34 @@ def silu_mul(out: torch.Tensor, gate_up, n_rows: int, interleaved: bool = False)
           and gate_up.dtype == out.dtype, "silu_mul: gate_up must be contiguous [n, 2I] of the output type")
     _need(not interleaved or inter % 8 == 0, "silu_mul: interleaved columns need a multiple of 8")
     code = _fn("elementwise", "tw_silu_mul")(_ptr(out), _ptr(gate_up), c_int(n_rows), c_int(inter),
-                                             c_int(1 if interleaved else 0), c_int(dtype_code(out.dtype)), _stream())
+                                             c_int(1 if interleaved else 0), c_int(act), _ptr(bias), c_int(dtype_code(out.dtype)),
+                                             _stream())
     _check(code, "silu_mul")
+
+
+def activate_rows(x: torch.Tensor, n_rows: int, act: int, bias: torch.Tensor | None = None) -> None:
+    """x[:n_rows] <- act(x[:n_rows] + bias) in place, fp32 arithmetic: a feed-forward without a gate."""
+    _cuda(x, bias)
+    _need(x.dim() == 2 and x.is_contiguous() and x.shape[0] >= n_rows, "activate_rows: contiguous rows")
+    _bias_check(bias, x.shape[1], x.dtype, "activate_rows")
+    code = _fn("elementwise", "tw_activate_rows")(_ptr(x), _ptr(bias), c_int(n_rows), c_int(x.shape[1]), c_int(act),
+                                                  c_int(dtype_code(x.dtype)), _stream())
+    _check(code, "activate_rows")
 
 
 def attention_generic(out: torch.Tensor, q: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
                       seq_slot: torch.Tensor, block_table: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
                       n_tokens: int, n_q_heads: int, n_kv_heads: int, head_dim: int, window: int, scale: float,
                       status: torch.Tensor, sink: torch.Tensor | None = None,
-                      bias_by_distance: torch.Tensor | None = None) -> None:
+                      bias_by_distance: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
     """Exact paged causal attention, one block per (token, head).  q may be a column
     slice of the packed qkv buffer (row stride is passed on).  The value pages may have rows of another
     length than the key pages (or be the key pages themselves); the output then has heads of that length.
     ``sink`` fp32 [Hq]: exp(sink[h]) joins the softmax's denominator.  ``bias_by_distance`` fp32 [rows, Hq]: row
-    min(position - key position, rows - 1) is added to the scaled score."""
-    _cuda(out, q, positions, seq_of_token, seq_slot, block_table, k_pages, v_pages, status, sink, bias_by_distance)
+    min(position - key position, rows - 1) is added to the scaled score.  ``window``: how far a query sees, as
+    ``visible_reach`` makes it.  ``gate`` fp32 [rows, Hq]: each head's output is multiplied by its entry."""
+    _cuda(out, q, positions, seq_of_token, seq_slot, block_table, k_pages, v_pages, status, sink, bias_by_distance, gate)
+    _gate_check(gate, n_tokens, n_q_heads)
     _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == n_q_heads and sink.is_contiguous()),
           "attention: the sink must be fp32 [Hq]")
     _need(bias_by_distance is None or (bias_by_distance.dtype == torch.float32 and bias_by_distance.dim() == 2
@@ -611,9 +638,71 @@ def attention_generic(out: torch.Tensor, q: torch.Tensor, positions: torch.Tenso
         _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages), c_int(n_tokens),
         c_int(n_q_heads), c_int(n_kv_heads), c_int(head_dim), c_int(v_pages.shape[3]), c_int(k_pages.shape[2]),
         c_int(k_pages.shape[0]), c_int(window), c_float(scale), _ptr(bias_by_distance),
-        c_int(0 if bias_by_distance is None else bias_by_distance.shape[0]), _ptr(sink), c_int(dtype_code(q.dtype)),
+        c_int(0 if bias_by_distance is None else bias_by_distance.shape[0]), _ptr(sink), _ptr(gate), c_int(dtype_code(q.dtype)),
         _ptr(status), _stream())
     _check(code, "attention_generic")
+
+
+def visible_reach(window: int | None, chunk: int | None) -> int:
+    """How far an attention kernel's queries see, as its ``window`` argument says it (csrc/common.cuh: tw_first_key):
+    a sliding window is positive, chunks of positions counted from 0 are negative, 0 is everything."""
+    if window and chunk:
+        raise ValueError("attention sees a sliding window or its own chunk, not both")
+    return int(window) if window else -int(chunk) if chunk else 0
+
+
+def _gate_check(gate: torch.Tensor | None, n_rows: int, n_q_heads: int) -> None:
+    _need(gate is None or (gate.dtype == torch.float32 and gate.dim() == 2 and gate.shape[1] == n_q_heads and gate.shape[0] >= n_rows
+                           and gate.is_contiguous()), "attention: the output gate must be fp32 [rows, Hq]")
+
+
+def attention_prepare(q_out: torch.Tensor, rows, n_tokens: int, n_q_heads: int, n_kv_heads: int, head_dim: int, v_dim: int,
+                      positions: torch.Tensor, seq_of_token: torch.Tensor, seq_slot: torch.Tensor, block_table: torch.Tensor,
+                      k_pages: torch.Tensor, v_pages: torch.Tensor, write_cache: bool, status: torch.Tensor, rot_dims: int = 0,
+                      inv_freq: torch.Tensor | None = None, interleaved: bool = False, magnitude: float = 1.0,
+                      gate: torch.Tensor | None = None, leave_values: torch.Tensor | None = None,
+                      mix_values: torch.Tensor | None = None, mix_weight: torch.Tensor | None = None) -> None:
+    """One pass over every token's projected row ``[q heads | k heads | v heads | one number per q head, with gate]``
+    (a tensor of the pages' type, or a ``SplitSum``): rotate the first ``rot_dims`` values of every q and k head by
+    position, write q to ``q_out`` [rows, Hq D], k and v to the token's place in the pages, and the sigmoid of the last
+    columns to ``gate`` (fp32 [rows, Hq]).  ``leave_values`` [rows, Hkv Dv] also receives the values; ``mix_values``
+    (what another layer left that way) is blended in before they are stored: (1 - w) v + w mix, w = ``mix_weight`` (an
+    fp32 tensor of one number)."""
+    _cuda(q_out, positions, seq_of_token, seq_slot, block_table, k_pages, v_pages, status, inv_freq, gate, leave_values, mix_values, mix_weight)
+    need = n_q_heads * head_dim + n_kv_heads * (head_dim + v_dim) + (n_q_heads if gate is not None else 0)
+    partial, nsplit, split_stride, stride = None, 0, 0, 0
+    if isinstance(rows, SplitSum):
+        partial, rows = rows.slices, None
+        nsplit, split_stride, width = partial.shape[0], partial.stride(0), partial.shape[2]
+        _need(partial.is_cuda and partial.dtype == torch.float32 and partial[0].is_contiguous() and partial.shape[1] >= n_tokens,
+              "attention_prepare: bad split source")
+    else:
+        _cuda(rows)
+        width, stride = rows.shape[1], rows.stride(0)
+        _need(rows.dtype == k_pages.dtype and rows.stride(1) == 1 and rows.shape[0] >= n_tokens, "attention_prepare: bad rows")
+    _need(width >= need, f"attention_prepare: a row has {width} columns, {need} are needed")
+    _need(q_out.dtype == k_pages.dtype == v_pages.dtype and q_out.is_contiguous() and q_out.shape[0] >= n_tokens
+          and q_out.shape[1] == n_q_heads * head_dim, "attention_prepare: q must be contiguous [rows, Hq D] of the pages' type")
+    _need(k_pages.is_contiguous() and v_pages.is_contiguous() and tuple(k_pages.shape[1:]) == (n_kv_heads, k_pages.shape[2], head_dim)
+          and tuple(v_pages.shape) == (*k_pages.shape[:3], v_dim), "attention_prepare: pages must be contiguous [pages, kv_heads, page, head size]")
+    _need(block_table.dtype == torch.int32 and block_table.is_contiguous(), "attention_prepare: bad block table")
+    _need(rot_dims % 2 == 0 and 0 <= rot_dims <= head_dim and (rot_dims == 0 or (
+        inv_freq is not None and inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dims // 2)), "attention_prepare: one fp32 rate per pair")
+    _gate_check(gate, n_tokens, n_q_heads)
+    _need(leave_values is None or mix_values is None, "attention_prepare: values are left or mixed, not both")
+    first = leave_values if leave_values is not None else mix_values
+    _need(first is None or (first.dtype == q_out.dtype and first.is_contiguous() and first.shape[0] >= n_tokens
+                            and first.shape[1] == n_kv_heads * v_dim), "attention_prepare: the kept values must be contiguous [rows, Hkv Dv]")
+    _need(mix_values is None or (mix_weight is not None and mix_weight.dtype == torch.float32 and mix_weight.numel() == 1),
+          "attention_prepare: mixing needs an fp32 weight")
+    role = 1 if leave_values is not None else 2 if mix_values is not None else 0
+    code = _fn("attention_prepare", "tw_attention_prepare")(
+        _ptr(q_out), _ptr(rows), c_int(stride), _ptr(partial), c_int(nsplit), c_long(split_stride), c_int(width), c_int(n_tokens),
+        c_int(n_q_heads), c_int(n_kv_heads), c_int(head_dim), c_int(v_dim), c_int(rot_dims), c_int(1 if interleaved else 0),
+        c_float(magnitude), _ptr(inv_freq), c_int(role), _ptr(mix_weight), _ptr(first), _ptr(gate), _ptr(positions), _ptr(seq_of_token),
+        _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages), c_int(k_pages.shape[2]),
+        c_int(k_pages.shape[0]), c_int(1 if write_cache else 0), c_int(dtype_code(q_out.dtype)), _ptr(status), _stream())
+    _check(code, "attention_prepare")
 
 
 def sample(out: torch.Tensor, logits: torch.Tensor, n_rows: int, temperature: torch.Tensor | None = None,
@@ -638,26 +727,32 @@ DECODE_SCRATCH_UNITS = 1024      # most (request, split) pairs whose partial res
 _SM_COUNT = 148
 
 
-def tensor_core_attention_supported(dtype: torch.dtype, head_dim: int) -> bool:
-    return dtype == torch.bfloat16 and head_dim % 16 == 0 and 16 <= head_dim <= 256
+def tensor_core_attention_supported(dtype: torch.dtype, head_dim: int, v_dim: int | None = None) -> bool:
+    """``v_dim``: the size of a value where it differs from ``head_dim``."""
+    return dtype == torch.bfloat16 and all(d % 16 == 0 and 16 <= d <= 256 for d in (head_dim, v_dim or head_dim))
 
 
-def tcgen05_attention_supported(dtype: torch.dtype, head_dim: int, page_size: int) -> bool:
+def head_size_defines(head_dim: int, v_dim: int) -> dict[str, int]:
+    """The compile-time sizes an attention library is built for."""
+    return {"TW_HEAD_DIM": head_dim} if v_dim == head_dim else {"TW_HEAD_DIM": head_dim, "TW_V_DIM": v_dim}
+
+
+def tcgen05_attention_supported(dtype: torch.dtype, head_dim: int, page_size: int, v_dim: int | None = None) -> bool:
     """The tcgen05 prefill attention takes bfloat16, head sizes 64 and 128, and pages of at least
     8 keys that divide a tile of 128 keys or are a multiple of it."""
-    return (dtype == torch.bfloat16 and head_dim in (64, 128) and page_size >= 8
+    return (dtype == torch.bfloat16 and head_dim in (64, 128) and (v_dim or head_dim) in (64, 128) and page_size >= 8
             and (128 % page_size == 0 or page_size % 128 == 0))
 
 
 TCGEN05_ATTENTION_MIN_TOKENS = 128
 
 
-def prefer_tcgen05_attention(dtype: torch.dtype, head_dim: int, page_size: int, max_q_len: int) -> bool:
+def prefer_tcgen05_attention(dtype: torch.dtype, head_dim: int, page_size: int, max_q_len: int, v_dim: int | None = None) -> bool:
     """Whether a step whose longest portion has ``max_q_len`` tokens runs its prompt attention on
     the tcgen05 kernel.  TESSWEAVE_PREFILL_ATTENTION=mma|tcgen05 forces one of the two (the latter
     only for shapes the kernel takes)."""
     import os
-    if not tcgen05_attention_supported(dtype, head_dim, page_size):
+    if not tcgen05_attention_supported(dtype, head_dim, page_size, v_dim):
         return False
     forced = os.environ.get("TESSWEAVE_PREFILL_ATTENTION")
     if forced == "mma":
@@ -715,14 +810,15 @@ def decode_counter_ints(n_seqs: int, n_kv_heads: int, group: int) -> int:
 
 
 def _attn_common_checks(out, q, block_table, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim):
-    _need(tensor_core_attention_supported(q.dtype, head_dim),
-          f"tensor-core attention takes bfloat16 and head sizes that are multiples of 16 up to 256, not {q.dtype}/{head_dim}")
+    _need(tensor_core_attention_supported(q.dtype, head_dim, v_pages.shape[3]),
+          f"tensor-core attention takes bfloat16 and head sizes that are multiples of 16 up to 256, not {q.dtype}/{head_dim}/{v_pages.shape[3]}")
     _need(n_q_heads % n_kv_heads == 0, "attention: query heads must be a multiple of key/value heads")
     _need(q.stride(1) == 1 and out.stride(1) == 1 and out.dtype == q.dtype == k_pages.dtype == v_pages.dtype,
           "attention: operands must be bfloat16 with unit inner stride")
     _need(q.stride(0) % 2 == 0 and q.storage_offset() % 2 == 0 and out.stride(0) % 2 == 0, "attention: rows must be 4-byte aligned")
     _need(k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape[3] == head_dim
-          and k_pages.shape[1] == n_kv_heads, "attention: cache pages must be contiguous [pages, kv_heads, page, head_dim]")
+          and k_pages.shape[1] == n_kv_heads and k_pages.shape[:3] == v_pages.shape[:3],
+          "attention: cache pages must be contiguous [pages, kv_heads, page, head_dim]")
     _need(block_table.dtype == torch.int32 and block_table.is_contiguous(), "attention: bad block table")
 
 
@@ -737,15 +833,19 @@ def _score_terms_checks(sink, bias_rows, n_q_heads):
 def attention_decode(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, n_seqs,
                      n_q_heads, n_kv_heads, head_dim, window, scale, nsplit, scratch, counters, status,
                      merge_in_scratch: bool = False, sink: torch.Tensor | None = None,
-                     bias_rows: torch.Tensor | None = None) -> None:
+                     bias_rows: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> None:
     """Split-KV attention for the requests of the batch that bring one token (others are skipped).
     Up to 16 slices merge inside a thread-block cluster; more (or all, with ``merge_in_scratch``)
     merge through ``scratch`` (fp32, the slices' partial results) and ``counters`` (int32, all
     zero, left zero), which find the block that finishes last.  ``sink`` fp32 [Hq]: exp(sink[h]) joins the
     denominator of head h.  ``bias_rows`` fp32 [Hq, distances]: entry min(position - key position, distances - 1)
-    of head h is added to its scaled score.  ``v_pages`` may be ``k_pages`` (values that are the keys)."""
+    of head h is added to its scaled score.  ``v_pages`` may be ``k_pages`` (values that are the keys).
+    ``window``: how far a query sees, as ``visible_reach`` makes it.  ``gate`` fp32 [rows, Hq]: each head's output of a
+    row is multiplied by its entry.  The value pages may have rows of another length; the output has heads of that length."""
     _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, scratch, counters, status,
-          sink, bias_rows)
+          sink, bias_rows, gate)
+    _gate_check(gate, 0, n_q_heads)
+    v_dim = v_pages.shape[3]
     _attn_common_checks(out, q, block_table, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim)
     _score_terms_checks(sink, bias_rows, n_q_heads)
     _need(out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0, "attention_decode: output rows must be 8-byte aligned")
@@ -753,7 +853,7 @@ def attention_decode(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block
     _need(1 <= nsplit <= DECODE_MAX_SPLITS, f"attention_decode: 1 to {DECODE_MAX_SPLITS} slices, not {nsplit}")
     if nsplit > 1:
         _need(scratch is not None and scratch.dtype == torch.float32 and scratch.data_ptr() % 16 == 0
-              and scratch.numel() >= n_seqs * n_q_heads * nsplit * (head_dim + 2), "attention_decode: scratch too small")
+              and scratch.numel() >= n_seqs * n_q_heads * nsplit * (v_dim + 2), "attention_decode: scratch too small")
         _need(counters is not None and counters.dtype == torch.int32
               and counters.numel() >= n_seqs * n_kv_heads * ((n_q_heads // n_kv_heads + 7) // 8),
               "attention_decode: too few counters")
@@ -761,11 +861,12 @@ def attention_decode(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block
             _ptr(seq_kv_len), _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages),
             c_int(n_seqs), c_int(n_q_heads), c_int(n_kv_heads), c_int(k_pages.shape[2]), c_int(k_pages.shape[0]),
             c_int(window), c_float(scale), c_int(nsplit), c_int(1 if merge_in_scratch else 0), _ptr(scratch), _ptr(counters))
-    if sink is None and bias_rows is None:
-        code = _fn("attention_bf16", "tw_attn_decode", {"TW_HEAD_DIM": head_dim})(*head, _ptr(status), _stream())
+    defines = head_size_defines(head_dim, v_dim)
+    if sink is None and bias_rows is None and gate is None:
+        code = _fn("attention_bf16", "tw_attn_decode", defines)(*head, _ptr(status), _stream())
     else:
-        code = _fn("attention_bf16", "tw_attn_decode_terms", {"TW_HEAD_DIM": head_dim})(
-            *head, _ptr(bias_rows), c_int(0 if bias_rows is None else bias_rows.shape[1]), _ptr(sink), _ptr(status), _stream())
+        code = _fn("attention_bf16", "tw_attn_decode_terms", defines)(
+            *head, _ptr(bias_rows), c_int(0 if bias_rows is None else bias_rows.shape[1]), _ptr(sink), _ptr(gate), _ptr(status), _stream())
     _check(code, "attention_decode")
 
 
@@ -893,14 +994,14 @@ def attention_decode_fused(out, source, bias, inv_freq, write_cache, seq_q_start
 # ---------------------------------------------------------------------------
 # decode attention fed by TMA (head sizes that are multiples of 64)
 # ---------------------------------------------------------------------------
-def decode_tma_supported(dtype: torch.dtype, head_dim: int, page_size: int) -> bool:
+def decode_tma_supported(dtype: torch.dtype, head_dim: int, page_size: int, v_dim: int | None = None) -> bool:
     """Whether single-token requests attend through ``attention_decode_tma``: bfloat16, a head size of 64, 128,
     192 or 256, and pages that are a whole fraction (at least 4 keys) or a whole multiple of a 64-key tile.
     TESSWEAVE_DECODE_TMA=0 keeps the kernel that loads keys through registers."""
     import os
     if os.environ.get("TESSWEAVE_DECODE_TMA", "1") == "0":
         return False
-    return (dtype == torch.bfloat16 and head_dim % 64 == 0 and 64 <= head_dim <= 256 and page_size >= 4
+    return (dtype == torch.bfloat16 and all(d % 64 == 0 and 64 <= d <= 256 for d in (head_dim, v_dim or head_dim)) and page_size >= 4
             and (64 % page_size == 0 or page_size % 64 == 0))
 
 
@@ -957,12 +1058,13 @@ def decode_attention_resident_early(blocks: int, nsplit: int) -> bool:
 def attention_decode_tma(out, q, source, bias, inv_freq, write_cache, seq_q_start, seq_q_len, seq_kv_len, seq_slot,
                          block_table, k_pages, v_pages, n_seqs, n_q_heads, n_kv_heads, head_dim, window, scale, nsplit,
                          scratch, counters, status, merge_in_scratch: bool = False, prefetch: torch.Tensor | None = None,
-                         stages: int = 0) -> None:
+                         stages: int = 0, gate: torch.Tensor | None = None) -> None:
     """Split-KV attention for the requests of the batch that bring one token, keys and values brought in by TMA.
     Either ``q`` (bf16 [rows, Hq D], 16-byte aligned rows) or ``source`` -- the step's untouched q/k/v product, a
     ``SplitSum`` or a bf16 [rows, (Hq + 2 Hkv) D] tensor, which the kernel biases, rotates and (``write_cache``)
     stores itself -- is given.  The other arguments are those of ``attention_decode`` / ``attention_decode_fused``;
-    ``stages`` is the depth of a block's ring of 64-key tiles (0: chosen from the size of the launch)."""
+    ``stages`` is the depth of a block's ring of 64-key tiles (0: chosen from the size of the launch).  ``window`` and
+    ``gate``: as for ``attention_decode``; with ``q`` the values may have another size than the keys."""
     import os
     width = (n_q_heads + 2 * n_kv_heads) * head_dim
     partial = dense = None
@@ -981,13 +1083,15 @@ def attention_decode_tma(out, q, source, bias, inv_freq, write_cache, seq_q_star
         _need(q is not None and q.is_cuda and q.dtype == torch.bfloat16 and q.stride(1) == 1 and q.data_ptr() % 16 == 0
               and q.stride(0) % 8 == 0, "attention_decode_tma: q must be bf16 with 16-byte aligned rows")
     _cuda(out, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, scratch, counters, status,
-          bias, inv_freq, prefetch)
-    _need(decode_tma_supported(out.dtype, head_dim, k_pages.shape[2]) or os.environ.get("TESSWEAVE_DECODE_TMA") == "0",
+          bias, inv_freq, prefetch, gate)
+    _gate_check(gate, 0, n_q_heads)
+    v_dim = v_pages.shape[3]
+    _need(decode_tma_supported(out.dtype, head_dim, k_pages.shape[2], v_dim) or os.environ.get("TESSWEAVE_DECODE_TMA") == "0",
           f"attention_decode_tma does not take head size {head_dim} with pages of {k_pages.shape[2]} keys in {out.dtype}")
     _need(out.dtype == k_pages.dtype == v_pages.dtype == torch.bfloat16, "attention_decode_tma: bfloat16 only")
     _need(n_q_heads % n_kv_heads == 0, "attention: query heads must be a multiple of key/value heads")
     _need(k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.shape[3] == head_dim
-          and k_pages.shape[1] == n_kv_heads and v_pages.shape == k_pages.shape
+          and k_pages.shape[1] == n_kv_heads and v_pages.shape[:3] == k_pages.shape[:3] and (source is None or v_dim == head_dim)
           and k_pages.data_ptr() % 16 == 0 and v_pages.data_ptr() % 16 == 0,
           "attention: cache pages must be contiguous, 16-byte aligned [pages, kv_heads, page, head_dim]")
     _need(block_table.dtype == torch.int32 and block_table.is_contiguous(), "attention: bad block table")
@@ -999,54 +1103,58 @@ def attention_decode_tma(out, q, source, bias, inv_freq, write_cache, seq_q_star
     _need(1 <= nsplit <= DECODE_MAX_SPLITS, f"attention_decode_tma: 1 to {DECODE_MAX_SPLITS} slices, not {nsplit}")
     if nsplit > 1:
         _need(scratch is not None and scratch.dtype == torch.float32 and scratch.data_ptr() % 16 == 0
-              and scratch.numel() >= n_seqs * n_q_heads * nsplit * (head_dim + 2), "attention_decode: scratch too small")
+              and scratch.numel() >= n_seqs * n_q_heads * nsplit * (v_dim + 2), "attention_decode: scratch too small")
         _need(counters is not None and counters.dtype == torch.int32
               and counters.numel() >= n_seqs * n_kv_heads * ((n_q_heads // n_kv_heads + 7) // 8),
               "attention_decode: too few counters")
     stages = stages or int(os.environ.get("TESSWEAVE_DECODE_STAGES", "0"))
-    code = _fn("attention_decode_tma", "tw_attn_decode_tma", {"TW_HEAD_DIM": head_dim})(
+    code = _fn("attention_decode_tma", "tw_attn_decode_tma", head_size_defines(head_dim, v_dim))(
         _ptr(out), c_int(out.stride(0)), _ptr(q), c_int(q.stride(0) if q is not None else 0), _ptr(partial), c_int(nslices),
         ctypes.c_longlong(slice_stride), _ptr(dense), c_int(dense_stride), _ptr(bias), _ptr(inv_freq),
         c_int(1 if write_cache else 0), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(seq_slot),
         _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages), c_int(n_seqs), c_int(n_q_heads),
         c_int(n_kv_heads), c_int(k_pages.shape[2]), c_int(k_pages.shape[0]), c_int(window), c_float(scale), c_int(nsplit),
         c_int(stages), c_int(1 if merge_in_scratch else 0), _ptr(scratch), _ptr(counters), _ptr(status), _ptr(prefetch),
-        ctypes.c_longlong(prefetch.numel() * prefetch.element_size() if prefetch is not None else 0), _stream())
+        ctypes.c_longlong(prefetch.numel() * prefetch.element_size() if prefetch is not None else 0), _ptr(gate), _stream())
     _check(code, "attention_decode_tma")
 
 
 def attention_prefill_tcgen05(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, n_seqs,
-                              max_q_len, n_q_heads, n_kv_heads, head_dim, window, scale, skip_single, status) -> None:
+                              max_q_len, n_q_heads, n_kv_heads, head_dim, window, scale, skip_single, status,
+                              gate: torch.Tensor | None = None) -> None:
     """The same as ``attention_prefill`` on the 5th-generation tensor cores (TMA, tcgen05.mma,
-    accumulators in tensor memory), for the shapes ``tcgen05_attention_supported`` names."""
-    _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, status)
+    accumulators in tensor memory), for the shapes ``tcgen05_attention_supported`` names and a positive scale."""
+    _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, status, gate)
+    _gate_check(gate, 0, n_q_heads)
     _attn_common_checks(out, q, block_table, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim)
-    _need(tcgen05_attention_supported(q.dtype, head_dim, k_pages.shape[2]),
+    _need(tcgen05_attention_supported(q.dtype, head_dim, k_pages.shape[2], v_pages.shape[3]),
           f"tcgen05 attention does not take head size {head_dim} with pages of {k_pages.shape[2]} keys")
     _need(q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0,
           "tcgen05 attention: rows of q and out must be 16-byte aligned")
-    code = _fn("attention_tcgen05", "tw_attn_prefill_tc5", {"TW_HEAD_DIM": head_dim})(
+    code = _fn("attention_tcgen05", "tw_attn_prefill_tc5", head_size_defines(head_dim, v_pages.shape[3]))(
         _ptr(out), c_int(out.stride(0)), _ptr(q), c_int(q.stride(0)), _ptr(seq_q_start), _ptr(seq_q_len),
         _ptr(seq_kv_len), _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages),
         c_int(n_seqs), c_int(max_q_len), c_int(n_q_heads), c_int(n_kv_heads), c_int(k_pages.shape[2]),
-        c_int(k_pages.shape[0]), c_int(window), c_float(scale), c_int(1 if skip_single else 0), _ptr(status), _stream())
+        c_int(k_pages.shape[0]), c_int(window), c_float(scale), c_int(1 if skip_single else 0), _ptr(gate), _ptr(status), _stream())
     _check(code, "attention_prefill_tcgen05")
 
 
 def attention_prefill(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, n_seqs,
                       max_q_len, n_q_heads, n_kv_heads, head_dim, window, scale, skip_single, status,
-                      sink: torch.Tensor | None = None, bias_rows: torch.Tensor | None = None) -> None:
-    """Flash attention over the paged cache for the requests that bring several tokens.  ``sink``, ``bias_rows`` and
-    ``v_pages`` that are ``k_pages``: as for ``attention_decode``."""
-    _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, status, sink, bias_rows)
+                      sink: torch.Tensor | None = None, bias_rows: torch.Tensor | None = None,
+                      gate: torch.Tensor | None = None) -> None:
+    """Flash attention over the paged cache for the requests that bring several tokens.  ``sink``, ``bias_rows``,
+    ``gate``, ``window`` and ``v_pages`` that are ``k_pages`` or have rows of another length: as for ``attention_decode``."""
+    _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, status, sink, bias_rows, gate)
+    _gate_check(gate, 0, n_q_heads)
     _attn_common_checks(out, q, block_table, k_pages, v_pages, n_q_heads, n_kv_heads, head_dim)
     _score_terms_checks(sink, bias_rows, n_q_heads)
-    code = _fn("attention_bf16", "tw_attn_prefill", {"TW_HEAD_DIM": head_dim})(
+    code = _fn("attention_bf16", "tw_attn_prefill", head_size_defines(head_dim, v_pages.shape[3]))(
         _ptr(out), c_int(out.stride(0)), _ptr(q), c_int(q.stride(0)), _ptr(seq_q_start), _ptr(seq_q_len),
         _ptr(seq_kv_len), _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages),
         c_int(n_seqs), c_int(max_q_len), c_int(n_q_heads), c_int(n_kv_heads), c_int(k_pages.shape[2]),
         c_int(k_pages.shape[0]), c_int(window), c_float(scale), c_int(1 if skip_single else 0), _ptr(bias_rows),
-        c_int(0 if bias_rows is None else bias_rows.shape[1]), _ptr(sink), _ptr(status), _stream())
+        c_int(0 if bias_rows is None else bias_rows.shape[1]), _ptr(sink), _ptr(gate), _ptr(status), _stream())
     _check(code, "attention_prefill")
 
 
@@ -1102,17 +1210,21 @@ def small_m_split(n: int, k: int, max_slices: int = 12, sms: int | None = None) 
 
 def gemm_small_m(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: int, kper: int | None = None,
                  silu_mul_pairs: bool = False, early_dependents: bool = False,
-                 prefetch: torch.Tensor | None = None) -> None:
+                 prefetch: torch.Tensor | None = None, bias: torch.Tensor | None = None, act: int | None = None) -> None:
     """out[:m] = x[:m] @ w.T for m <= 64 rows.  ``out`` is bf16 or fp32 [>=m, n]; or, when the
     product is split over k (kper < k), fp32 slices [slices, m, n]; or, with ``silu_mul_pairs``
-    (rows of w in groups of eight gates and their eight ups), bf16 [>=m, n / 2] = silu(gate) * up.
+    (rows of w in groups of eight gates and their eight ups), bf16 [>=m, n / 2] = act(gate) * up (silu by default).
+    ``bias`` (bf16 [n], in the order of the rows of w) is added first, of a split product to slice 0; without pairs an
+    ``act`` is applied to every value (not to slices).
     ``early_dependents``: the kernel launched next may become resident while this one runs (it waits for
     the result itself); worth it when that kernel is small.  ``prefetch``: a contiguous, 16-byte aligned tensor
     that the kernel after this one streams; the blocks ask for it to be brought into L2 when their own stream ends."""
-    _cuda(out, x, w)
+    _cuda(out, x, w, bias)
     if prefetch is not None:
         _need(prefetch.is_cuda and prefetch.is_contiguous(), "gemm_small_m: the tensor to prefetch must be contiguous")
     n, k = w.shape
+    _bias_check(bias, n, x.dtype, "gemm_small_m")
+    act = (ACT_SILU if silu_mul_pairs else ACT_NONE) if act is None else act
     _need(x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and x.is_contiguous()
           and x.shape[1] == k and k % 8 == 0 and m <= 64, "gemm_small_m: bf16 operands, k a multiple of 8, m <= 64")
     kper = kper or -(-k // 32) * 32
@@ -1132,7 +1244,7 @@ def gemm_small_m(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: int, kp
     if early_dependents:
         mode |= 16          # the kernel after this one may become resident while this one runs
     code = _fn("gemm_smallm", "tw_gemm_smallm")(_ptr(w), _ptr(x), c_int(m), c_int(n), c_int(k), c_int(kper), _ptr(out),
-                                                c_int(mode), c_int(stride), _ptr(prefetch),
+                                                c_int(mode), c_int(stride), _ptr(bias), c_int(act), _ptr(prefetch),
                                                 ctypes.c_longlong(prefetch.numel() * prefetch.element_size()
                                                                   if prefetch is not None else 0), _stream())
     _check(code, "gemm_small_m")
@@ -1173,12 +1285,15 @@ def pair_product_preferred(x: torch.Tensor, w: torch.Tensor, m: int) -> bool:
 
 
 def gemm_tcgen05_pair(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: int, status: torch.Tensor,
-                      silu_mul_pairs: bool = False) -> None:
+                      silu_mul_pairs: bool = False, bias: torch.Tensor | None = None, act: int | None = None) -> None:
     """out[:m] = x[:m] @ w.T for many rows, on pairs of thread blocks (tcgen05.mma.cta_group::2,
     256 x 256 tiles).  ``out`` is bf16 or fp32 [>=m, n]; with ``silu_mul_pairs`` (rows of w in
-    groups of eight gates and their eight ups) it is bf16 [>=m, n / 2] = silu(gate) * up."""
-    _cuda(out, x, w, status)
+    groups of eight gates and their eight ups) it is bf16 [>=m, n / 2] = act(gate) * up.  ``bias`` and ``act``: as for
+    ``gemm_small_m``."""
+    _cuda(out, x, w, status, bias)
     n, k = w.shape
+    _bias_check(bias, n, x.dtype, "gemm_tcgen05_pair")
+    act = (ACT_SILU if silu_mul_pairs else ACT_NONE) if act is None else act
     _need(x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.is_contiguous() and x.is_contiguous()
           and x.shape[1] == k and k % 8 == 0, "gemm_tcgen05_pair: contiguous bf16 operands, k a multiple of 8")
     _need(x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0, "gemm_tcgen05_pair: operands must be 16-byte aligned")
@@ -1192,7 +1307,8 @@ def gemm_tcgen05_pair(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: in
               and out.dtype in (torch.bfloat16, torch.float32), "gemm_tcgen05_pair: bad output")
         mode = 0 if out.dtype == torch.bfloat16 else 1
     code = _fn("gemm_tcgen05_pair", "tw_gemm_tcgen05_pair")(_ptr(x), _ptr(w), c_int(m), c_int(n), c_int(k), _ptr(out),
-                                                            c_int(mode), c_int(out.stride(0)), _ptr(status), _stream())
+                                                            c_int(mode), c_int(out.stride(0)), _ptr(bias), c_int(act), _ptr(status),
+                                                            _stream())
     _check(code, "gemm_tcgen05_pair")
 
 
@@ -1269,13 +1385,15 @@ def stream_split(n: int, k: int, allow: bool = True, sms: int | None = None) -> 
 
 def gemm_tcgen05_stream(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: int, status: torch.Tensor,
                         kper: int | None = None, silu_mul_pairs: bool = False, early_dependents: bool = False,
-                        prefetch: torch.Tensor | None = None) -> None:
+                        prefetch: torch.Tensor | None = None, bias: torch.Tensor | None = None, act: int | None = None) -> None:
     """out[:m] = x[:m] @ w.T for up to 128 rows on the 5th-generation tensor cores, the weights streamed once by a
     persistent kernel.  ``out`` is bf16 or fp32 [>=m, n]; fp32 slices [slices, m, n] when ``kper`` (a multiple of
     64) is less than k; with ``silu_mul_pairs`` (rows of w in groups of eight gates and their eight ups) bf16
-    [>=m, n / 2] = silu(gate) * up.  ``prefetch``: a contiguous, 16-byte aligned tensor that the kernel after
+    [>=m, n / 2] = act(gate) * up.  ``bias`` and ``act``: as for ``gemm_small_m``.  ``prefetch``: a contiguous, 16-byte aligned tensor that the kernel after
     this one streams; a block asks for its share of it to be brought into L2 once its own last copy is issued."""
-    _cuda(out, x, w, status)
+    _cuda(out, x, w, status, bias)
+    _bias_check(bias, w.shape[0], x.dtype, "gemm_tcgen05_stream")
+    act = (ACT_SILU if silu_mul_pairs else ACT_NONE) if act is None else act
     if prefetch is not None:
         _need(prefetch.is_cuda and prefetch.is_contiguous(), "gemm_tcgen05_stream: the tensor to prefetch must be contiguous")
     n, k = w.shape
@@ -1302,7 +1420,7 @@ def gemm_tcgen05_stream(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: 
         mode |= 16          # the kernel after this one may become resident while this one runs
     # the token rows the kernel reads: exactly m (rows beyond are filled with zeros by the copy engine)
     code = _fn("gemm_tcgen05_stream", "tw_gemm_tcgen05_stream")(_ptr(x), _ptr(w), c_int(m), c_int(n), c_int(k), c_int(kper),
-                                                                _ptr(out), c_int(mode), c_int(stride), _ptr(status),
+                                                                _ptr(out), c_int(mode), c_int(stride), _ptr(bias), c_int(act), _ptr(status),
                                                                 _ptr(prefetch), ctypes.c_longlong(
                                                                     prefetch.numel() * prefetch.element_size()
                                                                     if prefetch is not None else 0), _stream())
@@ -1536,6 +1654,20 @@ def moe_gate_up(act: torch.Tensor, h: torch.Tensor, w_gate_up: torch.Tensor, cho
                                         c_int(ff), c_int(experts), c_int(top), c_int(glu), c_float(limit), c_float(alpha),
                                         c_int(dtype_code(h.dtype)), _stream())
     _check(code, "moe_gate_up")
+
+
+def moe_up(act: torch.Tensor, h: torch.Tensor, w_up: torch.Tensor, chosen: torch.Tensor, n_rows: int, activation: int) -> None:
+    """act[row, j] = f(Wu_e h[row]) for the j-th chosen expert e of the row: experts without a gate, ``w_up`` [experts, ff,
+    width], f one of ``ACTIVATIONS``."""
+    _cuda(act, h, w_up, chosen)
+    experts, ff, width = w_up.shape
+    top = chosen.shape[1]
+    _need(w_up.is_contiguous() and h.stride(1) == 1 and h.shape[1] == width and h.dtype == w_up.dtype == act.dtype
+          and act.is_contiguous() and tuple(act.shape[1:]) == (top, ff) and act.shape[0] >= n_rows, "moe_up: bad operands")
+    _need(h.dtype == torch.float32 or (w_up.data_ptr() % 16 == 0), "moe_up: weights must be 16-byte aligned")
+    code = _fn("moe", "tw_moe_up")(_ptr(act), _ptr(h), c_int(h.stride(0)), _ptr(w_up), _ptr(chosen), c_int(n_rows), c_int(width),
+                                   c_int(ff), c_int(experts), c_int(top), c_int(activation), c_int(dtype_code(h.dtype)), _stream())
+    _check(code, "moe_up")
 
 
 def glu_rows(out: torch.Tensor, gate_up: torch.Tensor, n_rows: int, glu: int, limit: float = 0.0, alpha: float = 1.0) -> None:

@@ -6,5 +6,6 @@ from . import linurax  # noqa: F401  (registers "Linurax")
 from . import sapatar  # noqa: F401  (registers "Sapatar")
 from . import nufatar  # noqa: F401  (registers "Nufatar")
 from . import dugudra  # noqa: F401  (registers "Dugudra")
+from . import varivik  # noqa: F401  (registers "Varivik")
 
 __all__ = ["LayerSpec", "ModelSpec", "ScheduleEntry", "Model"]

@@ -15,10 +15,22 @@ class PagedSoftmaxMixer(Mixer):
     """What mixers that attend with a softmax over a paged cache share: the choice of the attention kernel for a
     step.  A subclass sets ``n_heads, n_kv_heads, head_dim, v_dim, same_dims, q_size, window, scale, sink, bias_rows,
     bias_by_distance, score_terms`` (``score_terms``: the softmax has a sink or a distance table, or the values are
-    the keys -- what only the exact and the mma.sync kernels know) and hands ``_attend`` rows whose first ``q_size``
-    columns are the queries, after it has stored the step's keys and values."""
+    the keys -- what only the exact and the mma.sync kernels know), and ``chunk`` where a token sees its own chunk of
+    positions instead of a window, and hands ``_attend`` rows whose first ``q_size`` columns are the queries, after it
+    has stored the step's keys and values."""
 
     b_qkv = None
+    chunk = None
+
+    @property
+    def reach(self) -> int:
+        """How far a query sees, as the kernels want it."""
+        return ops.visible_reach(self.window, self.chunk)
+
+    @property
+    def span(self) -> int | None:
+        """The most keys a query sees; None: all before it."""
+        return self.window if self.chunk is None else self.chunk
 
     def _prefetch_plan(self, ctx: StepContext):
         return None, None
@@ -26,50 +38,50 @@ class PagedSoftmaxMixer(Mixer):
     def _decode_launch(self, ctx: StepContext, cache: PagedView) -> tuple[bool, int, int]:
         """(fed by TMA?, slices per request, blocks) of the decode attention this step will launch."""
         group = self.n_heads // self.n_kv_heads
-        tma = not self.score_terms and ops.decode_tma_supported(self.runtime.dtype, self.head_dim, cache.page_size)
+        tma = not self.score_terms and ops.decode_tma_supported(self.runtime.dtype, self.head_dim, cache.page_size, self.v_dim)
         splits = ops.decode_tma_splits if tma else ops.decode_splits
-        # (the keys a request can see: a window bounds them, and the kernels cut those into the slices)
-        nsplit = splits(ctx.n_seqs, self.n_kv_heads, group, min(ctx.max_kv_len, self.window) if self.window else ctx.max_kv_len)
+        # (the keys a request can see: a window or a chunk bounds them, and the kernels cut those into the slices)
+        nsplit = splits(ctx.n_seqs, self.n_kv_heads, group, min(ctx.max_kv_len, self.span) if self.span else ctx.max_kv_len)
         return tma, nsplit, ctx.n_seqs * self.n_kv_heads * -(-group // 8) * nsplit
 
-    def _attend_tensor_cores(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView) -> None:
+    def _attend_tensor_cores(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView,
+                             gate: torch.Tensor | None = None) -> None:
         """bfloat16: flash attention for requests with several tokens, split-KV attention for
         requests with one; both read the same flat batch and skip the other's requests."""
-        window = self.window or 0
         singles = ctx.decode_only or ctx.fixed_shape or any(n == 1 for n in ctx.host_q_len)
         if not ctx.decode_only:
             # long portions: tcgen05 kernel (TMA, accumulators in tensor memory); short ones, and the shapes it
             # does not take, stay on the mma.sync kernel, which starts faster
             prefill = ops.attention_prefill
-            # (not with a window: that kernel copies whole key tiles, and the pages of a tile's keys before the
-            # earliest window may have been given back; the mma.sync kernel skips such keys one by one)
-            if not window and not self.score_terms and ops.prefer_tcgen05_attention(self.runtime.dtype, self.head_dim, cache.k_pages.shape[2], ctx.max_q_len):
+            if (not self.score_terms and self.scale > 0
+                    and ops.prefer_tcgen05_attention(self.runtime.dtype, self.head_dim, cache.k_pages.shape[2], ctx.max_q_len, self.v_dim)):
                 prefill = ops.attention_prefill_tcgen05
             prefill(out, q, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot,
                                   cache.block_table, cache.k_pages, cache.v_pages, ctx.n_seqs, ctx.max_q_len,
-                                  self.n_heads, self.n_kv_heads, self.head_dim, window, self.scale, singles, ctx.status,
-                                  **self._terms())
+                                  self.n_heads, self.n_kv_heads, self.head_dim, self.reach, self.scale, singles, ctx.status,
+                                  gate=gate, **self._terms())
         if singles:
-            self._decode(ctx, out, q, cache)
+            self._decode(ctx, out, q, cache, gate=gate)
 
-    def _decode(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor | None, cache: PagedView, fused=None) -> None:
+    def _decode(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor | None, cache: PagedView, fused=None,
+                gate: torch.Tensor | None = None) -> None:
         """Split-KV attention for the requests that bring one token; with ``fused`` = (product, rotation table,
         write_cache) the kernel makes q, k and v of the new token from the product itself.  Head sizes that are
         multiples of 64 take the kernel that is fed by TMA, the others the one that loads keys through registers."""
         group = self.n_heads // self.n_kv_heads
         tma, nsplit, _ = self._decode_launch(ctx, cache)
-        scratch = ctx.workspace.get("attn.decode_scratch", (ops.decode_scratch_floats(self.n_heads, self.head_dim),),
+        scratch = ctx.workspace.get("attn.decode_scratch", (ops.decode_scratch_floats(self.n_heads, self.v_dim),),
                                     torch.float32)
         counters = ctx.workspace.get(
             "attn.decode_counters", (ops.decode_counter_ints(ctx.n_seqs, self.n_kv_heads, group),), torch.int32, zero=True)
-        window = self.window or 0
+        window = self.reach
         product, table, write_cache = fused if fused is not None else (None, None, False)
         prefetch = self._prefetch_plan(ctx)[0] if fused is not None else None
         if tma:
             ops.attention_decode_tma(out, q, product, self.b_qkv if fused is not None else None, table, write_cache,
                                      ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot, cache.block_table,
                                      cache.k_pages, cache.v_pages, ctx.n_seqs, self.n_heads, self.n_kv_heads, self.head_dim,
-                                     window, self.scale, nsplit, scratch, counters, ctx.status, prefetch=prefetch)
+                                     window, self.scale, nsplit, scratch, counters, ctx.status, prefetch=prefetch, gate=gate)
         elif fused is not None:
             ops.attention_decode_fused(out, product, self.b_qkv, table, write_cache, ctx.seq_q_start, ctx.seq_q_len,
                                        ctx.seq_kv_len, ctx.seq_slot, cache.block_table, cache.k_pages, cache.v_pages,
@@ -79,20 +91,23 @@ class PagedSoftmaxMixer(Mixer):
             ops.attention_decode(out, q, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot,
                                  cache.block_table, cache.k_pages, cache.v_pages, ctx.n_seqs, self.n_heads,
                                  self.n_kv_heads, self.head_dim, window, self.scale, nsplit, scratch, counters,
-                                 ctx.status, **self._terms())
+                                 ctx.status, gate=gate, **self._terms())
 
     def _terms(self) -> dict:
         return {"sink": self.sink, "bias_rows": self.bias_rows} if self.score_terms else {}
 
-    def _attend(self, ctx: StepContext, out: torch.Tensor, qkv: torch.Tensor, cache: PagedView) -> None:
+    def _attend(self, ctx: StepContext, out: torch.Tensor, qkv: torch.Tensor, cache: PagedView,
+                gate: torch.Tensor | None = None) -> None:
+        """``gate`` (fp32 [rows, heads], or None): a number each head's output of a row is multiplied by."""
         q = qkv[:, : self.q_size]
-        if self.same_dims and ops.tensor_core_attention_supported(self.runtime.dtype, self.head_dim):
-            self._attend_tensor_cores(ctx, out, q, cache)
+        # (rows of q must start on 16-byte boundaries for these kernels' copies)
+        if ops.tensor_core_attention_supported(self.runtime.dtype, self.head_dim, self.v_dim) and q.stride(0) % 8 == 0:
+            self._attend_tensor_cores(ctx, out, q, cache, gate)
             return
         ops.attention_generic(out, q, ctx.positions, ctx.seq_of_token, ctx.seq_slot, cache.block_table,
                               cache.k_pages, cache.v_pages, ctx.n_tokens, self.n_heads, self.n_kv_heads,
-                              self.head_dim, self.window or 0, self.scale, ctx.status, sink=self.sink,
-                              bias_by_distance=self.bias_by_distance)
+                              self.head_dim, self.reach, self.scale, ctx.status, sink=self.sink,
+                              bias_by_distance=self.bias_by_distance, gate=gate)
 
 
 @register_part("mixer", "gqa_attention")
@@ -110,10 +125,10 @@ class GQAAttention(PagedSoftmaxMixer):
     flow_engine/cache.py:93-100 (slots).  Weight names are the checkpoint's (``names`` replaces them).
 
     ``v_head_dim``: the size of a value head where it differs from ``head_dim`` (the size of a query and a key
-    head); the output then has ``n_heads`` heads of that size.  Heads above 256 (up to 1024) attend with the exact
-    kernel in both run types.  Such a mixer, and one whose position encoding no
+    head); the output then has ``n_heads`` heads of that size.  Heads above 256 (up to 1024), and sizes that are no
+    multiples of 16, attend with the exact kernel in both run types.  Such a mixer, and one whose position encoding no
     kernel applies on the way, adds the bias, applies the encoding and stores keys and values as separate
-    steps, and attends with the exact kernel; everything else takes the fused and tensor-core kernels.
+    steps; everything else takes the fused kernels.
 
     ``values_are_keys``: there is no value projection; a position's value is its key as projected (and encoded), and
     the cache keeps one set of pages for both.  ``sink`` (a tensor name): a learned number per query head whose
@@ -130,6 +145,16 @@ class GQAAttention(PagedSoftmaxMixer):
     ``qk_norm`` (``q``, ``k``: tensor names; ``eps``): every head of q and of k is divided by its root mean square and
     multiplied by a weight [head_dim] that all heads share, before the position encoding (fp32; one kernel for both).
     Such a mixer takes the separate steps too.
+
+    ``chunk``: positions are counted off in chunks of that many from the request's start, and a token sees the keys of
+    its own chunk up to itself, floor(position / chunk) = floor(p / chunk), wherever a prompt was cut.
+    ``head_gate`` (a tensor name, [n_heads, hidden]): head h's output is multiplied by sigmoid(Wg h)_h.
+    ``value_mix`` (``name``: a tensor of one number; ``role``): a layer with role ``first`` leaves its values for the
+    later layers of the step, one with role ``mix`` caches (1 - w) v + w v_first instead of its own (fp32, rounded
+    once).  The number of the first such layer is loaded and not used.
+    A mixer with one of the last two takes one pass over the product's rows (``ops.attention_prepare``: slices of a
+    split product added, rotation of all or part of a head, blend, store, sigmoid of the gates) and then attends with
+    the kernels of its sizes, whose epilogues multiply by the gate.
     """
 
     NAMES = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
@@ -139,8 +164,19 @@ class GQAAttention(PagedSoftmaxMixer):
                  qkv_bias: bool, position: PartSpec, scale: float | None = None, window: int | None = None,
                  out_bias: bool = False, v_head_dim: int | None = None, names: dict[str, str] | None = None,
                  values_are_keys: bool = False, sink: str | None = None, distance_bias: dict | None = None,
-                 sink_value: float | None = None, qk_norm: dict | None = None):
+                 sink_value: float | None = None, qk_norm: dict | None = None, chunk: int | None = None,
+                 head_gate: str | None = None, value_mix: dict | None = None):
         super().__init__(runtime)
+        if chunk is not None and (chunk <= 0 or window is not None):
+            raise ValueError("attention: chunk must be positive, and goes without a window")
+        if value_mix is not None and value_mix["role"] not in ("first", "mix"):
+            raise ValueError(f"attention: the role in value_mix is 'first' or 'mix', not {value_mix['role']!r}")
+        self.chunk, self.head_gate, self.value_mix = chunk, head_gate, value_mix
+        self.prepared = head_gate is not None or value_mix is not None
+        if self.prepared and (qkv_bias or values_are_keys or sink is not None or sink_value is not None or qk_norm is not None
+                              or distance_bias is not None):
+            raise ValueError("attention: a head gate or mixed values go without biases, normalised heads, sinks, distance tables and "
+                             "values that are the keys")
         if min(hidden, n_heads, n_kv_heads, head_dim) <= 0 or n_heads % n_kv_heads:
             raise ValueError("attention: heads must be positive and n_heads a multiple of n_kv_heads")
         if (head_dim % 2 and position.kind != "none") or head_dim > 1024:
@@ -163,6 +199,8 @@ class GQAAttention(PagedSoftmaxMixer):
         self.q_size, self.kv_size = n_heads * head_dim, n_kv_heads * head_dim
         self.v_size, self.out_size = (0 if self.values_are_keys else n_kv_heads * self.v_dim), n_heads * self.v_dim
         self.qkv_width = self.q_size + self.kv_size + self.v_size
+        if self.prepared:       # one product gives the gates too; its rows end on a 16-byte boundary
+            self.qkv_width = -(-(self.qkv_width + (n_heads if head_gate is not None else 0)) // 8) * 8
         self.position = build_part("position", position, runtime)
         self.w_qkv = runtime.empty(self.qkv_width, hidden)
         self.b_qkv = runtime.empty(self.qkv_width, dtype=torch.float32) if qkv_bias else None
@@ -190,8 +228,12 @@ class GQAAttention(PagedSoftmaxMixer):
             self.bias_table = runtime.empty(rows, n_heads, dtype=torch.float32)
         # terms of the softmax that the kernels fed by TMA and the kernels that rotate on the way do not know
         self.score_terms = self.values_are_keys or self.sink is not None or self.distance_bias is not None
-        self.separate_steps = self.score_terms or self.qk_norm is not None     # no kernel that rotates on the way does these
+        self.separate_steps = self.score_terms or self.qk_norm is not None or self.prepared    # no kernel that rotates on the way does these
         self.bias_rows = None
+        if self.prepared:
+            if self.position.kind != "none" and self.position.rotary_plan(head_dim) is None:
+                raise ValueError(f"attention: position encoding {self.position.kind!r} is no rotation that one pass could apply")
+            self.mix_weight = runtime.empty(1, dtype=torch.float32) if value_mix is not None else None
 
     @staticmethod
     def distance_bucket(n: int, rows: int, far: float) -> int:
@@ -201,6 +243,9 @@ class GQAAttention(PagedSoftmaxMixer):
         return min(rows - 1, half + int(math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
 
     def finalize(self) -> None:
+        if self.prepared:
+            used = self.q_size + self.kv_size + self.v_size + (self.n_heads if self.head_gate is not None else 0)
+            self.w_qkv[used:].zero_()           # padding rows, whose columns nobody reads
         if self.distance_bias is not None:
             # every distance a query can see, row by row; distances from the last row on share its bucket (the last)
             rows, far = self.distance_bias["rows"], self.distance_bias["far"]
@@ -214,8 +259,13 @@ class GQAAttention(PagedSoftmaxMixer):
 
     def weights(self) -> list[WeightDecl]:
         q, kv, nm = self.q_size, self.kv_size, self.names
-        spans = (("q", 0, q), ("k", q, q + kv)) + ((("v", q + kv, self.qkv_width),) if not self.values_are_keys else ())
+        spans = (("q", 0, q), ("k", q, q + kv)) + ((("v", q + kv, q + kv + self.v_size),) if not self.values_are_keys else ())
         extra = []
+        if self.head_gate is not None:
+            at = q + kv + self.v_size
+            extra.append(WeightDecl(self.head_gate, (self.n_heads, self.hidden), dest=self.w_qkv[at:at + self.n_heads]))
+        if self.value_mix is not None:
+            extra.append(WeightDecl(self.value_mix["name"], (), role="vector", init="wide_normal", dest=self.mix_weight.view(())))
         if self.qk_norm is not None:
             extra += [WeightDecl(self.qk_norm["q"], (self.head_dim,), role="vector", init="one_plus_normal", dest=self.q_norm_w),
                       WeightDecl(self.qk_norm["k"], (self.head_dim,), role="vector", init="one_plus_normal", dest=self.k_norm_w)]
@@ -232,7 +282,7 @@ class GQAAttention(PagedSoftmaxMixer):
 
     def cache_need(self) -> PagedKV:
         return PagedKV(self.n_kv_heads, self.head_dim, self.window, None if self.same_dims else self.v_dim,
-                       values_are_keys=self.values_are_keys)
+                       values_are_keys=self.values_are_keys, chunk=self.chunk)
 
     def _fused_table(self):
         """The rotation table of the kernels that rotate on the way; None where the mixer takes the separate steps."""
@@ -256,7 +306,7 @@ class GQAAttention(PagedSoftmaxMixer):
         """h @ [Wq; Wk; Wv].T without the bias: a tensor, or the slices of a split product where the kernel
         that follows adds them itself (both rotary kernels do).  With the cache the attention will read, the
         product knows how large that launch will be and lets a small one settle on the SMs while it runs."""
-        rotary = self._fused_table() is not None
+        rotary = self._fused_table() is not None or self.prepared
         fused = self._fused_decode(ctx) is not None
         early = False
         if fused and cache is not None:
@@ -291,6 +341,8 @@ class GQAAttention(PagedSoftmaxMixer):
         """Bias, position encoding, cache write and attention for the step's rows; [rows, Hq * D]."""
         n, ws, dt = ctx.n_tokens, ctx.workspace, self.runtime.dtype
         table = self._fused_table()
+        if self.prepared:
+            return self._attend_prepared(ctx, qkv, cache, write_cache)
         source = None
         if isinstance(qkv, SplitSum):       # the kernels below add the slices themselves
             source, qkv = qkv, ws.get("attn.qkv", (n, self.qkv_width), dt)
@@ -334,4 +386,26 @@ class GQAAttention(PagedSoftmaxMixer):
                           cache.k_pages, cache.v_pages, n, self.n_heads, self.n_kv_heads, self.head_dim,
                           write_cache, ctx.status, source=source)
         self._attend(ctx, out, qkv, cache)
+        return out
+
+    def _attend_prepared(self, ctx: StepContext, qkv, cache: PagedView, write_cache: bool) -> torch.Tensor:
+        """One pass over the product's rows, then attention (mixers with a head gate or mixed values)."""
+        n, ws, dt = ctx.n_tokens, ctx.workspace, self.runtime.dtype
+        q = ws.get("attn.q", (n, self.q_size), dt)
+        out = ws.get("attn.out", (n, self.out_size), dt)
+        gate = ws.get("attn.gate", (n, self.n_heads), torch.float32) if self.head_gate is not None else None
+        more = {}
+        if self.position.kind != "none":
+            plan = self.position.rotary_plan(self.head_dim)
+            more.update(rot_dims=plan.rot_dims, inv_freq=plan.inv_freq, interleaved=plan.interleaved, magnitude=plan.magnitude)
+        if self.value_mix is not None and self.value_mix["role"] == "first":
+            ctx.kept["values"] = more["leave_values"] = ws.get("attn.first_values", (n, self.v_size), dt)
+        elif self.value_mix is not None:
+            kept = ctx.kept.get("values")
+            if kept is None or tuple(kept.shape) != (n, self.v_size):
+                raise RuntimeError("attention: no earlier layer of this step has left values of this layer's size to mix with")
+            more.update(mix_values=kept, mix_weight=self.mix_weight)
+        ops.attention_prepare(q, qkv, n, self.n_heads, self.n_kv_heads, self.head_dim, self.v_dim, ctx.positions, ctx.seq_of_token,
+                              ctx.seq_slot, cache.block_table, cache.k_pages, cache.v_pages, write_cache, ctx.status, gate=gate, **more)
+        self._attend(ctx, out, q, cache, gate)
         return out

@@ -72,16 +72,29 @@ class WeightDecl:
 class PagedKV:
     """Keys and values for every token (or the last ``window`` tokens), in pages.  ``v_head_dim``: the size of
     a value row where it differs from a key row's (``None``: the same).  ``values_are_keys``: a position's value is
-    its key; one set of pages serves as both."""
+    its key; one set of pages serves as both.  ``chunk``: positions are counted off in chunks of that many from the
+    request's start, and only keys of the chunk that is being filled are needed (not together with ``window``)."""
     kv_heads: int
     head_dim: int
     window: int | None = None
     v_head_dim: int | None = None
     values_are_keys: bool = False
+    chunk: int | None = None
 
     @property
     def value_dim(self) -> int:
         return self.head_dim if self.v_head_dim is None else self.v_head_dim
+
+    @property
+    def span(self) -> int | None:
+        """The most keys a token sees; None: all before it."""
+        return self.window if self.chunk is None else self.chunk
+
+    def first_needed(self, position: int) -> int:
+        """The first position whose key a token at ``position`` sees (tokens behind it see none before that either)."""
+        if self.chunk is not None:
+            return position - position % self.chunk
+        return 0 if self.window is None else max(0, position - self.window + 1)
 
 
 @dataclass(frozen=True)
@@ -225,6 +238,7 @@ class StepContext:
     decode_only: bool = False      # every sequence brings exactly one token
     fixed_shape: bool = False      # the launch is being captured: sizes must not depend on host values of this step
     device_tokens: torch.Tensor | None = None   # int32: token ids the previous step left on the device (id -(i+1) -> [i])
+    kept: dict = field(default_factory=dict)      # rows of this step that a layer leaves for later layers, by name
     upcoming_weights: torch.Tensor | None = None  # set by a block: what the part after the running one streams first
 
 

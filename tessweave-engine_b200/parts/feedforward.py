@@ -5,42 +5,60 @@ import torch
 
 from ..csrc import ops
 from .base import FeedForward, PartSpec, Runtime, StepContext, WeightDecl, build_part, dense_delta, join_name, register_part
-from .linear import grouped_matmul_nt, grouped_product_on_device, linear
+from .linear import grouped_matmul_nt, grouped_product_on_device, linear, matmul_nt
 
 
-@register_part("feed_forward", "swiglu")
-class SwiGLU(FeedForward):
-    """delta = (silu(h @ Wg.T) * (h @ Wu.T)) @ Wd.T, no biases.
+@register_part("feed_forward", "gated_mlp")
+class GatedMLP(FeedForward):
+    """delta = (act(h @ Wg.T [+ bg]) * (h @ Wu.T [+ bu])) @ Wd.T [+ bd], act one of ``ops.ACTIVATIONS``.
 
     gate and up are one product.  The reference packs the rows [Wg; Wu]
     (flow_engine/model.py:82-85); here, when the intermediate size is a multiple of 8, the rows
     alternate between eight gate rows and their eight up rows -- an exact permutation -- so
     that a tensor-core tile of the small-batch kernel holds a gate and its up in one thread and
-    writes silu(gate) * up directly.  The activation runs in fp32.
-    Reference: flow_engine/model.py:68-85.
+    writes act(gate) * up directly; the biases of gate and up lie in the same order.  The activation runs in fp32.
+    Reference (silu, no biases): flow_engine/model.py:68-85.
     """
 
     NAMES = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+    BIAS_NAMES = ("gate_proj.bias", "up_proj.bias", "down_proj.bias")
 
-    def __init__(self, runtime: Runtime, hidden: int, intermediate: int, names: tuple[str, str, str] | None = None):
-        """``names``: the checkpoint's names of the gate, up and down matrices (default: the reference's)."""
+    def __init__(self, runtime: Runtime, hidden: int, intermediate: int, names: tuple[str, str, str] | None = None,
+                 activation: str = "silu", bias_names: tuple[str, str, str] | None = None):
+        """``names``: the checkpoint's names of the gate, up and down matrices (default: the reference's);
+        ``bias_names``: of their biases (None: no biases)."""
         super().__init__(runtime)
         self.names = tuple(names) if names else self.NAMES
+        self.bias_names = tuple(bias_names) if bias_names else None
         if min(hidden, intermediate) <= 0:
-            raise ValueError("swiglu needs positive sizes")
+            raise ValueError("a gated feed-forward needs positive sizes")
+        if activation not in ops.ACTIVATIONS:
+            raise ValueError(f"unknown activation {activation!r} (known: {', '.join(sorted(ops.ACTIVATIONS))})")
+        self.act = ops.ACTIVATIONS[activation]
         self.hidden, self.intermediate = hidden, intermediate
         self.w_gate_up = runtime.empty(2 * intermediate, hidden)
         self.w_down = runtime.empty(hidden, intermediate)
+        self.b_gate_up = runtime.empty(2 * intermediate) if self.bias_names else None
+        self.b_down = runtime.empty(hidden) if self.bias_names else None
         self.interleaved = intermediate % 8 == 0
+
+    def _halves(self, packed: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
+        """The gate rows and the up rows of a packed tensor, as views."""
+        i = self.intermediate
+        if not self.interleaved:
+            return packed[:i], packed[i:]
+        groups = packed.view(i // 8, 2, 8, *packed.shape[1:])
+        return groups[:, 0], groups[:, 1]                  # [i / 8, 8, ...] views; the loader reshapes the source
 
     def weights(self) -> list[WeightDecl]:
         i = self.intermediate
-        if self.interleaved:
-            groups = self.w_gate_up.view(i // 8, 2, 8, self.hidden)
-            gate, up = groups[:, 0], groups[:, 1]          # [i / 8, 8, hidden] views; the loader reshapes the source
-        else:
-            gate, up = self.w_gate_up[:i], self.w_gate_up[i:]
-        return [WeightDecl(self.names[0], (i, self.hidden), dest=gate),
+        gate, up = self._halves(self.w_gate_up)
+        biases = []
+        if self.bias_names:
+            bg, bu = self._halves(self.b_gate_up)
+            biases = [WeightDecl(self.bias_names[0], (i,), dest=bg), WeightDecl(self.bias_names[1], (i,), dest=bu),
+                      WeightDecl(self.bias_names[2], (self.hidden,), dest=self.b_down)]
+        return biases + [WeightDecl(self.names[0], (i, self.hidden), dest=gate),
                 WeightDecl(self.names[1], (i, self.hidden), dest=up),
                 WeightDecl(self.names[2], (self.hidden, i), dest=self.w_down)]
 
@@ -52,20 +70,21 @@ class SwiGLU(FeedForward):
 
     def down(self, ctx: StepContext, act: torch.Tensor):
         """delta = act @ Wd.T (a tensor, or the slices of the product for the next norm to add)."""
-        return linear(ctx, "ffn.delta", act, self.w_down, allow_split=True, consumer_early=True)
+        return linear(ctx, "ffn.delta", act, self.w_down, allow_split=True, consumer_early=True, bias=self.b_down)
 
     def gate_up(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
-        """act = silu(h @ Wg.T) * (h @ Wu.T), by whichever kernel takes the step's number of rows."""
+        """act(gate) * up, by whichever kernel takes the step's number of rows."""
         n, ws, dt = ctx.n_tokens, ctx.workspace, self.runtime.dtype
         act = ws.get("ffn.act", (n, self.intermediate), dt)
+        how = {"act": self.act, "bias": self.b_gate_up}
         if self.interleaved and ops.small_m_supported(h, self.w_gate_up, n):
-            ops.gemm_small_m(act, h, self.w_gate_up, n, silu_mul_pairs=True,
+            ops.gemm_small_m(act, h, self.w_gate_up, n, silu_mul_pairs=True, **how,
                              prefetch=ops.weight_head(self.w_down, ops.product_prefetch_bytes()))
         elif (self.interleaved and ops.stream_product_preferred(h, self.w_gate_up, n)
               and (ops.stream_whole_k_balanced(2 * self.intermediate) or ops.stream_split_gate_up_enabled())):
             # decode steps of 9 to 64 requests: persistent tcgen05 kernel, weights as the 128-row operand
             if ops.stream_whole_k_balanced(2 * self.intermediate):
-                ops.gemm_tcgen05_stream(act, h, self.w_gate_up, n, ctx.status, silu_mul_pairs=True,    # SiLU.mul in its epilogue
+                ops.gemm_tcgen05_stream(act, h, self.w_gate_up, n, ctx.status, silu_mul_pairs=True, **how,    # act.mul in its epilogue
                                         prefetch=ops.weight_head(self.w_down, ops.product_prefetch_bytes()))
             else:
                 # the row tiles alone would leave half of the blocks with half of the work: slices over k, added
@@ -73,15 +92,64 @@ class SwiGLU(FeedForward):
                 split, kper = ops.stream_split(2 * self.intermediate, self.hidden)
                 slices = ws.get("ffn.gate_up.slices", (split, n, 2 * self.intermediate), torch.float32)
                 ops.gemm_tcgen05_stream(slices if split > 1 else slices[0], h, self.w_gate_up, n, ctx.status, kper=kper)
-                ops.silu_mul(act, ops.SplitSum(slices), n, True)
+                ops.silu_mul(act, ops.SplitSum(slices), n, True, **how)
         elif self.interleaved and ops.pair_product_preferred(h, self.w_gate_up, n):
             # prompt steps: 256 x 256 tiles on pairs of thread blocks (tcgen05.mma.cta_group::2), SiLU.mul in the
             # epilogue, so the [tokens, 2 * intermediate] product never reaches memory
-            ops.gemm_tcgen05_pair(act, h, self.w_gate_up, n, ctx.status, silu_mul_pairs=True)
+            ops.gemm_tcgen05_pair(act, h, self.w_gate_up, n, ctx.status, silu_mul_pairs=True, **how)
         else:
             gate_up = linear(ctx, "ffn.gate_up", h, self.w_gate_up)
-            ops.silu_mul(act, gate_up, n, self.interleaved)
+            ops.silu_mul(act, gate_up, n, self.interleaved, **how)
         return act
+
+
+@register_part("feed_forward", "swiglu")
+class SwiGLU(GatedMLP):
+    """delta = (silu(h @ Wg.T) * (h @ Wu.T)) @ Wd.T, no biases."""
+
+    def __init__(self, runtime: Runtime, hidden: int, intermediate: int, names: tuple[str, str, str] | None = None):
+        super().__init__(runtime, hidden, intermediate, names)
+
+
+@register_part("feed_forward", "plain_mlp")
+class PlainMLP(FeedForward):
+    """delta = act(h @ Wu.T) @ Wd.T: two matrices, no gate, no biases; act one of ``ops.ACTIVATIONS``.
+
+    Where a hand-written kernel takes the step's number of rows the activation is in its epilogue (fp32, one rounding);
+    else the library's product is followed by a pass over its rows."""
+
+    def __init__(self, runtime: Runtime, hidden: int, intermediate: int, activation: str, names: tuple[str, str] = ("up", "down")):
+        super().__init__(runtime)
+        if min(hidden, intermediate) <= 0:
+            raise ValueError("plain_mlp needs positive sizes")
+        if activation not in ops.ACTIVATIONS:
+            raise ValueError(f"unknown activation {activation!r} (known: {', '.join(sorted(ops.ACTIVATIONS))})")
+        self.hidden, self.intermediate, self.names = hidden, intermediate, tuple(names)
+        self.act = ops.ACTIVATIONS[activation]
+        self.w_up = runtime.empty(intermediate, hidden)
+        self.w_down = runtime.empty(hidden, intermediate)
+
+    def weights(self) -> list[WeightDecl]:
+        return [WeightDecl(self.names[0], (self.intermediate, self.hidden), dest=self.w_up),
+                WeightDecl(self.names[1], (self.hidden, self.intermediate), dest=self.w_down)]
+
+    def streamed_first(self) -> torch.Tensor:
+        return self.w_up
+
+    def forward(self, ctx: StepContext, h: torch.Tensor):
+        n, ws, dt = ctx.n_tokens, ctx.workspace, self.runtime.dtype
+        act = ws.get("mlp.act", (n, self.intermediate), dt)
+        if ops.small_m_supported(h, self.w_up, n):
+            ops.gemm_small_m(act, h, self.w_up, n, act=self.act, prefetch=ops.weight_head(self.w_down, ops.product_prefetch_bytes()))
+        elif ops.stream_product_preferred(h, self.w_up, n) and ops.stream_whole_k_balanced(self.intermediate):
+            ops.gemm_tcgen05_stream(act, h, self.w_up, n, ctx.status, act=self.act,
+                                    prefetch=ops.weight_head(self.w_down, ops.product_prefetch_bytes()))
+        elif ops.pair_product_preferred(h, self.w_up, n):
+            ops.gemm_tcgen05_pair(act, h, self.w_up, n, ctx.status, act=self.act)
+        else:
+            matmul_nt(act, h, self.w_up)
+            ops.activate_rows(act, n, self.act)
+        return linear(ctx, "mlp.delta", act, self.w_down, allow_split=True, consumer_early=True)
 
 
 @register_part("feed_forward", "routed_experts")
@@ -107,7 +175,9 @@ class RoutedExperts(FeedForward):
     the weights are their s times ``weight_scale``, not renormalised.  ``identity`` n: the router has n outputs more
     than there are experts; such an output is an expert without tensors whose result is the token's row itself.
     ``activation``: ``{"kind": "clamped", "limit": l, "alpha": a}`` makes an expert's inner rows
-    g sigmoid(a g) (u + 1) with g = min(Wg h, l), u = clamp(Wu h, -l, l) instead of silu(Wg h) (Wu h).
+    g sigmoid(a g) (u + 1) with g = min(Wg h, l), u = clamp(Wu h, -l, l) instead of silu(Wg h) (Wu h).  ``{"kind":
+    "plain", "function": f}``: experts without a gate, f(Wu h) with f one of ``ops.ACTIVATIONS`` (tensors ``up`` and
+    ``down`` only, up stacked as [experts, ff, hidden]).
     """
 
     GROUPED_MIN_ROWS = 1       # measured at 7B and 1.5B layer sizes: the sorted way is the faster one from two or three rows on
@@ -127,9 +197,14 @@ class RoutedExperts(FeedForward):
         self.identity, self.outputs = int(identity), experts + int(identity)
         self.score_all, self.weight_scale = bool(score_all), float(weight_scale)
         self.glu, self.glu_limit, self.glu_alpha = ops.GLU_SILU, 0.0, 1.0
-        if activation is not None:
+        self.plain_act = None          # set for experts without a gate
+        if activation is not None and activation.get("kind") == "plain":
+            if activation.get("function") not in ops.ACTIVATIONS:
+                raise ValueError(f"routed_experts: unknown activation {activation!r} (known functions: {', '.join(sorted(ops.ACTIVATIONS))})")
+            self.plain_act = ops.ACTIVATIONS[activation["function"]]
+        elif activation is not None:
             if activation.get("kind") != "clamped" or not float(activation["limit"]) > 0:
-                raise ValueError(f"routed_experts: unknown activation {activation!r} (known: clamped with a positive limit)")
+                raise ValueError(f"routed_experts: unknown activation {activation!r} (known: plain, and clamped with a positive limit)")
             self.glu, self.glu_limit, self.glu_alpha = ops.GLU_CLAMPED, float(activation["limit"]), float(activation.get("alpha", 1.0))
         self.names = {"router": "router", "router_bias": "router.b", "expert": "e", "gate": "gate", "up": "up", "down": "down",
                       "shared": "shared", "shared_gate": "shared.sg", **(names or {})}
@@ -137,7 +212,9 @@ class RoutedExperts(FeedForward):
         self.b_router = runtime.empty(self.outputs, dtype=torch.float32) if router_bias else None
         self.correction_name = correction
         self.correction = runtime.empty(self.outputs, dtype=torch.float32) if correction is not None else None
-        self.w_gate_up = runtime.empty(experts, 2, intermediate, hidden)
+        self.gated = self.plain_act is None
+        self.w_gate_up = runtime.empty(experts, 2, intermediate, hidden) if self.gated else None
+        self.w_up = None if self.gated else runtime.empty(experts, intermediate, hidden)
         self.w_down = runtime.empty(experts, hidden, intermediate)
         self.shared = build_part("feed_forward", shared, runtime) if shared is not None else None
         self.w_shared_gate = runtime.empty(1, hidden) if shared_gate else None
@@ -152,8 +229,9 @@ class RoutedExperts(FeedForward):
             decls.append(WeightDecl(self.correction_name, (self.outputs,), role="vector", init="wide_normal", dest=self.correction))
         for e in range(self.experts):
             p = f"{nm['expert']}{e}"
-            decls += [WeightDecl(join_name(p, nm["gate"]), (f, hid), dest=self.w_gate_up[e, 0]),
-                      WeightDecl(join_name(p, nm["up"]), (f, hid), dest=self.w_gate_up[e, 1]),
+            if self.gated:
+                decls.append(WeightDecl(join_name(p, nm["gate"]), (f, hid), dest=self.w_gate_up[e, 0]))
+            decls += [WeightDecl(join_name(p, nm["up"]), (f, hid), dest=self.w_gate_up[e, 1] if self.gated else self.w_up[e]),
                       WeightDecl(join_name(p, nm["down"]), (hid, f), dest=self.w_down[e])]
         if self.shared is not None:
             decls += [WeightDecl(join_name(nm["shared"], w.name), w.shape, w.role, w.init, w.dest) for w in self.shared.weights()]
@@ -193,7 +271,10 @@ class RoutedExperts(FeedForward):
             # (a library without a grouped product reads the group bounds on the host: not inside a captured step)
             self._grouped(ctx, h, chosen, weight, shared, gate, out, sorted_buffers)
             return out
-        ops.moe_gate_up(act, h, self.w_gate_up, chosen, n, glu=self.glu, limit=self.glu_limit, alpha=self.glu_alpha)
+        if self.gated:
+            ops.moe_gate_up(act, h, self.w_gate_up, chosen, n, glu=self.glu, limit=self.glu_limit, alpha=self.glu_alpha)
+        else:
+            ops.moe_up(act, h, self.w_up, chosen, n, self.plain_act)
         ops.moe_down(out, act, self.w_down, chosen, weight, shared, gate, n, h=h if self.identity else None, identity=self.identity)
         return out
 
@@ -218,11 +299,15 @@ class RoutedExperts(FeedForward):
         order, place, ends, xs, act = buffers
         ops.moe_sort(order, place, ends, chosen, n)
         ops.moe_gather(xs, h, order, pairs, self.top)
-        gate_up = grouped_matmul_nt(xs, self.w_gate_up.view(self.experts, 2 * self.intermediate, self.hidden), ends)
-        if self.glu == ops.GLU_SILU:
-            ops.silu_mul(act, gate_up, pairs, False)
+        if not self.gated:
+            act = grouped_matmul_nt(xs, self.w_up, ends)
+            ops.activate_rows(act, pairs, self.plain_act)
         else:
-            ops.glu_rows(act, gate_up, pairs, self.glu, self.glu_limit, self.glu_alpha)
+            gate_up = grouped_matmul_nt(xs, self.w_gate_up.view(self.experts, 2 * self.intermediate, self.hidden), ends)
+            if self.glu == ops.GLU_SILU:
+                ops.silu_mul(act, gate_up, pairs, False)
+            else:
+                ops.glu_rows(act, gate_up, pairs, self.glu, self.glu_limit, self.glu_alpha)
         ys = grouped_matmul_nt(act, self.w_down, ends)
         if self.identity:
             ops.moe_combine(out, ys, place, weight, shared, gate, n, chosen=chosen, h=h, experts=self.experts, identity=self.identity)

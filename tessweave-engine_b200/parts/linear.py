@@ -43,15 +43,17 @@ def verify_true_fp32(device) -> None:
                            f"(256 x (1 + 2**-12)**2 came out {float(got[0, 0])!r}); a reduced-precision matrix mode is on")
 
 
-def matmul_nt(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    """out[n, o] = sum_i x[n, i] * w[o, i].  x and w are of one element type; out is of the
-    same type, or fp32 for a bf16 product whose result must not be rounded (the logits)."""
+def matmul_nt(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None) -> torch.Tensor:
+    """out[n, o] = sum_i x[n, i] * w[o, i] [+ bias[o]].  x, w and bias are of one element type; out is of the
+    same type, or fp32 for a bf16 product whose result must not be rounded (the logits; without a bias)."""
     if not _configured:
         configure_matmul_precision()
     if not x.is_cuda:
         raise RuntimeError("matrix products run on the GPU only; this engine has no CPU path")
     ops.note_call("library product (cuBLAS)")
-    if out.dtype != x.dtype:
+    if bias is not None:
+        torch.addmm(bias, x, w.t(), out=out)
+    elif out.dtype != x.dtype:
         torch.mm(x, w.t(), out_dtype=out.dtype, out=out)
     else:
         torch.mm(x, w.t(), out=out)
@@ -60,8 +62,9 @@ def matmul_nt(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> torch.Tens
 
 def linear(ctx, name: str, x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype | None = None,
            allow_split: bool = False, consumer_early: bool = False, max_slices: int = 12,
-           prefetch: torch.Tensor | None = None):
-    """``x @ w.T`` into the workspace buffer ``name``.
+           prefetch: torch.Tensor | None = None, bias: torch.Tensor | None = None):
+    """``x @ w.T [+ bias]`` into the workspace buffer ``name`` (``bias``: one value of x's type per output; a ``SplitSum``
+    holds it in its first slice).
 
     Steps with up to 8 rows (decode) in bfloat16 go through the weight-streaming kernel of
     csrc/gemm_smallm.cu; products of 9 to 64 rows with a large matrix (down, logits) through the persistent
@@ -83,27 +86,27 @@ def linear(ctx, name: str, x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dt
         if split > 1 and allow_split:
             slices = ctx.workspace.get(name + ".slices", (split, m, n), torch.float32)
             ops.gemm_tcgen05_stream(slices, x, w, m, ctx.status, kper=kper, early_dependents=consumer_early,
-                                    prefetch=prefetch)
+                                    prefetch=prefetch, bias=bias)
             return SplitSum(slices)
         if split == 1:
             out = ctx.workspace.get(name, (m, n), dtype)
-            ops.gemm_tcgen05_stream(out, x, w, m, ctx.status, early_dependents=consumer_early, prefetch=prefetch)
+            ops.gemm_tcgen05_stream(out, x, w, m, ctx.status, early_dependents=consumer_early, prefetch=prefetch, bias=bias)
             return out
         # slices that nobody would add: the library's product below, which reduces its own split inside the kernel
     if x.is_cuda and ops.small_m_supported(x, w, m):
         split, kper = ops.small_m_split(n, w.shape[1], max_slices if allow_split else 12)
         if split > 1 and allow_split:
             slices = ctx.workspace.get(name + ".slices", (split, m, n), torch.float32)
-            ops.gemm_small_m(slices, x, w, m, kper, early_dependents=consumer_early, prefetch=prefetch)
+            ops.gemm_small_m(slices, x, w, m, kper, early_dependents=consumer_early, prefetch=prefetch, bias=bias)
             return SplitSum(slices)
         if split > 1:
             slices = ctx.workspace.get(name + ".slices", (split, m, n), torch.float32)
-            ops.gemm_small_m(slices, x, w, m, kper)
+            ops.gemm_small_m(slices, x, w, m, kper, bias=bias)
             return SplitSum(slices).dense(dtype, ctx.workspace.get(name, (m, n), dtype))
         out = ctx.workspace.get(name, (m, n), dtype)
-        ops.gemm_small_m(out, x, w, m, early_dependents=consumer_early, prefetch=prefetch)
+        ops.gemm_small_m(out, x, w, m, early_dependents=consumer_early, prefetch=prefetch, bias=bias)
         return out
-    return matmul_nt(ctx.workspace.get(name, (m, n), dtype), x, w)
+    return matmul_nt(ctx.workspace.get(name, (m, n), dtype), x, w, bias)
 
 
 _grouped_library: list = [None]     # True / False once the library's grouped product has been tried

@@ -104,6 +104,28 @@ class RotaryEmbedding(PositionEncoding):
                              magnitude=self.magnitude)
 
 
+def checked_bands(bands: dict | None) -> dict | None:
+    """The four numbers of a ``bands`` parameter as floats, or None."""
+    if bands is None:
+        return None
+    b = {k: float(bands[k]) for k in ("factor", "low", "high", "original")}
+    if not (b["factor"] > 0 and b["original"] > 0 and b["low"] >= 0 and b["high"] > b["low"]):
+        raise ValueError("rope: bands need positive factor and original, low not negative, and high above low")
+    return b
+
+
+def banded_frequencies(theta: float, dims: int, bands: dict) -> list[float]:
+    """The turning rate of every pair under the rule of three bands (see ``InterleavedRotaryEmbedding``), in double
+    precision."""
+    out = []
+    for i in range(dims // 2):
+        f = theta ** (-2.0 * i / dims)
+        turns = bands["original"] * f / (2.0 * math.pi)             # turns over the original length
+        share = min(max((turns - bands["low"]) / (bands["high"] - bands["low"]), 0.0), 1.0)
+        out.append(share * f + (1.0 - share) * f / bands["factor"])
+    return out
+
+
 @register_part("position", "rope_interleaved")
 class InterleavedRotaryEmbedding(PositionEncoding):
     """Rotary encoding on neighbouring pairs, over the first ``dims`` values of a head (all of it when
@@ -114,11 +136,20 @@ class InterleavedRotaryEmbedding(PositionEncoding):
 
     all in fp32.  The table of f_i is made once per head size on the host.  ``yarn`` as for ``rope``: stretched
     rates per pair, and cos and sin both multiplied by 0.1 ln(factor) + 1.
+
+    ``bands`` (``factor``, ``low``, ``high``, ``original``): the frequency scaling of Llama 3.1.  A pair that makes at
+    least ``high`` turns over the ``original`` length keeps its rate, one that makes at most ``low`` turns is slowed by
+    ``factor``, and between the two the rate is the blend s f_i + (1 - s) f_i / factor with
+    s = (turns - low) / (high - low); cos and sin are not scaled.
     """
 
-    def __init__(self, runtime: Runtime, theta: float, dims: int | None = None, yarn: dict | None = None):
+    def __init__(self, runtime: Runtime, theta: float, dims: int | None = None, yarn: dict | None = None,
+                 bands: dict | None = None):
         super().__init__(runtime)
         self.yarn, self.magnitude = checked_yarn(yarn, theta)
+        self.bands = checked_bands(bands)
+        if self.yarn is not None and self.bands is not None:
+            raise ValueError("rope: the rates are stretched by yarn or by bands, not both")
         if not theta > 0:
             raise ValueError("rope theta must be positive")
         if dims is not None and (dims < 0 or dims % 2):
@@ -132,7 +163,9 @@ class InterleavedRotaryEmbedding(PositionEncoding):
             dims = head_dim if self.dims is None else self.dims
             if dims > head_dim or dims % 2:
                 raise ValueError(f"rope over {dims} dims does not fit a head of {head_dim}")
-            if self.yarn is None:
+            if self.bands is not None:
+                inv = torch.tensor(banded_frequencies(self.theta, dims, self.bands), dtype=torch.float64).to(torch.float32)
+            elif self.yarn is None:
                 inv = self.theta ** (-torch.arange(0, dims, 2, dtype=torch.float32) / max(dims, 1))
             else:
                 inv = torch.tensor(stretched_frequencies(self.theta, dims, self.yarn), dtype=torch.float64).to(torch.float32)

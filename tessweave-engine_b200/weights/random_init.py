@@ -95,6 +95,8 @@ def fill_random(model: Model, seed: int = 0, std: float | None = None) -> Model:
             noise = torch.randn(decl.shape, generator=g, device=device, dtype=torch.float32)
             decl.dest.copy_(torch.eye(decl.shape[0], decl.shape[1], device=device) + std * noise)
             continue
+        if decl.dest.dim() == 0:                # a single number: drawn as a row of one, in place
+            decl.dest = decl.dest.view(1)
         rows = decl.dest.shape[0]
         step = max(1, (64 << 20) // max(1, decl.dest[0].numel() if decl.dest.dim() > 1 else 1))
         for begin in range(0, rows, step):      # in slabs, so no second full-size copy is alive
