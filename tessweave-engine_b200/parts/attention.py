@@ -179,7 +179,7 @@ class GQAAttention(PagedSoftmaxMixer):
                              "values that are the keys")
         if min(hidden, n_heads, n_kv_heads, head_dim) <= 0 or n_heads % n_kv_heads:
             raise ValueError("attention: heads must be positive and n_heads a multiple of n_kv_heads")
-        if (head_dim % 2 and position.kind != "none") or head_dim > 1024:
+        if (head_dim % 2 and position.kind != "none" and not self.prepared) or head_dim > 1024:
             raise ValueError(f"attention: head_dim {head_dim} must be at most 1024, and even where heads are rotated")
         if out_bias:
             raise ValueError("attention: a bias on the output projection is not implemented")

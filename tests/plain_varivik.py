@@ -36,7 +36,7 @@ def turning_rates(dims, base, scaling):
         if scaling is not None:
             length = 2.0 * math.pi / f
             low, high, original, factor = (float(scaling[k]) for k in ("low", "high", "original", "factor"))
-            if length > original / low:
+            if length * low > original:
                 f = f / factor
             elif length >= original / high:
                 s = (original / length - low) / (high - low)
