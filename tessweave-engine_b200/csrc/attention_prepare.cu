@@ -94,8 +94,8 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&x)[8]) {
 }
 
 // VEC: eight neighbouring columns per item (pairs of neighbours, head sizes that are multiples of 8, 16-byte aligned
-// rows); otherwise a pair, or a single value that is not rotated, per item.
-template <typename T, bool VEC>
+// rows); otherwise a pair, or a single value that is not rotated, per item.  SLICES: `partial` is the source.
+template <typename T, bool VEC, bool SLICES>
 __global__ void __launch_bounds__(256)
 attention_prepare_kernel(T* __restrict__ q_out, const T* __restrict__ rows, int row_stride, const float* __restrict__ partial,
                          int nsplit, size_t split_stride, T* first, T* __restrict__ k_cache, T* __restrict__ v_cache,
@@ -128,42 +128,59 @@ attention_prepare_kernel(T* __restrict__ q_out, const T* __restrict__ rows, int 
     const int at = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
     if constexpr (VEC) {
         const int n8 = (q_size + k_size + v_size) >> 3;
-        for (int item = at; item < n8; item += step) {
-            const int col = item << 3;
-            float x[8];
-            if (prow) sum_slices<8>(prow + col, nsplit, split_stride, x);
-            else load8(row + col, x);
-            if (col < q_size + k_size) {
-                const int c = col < q_size ? col : col - q_size;
-                const int head = c / D, d = c - head * D;
+        // rows: the loads of up to three items go out before the first store (one round trip to memory, not three)
+        constexpr int AHEAD = SLICES ? 1 : 3, RAW = sizeof(T) / 2;
+        for (int base = at; base < n8; base += AHEAD * step) {
+            uint4 raw[AHEAD][RAW];
+            if constexpr (!SLICES) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    if (d + 2 * e < a.rot_dims) {
-                        const float2 t = turn[(d >> 1) + e];
-                        const float u = x[2 * e], v = x[2 * e + 1];
-                        x[2 * e] = u * t.x - v * t.y;
-                        x[2 * e + 1] = v * t.x + u * t.y;
+                for (int j = 0; j < AHEAD; ++j) {
+                    const int item = base + j * step;
+#pragma unroll
+                    for (int r = 0; r < RAW; ++r)
+                        raw[j][r] = item < n8 ? __ldg(reinterpret_cast<const uint4*>(row + (item << 3)) + r) : make_uint4(0u, 0u, 0u, 0u);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < AHEAD; ++j) {
+                const int item = base + j * step;
+                if (item >= n8) break;
+                const int col = item << 3;
+                float x[8];
+                if constexpr (SLICES) sum_slices<8>(prow + col, nsplit, split_stride, x);
+                else load8(reinterpret_cast<const T*>(&raw[j][0]), x);
+                if (col < q_size + k_size) {
+                    const int c = col < q_size ? col : col - q_size;
+                    const int head = c / D, d = c - head * D;
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        if (d + 2 * e < a.rot_dims) {
+                            const float2 t = turn[(d >> 1) + e];
+                            const float u = x[2 * e], v = x[2 * e + 1];
+                            x[2 * e] = u * t.x - v * t.y;
+                            x[2 * e + 1] = v * t.x + u * t.y;
+                        }
                     }
-                }
-                if (col < q_size) store8(q_out + (size_t)n * q_size + col, x);
-                else if (store) store8(k_cache + (((size_t)page * a.Hkv + head) * a.page_size + in_page) * D + d, x);
-            } else {
-                const int c = col - q_size - k_size;
-                const int head = c / Dv, d = c - head * Dv;
-                if (a.v_role == 2) {
-                    float f[8];
-                    load8(first + (size_t)n * v_size + c, f);
+                    if (col < q_size) store8(q_out + (size_t)n * q_size + col, x);
+                    else if (store) store8(k_cache + (((size_t)page * a.Hkv + head) * a.page_size + in_page) * D + d, x);
+                } else {
+                    const int c = col - q_size - k_size;
+                    const int head = c / Dv, d = c - head * Dv;
+                    if (a.v_role == 2) {
+                        float f[8];
+                        load8(first + (size_t)n * v_size + c, f);
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) x[e] = (1.f - lam) * x[e] + lam * f[e];
-                } else if (a.v_role == 1) {
-                    store8(first + (size_t)n * v_size + c, x);
+                        for (int e = 0; e < 8; ++e) x[e] = (1.f - lam) * x[e] + lam * f[e];
+                    } else if (a.v_role == 1) {
+                        store8(first + (size_t)n * v_size + c, x);
+                    }
+                    if (store) store8(v_cache + (((size_t)page * a.Hkv + head) * a.page_size + in_page) * Dv + d, x);
                 }
-                if (store) store8(v_cache + (((size_t)page * a.Hkv + head) * a.page_size + in_page) * Dv + d, x);
             }
         }
     } else {
         auto load1 = [&](int col) -> float {
-            if (!prow) return tw_to_float(row[col]);
+            if constexpr (!SLICES) return tw_to_float(row[col]);
             float x[1];
             sum_slices<1>(prow + col, nsplit, split_stride, x);
             return x[0];
@@ -201,7 +218,7 @@ attention_prepare_kernel(T* __restrict__ q_out, const T* __restrict__ rows, int 
         const int g_col = q_size + k_size + v_size;
         for (int h = at; h < a.Hq; h += step) {
             float z[1];
-            if (prow) sum_slices<1>(prow + g_col + h, nsplit, split_stride, z);
+            if constexpr (SLICES) sum_slices<1>(prow + g_col + h, nsplit, split_stride, z);
             else z[0] = tw_to_float(row[g_col + h]);
             a.gate[(size_t)n * a.Hq + h] = 1.f / (1.f + expf(-z[0]));
         }
@@ -216,7 +233,8 @@ int launch(void* q_out, const void* rows, int row_stride, const float* partial, 
     const int room = (2 * 148 + n_tokens - 1) / n_tokens;
     if (parts > room) parts = room;
     if (parts < 1) parts = 1;
-    return tw_launch(attention_prepare_kernel<T, VEC>, dim3(n_tokens, parts), dim3(256), (size_t)(a.rot_dims / 2) * sizeof(float2),
+    auto kernel = partial ? attention_prepare_kernel<T, VEC, true> : attention_prepare_kernel<T, VEC, false>;
+    return tw_launch(kernel, dim3(n_tokens, parts), dim3(256), (size_t)(a.rot_dims / 2) * sizeof(float2),
                      stream, 1, (T*)q_out, (const T*)rows, row_stride, partial, nsplit, (size_t)split_stride, (T*)first,
                      (T*)k_cache, (T*)v_cache, a);
 }

@@ -1,5 +1,5 @@
 // Paged causal attention for prompt portions on the 5th-generation tensor cores, for one head
-// size (compile with -DTW_HEAD_DIM=64 or 128; values of the other size: -DTW_V_DIM).
+// size (compile with -DTW_HEAD_DIM=64 or 128; values of another size: -DTW_V_DIM=32, 64 or 128).
 //
 // A block serves up to 256 rows of one (request, key/value head), a row being a (token, query
 // head of the group) pair, as two tiles of 128 rows, and walks the request's keys in tiles of
@@ -48,11 +48,11 @@ constexpr int BM = 128;                       // rows of a query tile = TMEM lan
 constexpr int NQ = 2;                         // query tiles per block
 constexpr int BN = 128;                       // keys per tile
 constexpr int DV = TW_V_DIM;
-static_assert(DV == 64 || DV == 128, "the tcgen05 attention is built for value sizes 64 and 128");
+static_assert(DV == 32 || DV == 64 || DV == 128, "the tcgen05 attention is built for value sizes 32, 64 and 128");
 constexpr int KB = D / 64;                    // 64-column blocks of a row of q or k
-constexpr int VB = DV / 64;                   // 64-column blocks of a row of v
+constexpr int VB = (DV + 63) / 64;            // 64-column blocks of a row of v (32 values: the copy fills the rest with zeros)
 constexpr int BLK = 128 * 128;                // bytes of a [128 rows][64 columns] swizzled block
-constexpr int KV_STAGES = D == 64 && DV == 64 ? 4 : 2;   // K and V have rings of their own
+constexpr int KV_STAGES = D == 64 && DV <= 64 ? 4 : 2;   // K and V have rings of their own
 constexpr int Q_BYTES = NQ * KB * BLK;
 constexpr int K_STAGE_BYTES = KB * BLK, V_STAGE_BYTES = VB * BLK;
 constexpr int SMEM_TILES = Q_BYTES + KV_STAGES * (K_STAGE_BYTES + V_STAGE_BYTES);

@@ -79,7 +79,8 @@ __device__ __forceinline__ float tw_block_max(float v, float* scratch) {
 enum : int { TW_ACT_NONE = 0, TW_ACT_SILU = 1, TW_ACT_GELU_TANH = 2, TW_ACT_RELU_SQUARED = 3 };
 __device__ __forceinline__ float tw_activate(float z, int act) {
     if (act == TW_ACT_SILU) return z / (1.0f + expf(-z));
-    if (act == TW_ACT_GELU_TANH) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    // 0.5 z (1 + tanh(y)) = z / (1 + exp(-2 y)), which does not cancel for negative z;  y = sqrt(2 / pi) (z + 0.044715 z^3)
+    if (act == TW_ACT_GELU_TANH) return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
     if (act == TW_ACT_RELU_SQUARED) { z = fmaxf(z, 0.f); return z * z; }
     return z;
 }

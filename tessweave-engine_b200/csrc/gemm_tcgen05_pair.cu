@@ -102,6 +102,22 @@ __device__ __forceinline__ void store_chunk(uint32_t (&v)[16], void* out, int ou
 #pragma unroll
         for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(tw_activate(__uint_as_float(v[j]), ep.act));
     }
+    if (out_mode == OUT_GATED && ep.act == TW_ACT_GELU_TANH) {
+        uint4 p;
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&p);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            float a[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const float z = __uint_as_float(v[2 * j + e]);      // (as tw_activate, with the fast exponential)
+                a[e] = z / (1.f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))) * __uint_as_float(v[8 + 2 * j + e]);
+            }
+            h[j] = __floats2bfloat162_rn(a[0], a[1]);
+        }
+        *reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(out) + (size_t)row * out_stride + (col >> 1)) = p;
+        return;
+    }
     if (out_mode == OUT_GATED && ep.act != TW_ACT_SILU) {
         uint4 p;
         __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&p);

@@ -738,9 +738,9 @@ def head_size_defines(head_dim: int, v_dim: int) -> dict[str, int]:
 
 
 def tcgen05_attention_supported(dtype: torch.dtype, head_dim: int, page_size: int, v_dim: int | None = None) -> bool:
-    """The tcgen05 prefill attention takes bfloat16, head sizes 64 and 128, and pages of at least
+    """The tcgen05 prefill attention takes bfloat16, head sizes 64 and 128, values of 32, 64 or 128, and pages of at least
     8 keys that divide a tile of 128 keys or are a multiple of it."""
-    return (dtype == torch.bfloat16 and head_dim in (64, 128) and (v_dim or head_dim) in (64, 128) and page_size >= 8
+    return (dtype == torch.bfloat16 and head_dim in (64, 128) and (v_dim or head_dim) in (32, 64, 128) and page_size >= 8
             and (128 % page_size == 0 or page_size % 128 == 0))
 
 

@@ -100,7 +100,7 @@ def step_times(model, batch: int, context: int, prefill_tokens: int, page_size: 
         runner.check_status()
         ms = begin.elapsed_time(end) / steps
         element = 2
-        nbytes = model.step_weight_bytes(b) + b * (start + warmup + steps / 2) * model.cache_bytes_per_token(element)
+        nbytes = model.step_weight_bytes(b) + b * model.cache_bytes_seen(start + warmup + steps // 2, element)
         out[f"decode_b{b}_ms"] = ms
         out[f"decode_b{b}_tok_s"] = b / (ms / 1e3)
         out[f"decode_b{b}_step_bytes"] = nbytes
@@ -669,6 +669,152 @@ def dugudra_kernel_table(config: dict, batch: int, context: int, prefill_tokens:
             [(lambda r=r, d=d, o=o: norm.apply(ctx, o, r, d, m, delta_scale=cfg.residual_mult)) for r, d, o in sets],
             m * W * (4 + 2 + 4 + 2), 0.0, reps=8)
         del sets
+        torch.cuda.empty_cache()
+    if int(status) != 0:
+        raise RuntimeError(f"a kernel reported status {int(status)} during the kernel table")
+    return rows
+
+
+# ---------------------------------------------------------------------------
+# the Varivik decoder
+# ---------------------------------------------------------------------------
+def varivik_config_like(qwen: dict, layers: int, vdim: int | None = None) -> dict:
+    """A Varivik config.json with the sizes of the Qwen2 configuration ``qwen``: Qwen2's head counts and head size
+    (values of ``vdim``, default the same), half of a head rotated with scaled rates, chunks of 1,024 positions; a dense
+    feed-forward of Qwen2's size in every second layer, in the others eight experts of a quarter of it (two chosen)
+    beside a shared one of half of it."""
+    heads, kv, dim, width, ff = (qwen[k] for k in ("num_attention_heads", "num_key_value_heads", "head_dim", "hidden_size", "intermediate_size"))
+    mixer = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim or dim, "scale": dim ** -0.5, "mask": {"size": 1024}, "v_mix": True,
+             "rot": {"dims": dim // 2, "base": qwen["rope_theta"], "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    mlps = [{"kind": "dense", "ff": ff},
+            {"kind": "moe", "router": {"experts": 8, "top": 2}, "expert": {"ff": ff // 4}, "shared": {"ff": ff // 2}}]
+    return {"architecture": "Varivik", "vocab": qwen["vocab_size"], "width": width, "norm": {"eps": qwen["rms_norm_eps"]},
+            "layers": [{"type": "attention", "mixer": mixer, "mlp": mlps[i % 2]} for i in range(layers)]}
+
+
+def _visible_pairs(tokens: int, chunk: int | None) -> float:
+    """(query, key) pairs of a whole prompt of ``tokens`` tokens."""
+    if chunk is None:
+        return tokens * (tokens + 1) / 2
+    full, rest = divmod(tokens, chunk)
+    return full * chunk * (chunk + 1) / 2 + rest * (rest + 1) / 2
+
+
+def varivik_kernel_table(config: dict, batch: int, context: int, prefill_tokens: int, hbm_gbs: float, tflops: float,
+                         page_size: int = 16, value_dims: tuple = (None,), feed_forward: bool = True) -> list[dict]:
+    """The Varivik kernels alone, each inside a CUDA graph with operands rotated beyond L2, for a decode step of
+    ``batch`` rows and a prompt step: the pass over the projected rows, attention over chunks with gates (for every value
+    size of ``value_dims``; None: the configuration's), the gelu feed-forward with biases, the router, the experts and
+    the shared expert.  fraction = max(bytes / HBM peak, FLOPs / tensor peak) / time."""
+    import tessweave_engine_b200 as tw
+    from ..models.varivik import attention_spec, feed_forward_spec
+    from ..config.varivik_config import DenseConfig
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    rt = Runtime(dev, bf)
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    rows: list[dict] = []
+
+    def add(name, m, thunks, nbytes, flops, reps=4, note=""):
+        kernel = _kernels_of(thunks[0])
+        us = _graph_us(thunks, reps)
+        floor = max(nbytes / (hbm_gbs * 1e9), flops / (tflops * 1e12)) * 1e6
+        rows.append({"op": name, "rows": m, "kernel": kernel, "us": round(us, 2), "mbytes": round(nbytes / 1e6, 2),
+                     "gflop": round(flops / 1e9, 2), "floor_us": round(floor, 2), "frac": round(floor / us, 3),
+                     "bound": "hbm" if nbytes / (hbm_gbs * 1e9) >= flops / (tflops * 1e12) else "tensor", "note": note})
+
+    for m, phase in ((batch, "decode"), (prefill_tokens, "prefill")):
+        requests = batch if phase == "decode" else 1
+        per = m // requests
+        ws = Workspace(dev)
+        kv_tokens = context if phase == "decode" else m
+        ctx = _context(rt, ws, status, [context - 1] * m if phase == "decode" else list(range(m)),
+                       [r for r in range(requests) for _ in range(per)], list(range(requests)), [r * per for r in range(requests)],
+                       [per] * requests, [context] * requests if phase == "decode" else [m])
+        blocks = -(-kv_tokens // page_size)
+        for vdim in value_dims:
+            typed, _ = tw.resolve({**config, "layers": [{**l, "mixer": {**l["mixer"], **({"vdim": vdim} if vdim else {})}} for l in config["layers"]]})
+            side = typed.layers[0].mixer
+            first = build_part("mixer", attention_spec(typed, side, True), rt)
+            att = build_part("mixer", attention_spec(typed, side, False), rt)
+            for part in (first, att):
+                _fill(part)
+                part.finalize()
+            att.mix_weight.fill_(0.4)
+            Hq, G, D, Dv = att.n_heads, att.n_kv_heads, att.head_dim, att.v_dim
+            seen = (kv_tokens - 1) % side.chunk + 1 if side.chunk else kv_tokens
+            per_key = G * (D + Dv) * 2
+            caches = []
+            for _ in range(_copies(requests * (seen if phase == "decode" else kv_tokens) * per_key)):
+                cache = CacheManager([(att.cache_need(), None)], page_size, requests * blocks, requests, kv_tokens, bf, dev, prefix_cache=False)
+                for g in cache.groups:
+                    g.k.normal_(0, 0.5)
+                    g.v.normal_(0, 0.5)
+                for _r in range(requests):
+                    cache.ensure(cache.admit(None), kv_tokens)
+                cache.sync_tables()
+                caches.append(cache)
+            views = [c.view(0) for c in caches]
+            projs = [torch.randn(m, att.qkv_width, device=dev, dtype=bf) for _ in range(_copies(m * att.qkv_width * 2) if phase == "prefill" else 2)]
+            ctx.kept["values"] = torch.randn(m, att.v_size, device=dev, dtype=bf)
+            plan = att.position.rotary_plan(D)
+            qs = [torch.empty(m, att.q_size, device=dev, dtype=bf) for _ in range(2)]
+            gate = torch.rand(m, Hq, device=dev)
+            add(f"{phase}: rotation, blend of values, store, gates ({D} / {Dv})", m,
+                [(lambda v=v, i=i: ops.attention_prepare(
+                    qs[i % 2], projs[i % len(projs)], m, Hq, G, D, Dv, ctx.positions, ctx.seq_of_token, ctx.seq_slot, v.block_table,
+                    v.k_pages, v.v_pages, True, status, rot_dims=plan.rot_dims, inv_freq=plan.inv_freq, interleaved=True, gate=gate,
+                    mix_values=ctx.kept["values"], mix_weight=att.mix_weight)) for i, v in enumerate(views)],
+                m * (2 * att.qkv_width + att.v_size) * 2, 0.0, reps=4)
+            outs = [torch.empty(m, att.out_size, device=dev, dtype=bf) for _ in range(2)]
+            q = torch.randn(m, att.q_size, device=dev, dtype=bf)
+            if phase == "decode":
+                nbytes, flops = m * seen * per_key + m * (att.q_size + att.out_size) * 2, 2.0 * m * Hq * (D + Dv) * seen
+            else:
+                nbytes = m * (att.q_size + att.out_size) * 2 + m * per_key
+                flops = 2.0 * Hq * (D + Dv) * _visible_pairs(m, side.chunk)
+            add(f"{phase}: attention over chunks of {side.chunk}, gates ({D} / {Dv})", m,
+                [(lambda v=v, i=i: att._attend(ctx, outs[i % 2], q, v, gate)) for i, v in enumerate(views)], nbytes, flops,
+                reps=2 if phase == "prefill" else 4)
+            del caches, views, projs, outs, q, qs, att, first
+            torch.cuda.empty_cache()
+        if not feed_forward:
+            continue
+        typed, _ = tw.resolve(config)
+        W = typed.width
+        hs = [torch.randn(m, W, device=dev, dtype=bf) for _ in range(_copies(m * W * 2) if phase == "prefill" else 4)]
+        # ---- the gelu feed-forward with biases
+        mlp = next(l.mlp for l in typed.layers if isinstance(l.mlp, DenseConfig))
+        parts = [build_part("feed_forward", feed_forward_spec(typed, mlp), rt) for _ in range(2)]
+        for part in parts:
+            _fill(part)
+            part.b_gate_up.normal_(0, 0.1)
+            part.b_down.normal_(0, 0.1)
+        acts = [torch.randn(m, mlp.ff, device=dev, dtype=bf) for _ in range(2)]
+        add(f"{phase}: gate/up product + biases + gelu.mul", m, [(lambda p=p, i=i: p.gate_up(ctx, hs[i % len(hs)])) for i, p in enumerate(parts)],
+            2 * mlp.ff * W * 2 + m * (W + mlp.ff) * 2, 2.0 * m * 2 * mlp.ff * W, reps=3)
+        add(f"{phase}: down product + bias", m, [(lambda p=p, i=i: p.down(ctx, acts[i])) for i, p in enumerate(parts)],
+            mlp.ff * W * 2 + m * (W + mlp.ff) * 2, 2.0 * m * mlp.ff * W, reps=3)
+        del parts, acts
+        torch.cuda.empty_cache()
+        # ---- experts
+        mlp = next(l.mlp for l in typed.layers if l.mlp is not None and not isinstance(l.mlp, DenseConfig))
+        parts = [build_part("feed_forward", feed_forward_spec(typed, mlp), rt)
+                 for _ in range(_copies(mlp.experts * 2 * mlp.ff * W * 2) if phase == "decode" else 2)]
+        for part in parts:
+            _fill(part)
+            part.w_router.normal_(0, 0.5)
+        touched = min(mlp.experts, m * mlp.top)
+        add(f"{phase}: router over {mlp.experts} experts, {mlp.top} chosen, shared gate", m,
+            [(lambda p=p, i=i: p.route(ctx, hs[i % len(hs)])) for i, p in enumerate(parts)], m * W * 2 + (mlp.experts + 1) * W * 2, 0.0, reps=8)
+        add(f"{phase}: shared expert (up, square of relu, down)", m,
+            [(lambda p=p, i=i: p.shared.forward(ctx, hs[i % len(hs)])) for i, p in enumerate(parts)],
+            2 * mlp.shared_ff * W * 2 + m * (W + 2 * mlp.shared_ff + W) * 2, 2.0 * m * 2 * mlp.shared_ff * W, reps=3)
+        add(f"{phase}: router, chosen experts, shared expert and the weighted sum", m,
+            [(lambda p=p, i=i: p.forward(ctx, hs[i % len(hs)])) for i, p in enumerate(parts)],
+            touched * 2 * mlp.ff * W * 2 + 2 * mlp.shared_ff * W * 2 + m * W * 4,
+            2.0 * m * 2 * W * (mlp.top * mlp.ff + mlp.shared_ff), reps=2,
+            note="bytes: the matrices of the experts a step of this size touches at most, once")
+        del parts, hs
         torch.cuda.empty_cache()
     if int(status) != 0:
         raise RuntimeError(f"a kernel reported status {int(status)} during the kernel table")

@@ -102,6 +102,13 @@ class Model:
         return sum(need.kv_heads * (need.head_dim + (0 if need.values_are_keys else need.value_dim)) * element_bytes
                    for entry, _ in self.cache_needs() for need in flat_needs(entry) if isinstance(need, PagedKV))
 
+    def cache_bytes_seen(self, tokens: int, element_bytes: int) -> int:
+        """Bytes of keys and values that the last of ``tokens`` tokens of a request sees (a window or a chunk bounds
+        what a layer reads)."""
+        return sum(need.kv_heads * (need.head_dim + (0 if need.values_are_keys else need.value_dim)) * element_bytes
+                   * (tokens - need.first_needed(tokens - 1))
+                   for entry, _ in self.cache_needs() for need in flat_needs(entry) if isinstance(need, PagedKV))
+
     def state_bytes_per_request(self) -> int:
         """Bytes of fixed-size state one request holds beside its pages."""
         return sum(need.numel * torch.empty((), dtype=need.dtype).element_size()

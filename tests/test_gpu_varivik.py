@@ -254,7 +254,8 @@ def test_values_blended_with_the_first_layers(dtype):
 
 KERNEL_CASES = [  # heads, kv heads, key size, value size, page, reach
     (8, 2, 128, 128, 16, -300), (4, 4, 64, 64, 16, -128), (6, 2, 128, 64, 32, -200), (8, 1, 64, 128, 16, -70), (4, 2, 64, 64, 64, 150),
-    (28, 4, 128, 128, 16, 260), (2, 1, 128, 64, 256, -333), (4, 2, 64, 64, 16, 0), (5, 5, 128, 64, 8, -1000)]
+    (28, 4, 128, 128, 16, 260), (2, 1, 128, 64, 256, -333), (4, 2, 64, 64, 16, 0), (5, 5, 128, 64, 8, -1000), (8, 2, 64, 32, 16, -200),
+    (3, 1, 128, 32, 16, -90), (4, 4, 64, 32, 32, 0)]
 
 
 @pytest.mark.parametrize("case", KERNEL_CASES)
