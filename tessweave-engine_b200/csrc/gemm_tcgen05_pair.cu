@@ -93,7 +93,18 @@ __device__ __forceinline__ uint32_t instr_desc_pair() {
 // One accumulator row of 16 columns, biased, activated and written the way `ep` and `out_mode` say.
 __device__ __forceinline__ void store_chunk(uint32_t (&v)[16], void* out, int out_mode, int out_stride, int row, int col,
                                             int rows_b, const TwEpilogue& ep) {
-    if (ep.bias) {
+    if (ep.bias && col + 16 <= rows_b && (reinterpret_cast<uintptr_t>(ep.bias + col) & 15) == 0) {
+        uint4 raw[2];           // the same sixteen values for every row: two loads, answered by L1
+        raw[0] = __ldg(reinterpret_cast<const uint4*>(ep.bias + col));
+        raw[1] = __ldg(reinterpret_cast<const uint4*>(ep.bias + col) + 1);
+        const __nv_bfloat162* b2 = reinterpret_cast<const __nv_bfloat162*>(raw);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const float2 f = __bfloat1622float2(b2[j]);
+            v[2 * j] = __float_as_uint(__uint_as_float(v[2 * j]) + f.x);
+            v[2 * j + 1] = __float_as_uint(__uint_as_float(v[2 * j + 1]) + f.y);
+        }
+    } else if (ep.bias) {
 #pragma unroll
         for (int j = 0; j < 16; ++j)
             if (col + j < rows_b) v[j] = __float_as_uint(__uint_as_float(v[j]) + __bfloat162float(ep.bias[col + j]));
