@@ -44,7 +44,8 @@ template <int BN> struct Config {
 };
 
 // Item i of the kernel: weight rows 128 (i / ksplit) .., k from (i % ksplit) * kper.
-template <int BN>
+// EPI: the sums get a bias or an activation other than SiLU on gates (kept apart from the plain form's epilogue).
+template <int BN, bool EPI>
 __global__ void __launch_bounds__(THREADS)
 gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, int n_rows,
                    int m_tokens, int K, int kper, int ksplit, void* __restrict__ out, int out_mode, int out_stride,
@@ -152,7 +153,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
             if (!ok) break;
             tc_fence_after();
             const int row = (item / ksplit) * BM + quarter * 32 + lane;          // weight row = output feature
-            const float row_bias = ep.bias && slice == 0 && row < n_rows ? __bfloat162float(ep.bias[row]) : 0.f;
+            const float row_bias = EPI && ep.bias && slice == 0 && row < n_rows ? __bfloat162float(ep.bias[row]) : 0.f;
 #pragma unroll 1
             for (int c0 = 0; c0 < BN; c0 += 16) {
                 if (c0 >= m_tokens) break;
@@ -162,12 +163,12 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                     // rows 16 g .. 16 g + 7 are gates, the eight after them their ups: lane l < 8 (mod 16) takes the up from lane l + 8
 #pragma unroll
                     for (int j = 0; j < 16; ++j) {
-                        const float gt = __uint_as_float(v[j]) + row_bias;
+                        const float gt = EPI ? __uint_as_float(v[j]) + row_bias : __uint_as_float(v[j]);
                         const float up = __shfl_down_sync(0xffffffffu, gt, 8);
                         const int tok = c0 + j;
                         if ((lane & 8) == 0 && row < n_rows && tok < m_tokens)
                             reinterpret_cast<bf16*>(out)[(size_t)tok * out_stride + (row >> 4) * 8 + (lane & 7)] =
-                                __float2bfloat16_rn(tw_activate(gt, ep.act) * up);
+                                __float2bfloat16_rn(tw_activate(gt, EPI ? ep.act : (int)TW_ACT_SILU) * up);
                     }
                     continue;
                 }
@@ -176,8 +177,11 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
                 for (int j = 0; j < 16; ++j) {
                     const int tok = c0 + j;
                     if (tok >= m_tokens) break;
-                    float f = __uint_as_float(v[j]) + row_bias;
-                    if (out_mode != OUT_PARTIAL) f = tw_activate(f, ep.act);
+                    float f = __uint_as_float(v[j]);
+                    if constexpr (EPI) {
+                        f += row_bias;
+                        if (out_mode != OUT_PARTIAL) f = tw_activate(f, ep.act);
+                    }
                     if (out_mode == OUT_BF16)
                         reinterpret_cast<bf16*>(out)[(size_t)tok * out_stride + row] = __float2bfloat16_rn(f);
                     else if (out_mode == OUT_F32)
@@ -203,14 +207,17 @@ int launch(const void* w, int n, const void* x, int m, int K, int kper, int kspl
     using C = Config<BN>;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+        cudaError_t e = cudaFuncSetAttribute(gemm_stream_kernel<BN, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+        if (e != cudaSuccess) return (int)e;
+        e = cudaFuncSetAttribute(gemm_stream_kernel<BN, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
         if (e != cudaSuccess) return (int)e;
         attr_set = true;
     }
+    const bool epi = ep.bias || ep.act != ((out_mode & ~OUT_EARLY_DEPENDENTS) == OUT_GATED ? TW_ACT_SILU : TW_ACT_NONE);
     CUtensorMap mw, mx;
     if (int e = get_map(w, n, K, BM, &mw)) return e;
     if (int e = get_map(x, m, K, BN, &mx)) return e;
-    return tw_launch(gemm_stream_kernel<BN>, dim3(blocks), dim3(THREADS), (size_t)C::SMEM, stream, 1, mw, mx, n, m, K, kper, ksplit,
+    return tw_launch(epi ? gemm_stream_kernel<BN, true> : gemm_stream_kernel<BN, false>, dim3(blocks), dim3(THREADS), (size_t)C::SMEM, stream, 1, mw, mx, n, m, K, kper, ksplit,
                      out, out_mode, out_stride, ep, status, next_weights, next_bytes);
 }
 
