@@ -75,14 +75,65 @@ TW_EXPORT int tw_embed(void* resid, const void* table, const int* ids, const int
 // The delta is either a dense tensor of the activation type or `nsplit` fp32 slices of a
 // split matrix product ([slice][row][hidden], slices `split_stride` floats apart), which
 // are added here in slice order.
+//
+// PAIR: a layer whose two sub-layers read the same stream through norms of their own.  Two deltas join the stream in one
+// sum, v = resid + delta_scale * (delta + pair.delta) (either may be absent), and the normalised rows leave twice, each
+// time with a weight of its own (pair.out may be null: one result).
+template <typename T> struct TwNormPair {
+    const T* delta;
+    const float* partial; int nsplit; size_t split_stride;
+    const float* weight;
+    T* out;
+};
+// The sum of a split product's slices at one element, in the order every consumer uses: whole groups of four into four
+// sums by slice mod 4, the rest into the first, then (s0 + s1) + (s2 + s3).
+__device__ __forceinline__ float tw_slices_at(const float* __restrict__ ps, int nsplit, size_t split_stride, int i) {
+    float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+    int k = 0;
+    for (; k + 4 <= nsplit; k += 4) {
+        s0 += ps[(size_t)k * split_stride + i];
+        s1 += ps[(size_t)(k + 1) * split_stride + i];
+        s2 += ps[(size_t)(k + 2) * split_stride + i];
+        s3 += ps[(size_t)(k + 3) * split_stride + i];
+    }
+    for (; k < nsplit; ++k) s0 += ps[(size_t)k * split_stride + i];
+    return (s0 + s1) + (s2 + s3);
+}
+// The same for a kernel that is nothing but latency: the first sixteen slices are loaded before anything is added, so
+// that they are one round trip to L2 and not one per group.
+__device__ __forceinline__ float tw_slices_ahead_at(const float* __restrict__ ps, int nsplit, size_t split_stride, int i) {
+    float t[16];
+#pragma unroll
+    for (int u = 0; u < 16; ++u) t[u] = u < nsplit ? ps[(size_t)u * split_stride + i] : 0.f;
+    const int full = nsplit & ~3;
+    float sum[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int u = 0; u < 16; ++u) {
+        if (u < full) sum[u & 3] += t[u];
+    }
+    int k = 16;
+    for (; k + 4 <= nsplit; k += 4) {
+        sum[0] += ps[(size_t)k * split_stride + i];
+        sum[1] += ps[(size_t)(k + 1) * split_stride + i];
+        sum[2] += ps[(size_t)(k + 2) * split_stride + i];
+        sum[3] += ps[(size_t)(k + 3) * split_stride + i];
+    }
+#pragma unroll
+    for (int u = 0; u < 16; ++u) {
+        if (u >= full && u < nsplit) sum[0] += t[u];
+    }
+    for (k = max(k, full); k < nsplit; ++k) sum[0] += ps[(size_t)k * split_stride + i];
+    return (sum[0] + sum[1]) + (sum[2] + sum[3]);
+}
 #define TW_NORM_THREADS 512
 #define TW_NORM_MAXV 16          // values a thread keeps in registers: rows up to 512 * 16 wide take the one-pass path
 
-template <typename T, bool ONE_PASS>
+template <typename T, bool ONE_PASS, bool PAIR>
 __global__ void __launch_bounds__(TW_NORM_THREADS)
 add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __restrict__ delta,
                    const float* __restrict__ partial, int nsplit, size_t split_stride,
-                   const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale) {
+                   const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale,
+                   TwNormPair<T> pair) {
     __shared__ float scratch[33];
     const int r = blockIdx.x;
     TW_TIMELINE_SCOPE(TW_K_NORM);
@@ -93,20 +144,15 @@ add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __re
     float* x = resid + (size_t)src * hidden;
     const T* d = delta ? delta + (size_t)src * hidden : nullptr;
     const float* ps = partial ? partial + (size_t)src * hidden : nullptr;
-    const bool has_delta = d || ps;
+    const T* d2 = PAIR && pair.delta ? pair.delta + (size_t)src * hidden : nullptr;
+    const float* ps2 = PAIR && pair.partial ? pair.partial + (size_t)src * hidden : nullptr;
+    const bool has_delta = d || ps || d2 || ps2;
     auto delta_at = [&](int i) -> float {
-        if (d) return tw_to_float(d[i]) * dscale;
-        float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;      // fixed order: ((s0 + s1) + (s2 + s3)) over interleaved slices
-        int k = 0;
-        for (; k + 4 <= nsplit; k += 4) {
-            s0 += ps[(size_t)k * split_stride + i];
-            s1 += ps[(size_t)(k + 1) * split_stride + i];
-            s2 += ps[(size_t)(k + 2) * split_stride + i];
-            s3 += ps[(size_t)(k + 3) * split_stride + i];
-        }
-        for (; k < nsplit; ++k) s0 += ps[(size_t)k * split_stride + i];
-        return ((s0 + s1) + (s2 + s3)) * dscale;
+        float v = d ? tw_to_float(d[i]) : (ps ? tw_slices_at(ps, nsplit, split_stride, i) : 0.f);
+        if (PAIR) v += d2 ? tw_to_float(d2[i]) : (ps2 ? tw_slices_at(ps2, pair.nsplit, pair.split_stride, i) : 0.f);
+        return v * dscale;
     };
+    T* o2 = PAIR && pair.out ? pair.out + (size_t)r * hidden : nullptr;
     T* o = out + (size_t)r * hidden;
     if (ONE_PASS) {
         float v[TW_NORM_MAXV];
@@ -127,7 +173,10 @@ add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __re
 #pragma unroll
         for (int j = 0; j < TW_NORM_MAXV; ++j) {
             const int i = threadIdx.x + j * TW_NORM_THREADS;
-            if (i < hidden) o[i] = tw_from_float<T>((v[j] * inv) * weight[i]);
+            if (i < hidden) {
+                o[i] = tw_from_float<T>((v[j] * inv) * weight[i]);
+                if (PAIR && o2) o2[i] = tw_from_float<T>((v[j] * inv) * pair.weight[i]);
+            }
         }
     } else {
         float ss = 0.f;
@@ -143,6 +192,7 @@ add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __re
             float v = x[i];
             if (rows && has_delta) v += delta_at(i);
             o[i] = tw_from_float<T>((v * inv) * weight[i]);
+            if (PAIR && o2) o2[i] = tw_from_float<T>((v * inv) * pair.weight[i]);
         }
     }
 }
@@ -155,11 +205,12 @@ add_rmsnorm_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __re
 #define TW_NORM_CTHREADS 256
 #define TW_NORM_CMAXV 4
 
-template <typename T>
+template <typename T, bool PAIR>
 __global__ void __launch_bounds__(TW_NORM_CTHREADS)
 add_rmsnorm_cluster_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __restrict__ delta,
                            const float* __restrict__ partial, int nsplit, size_t split_stride,
-                           const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale) {
+                           const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale,
+                           TwNormPair<T> pair) {
     __shared__ float scratch[33];
     __shared__ float all_ss[TW_NORM_CLUSTER];      // every block's sum of squares, written here by the blocks themselves
     TW_TIMELINE_SCOPE(TW_K_NORM_CLUSTER);
@@ -171,11 +222,12 @@ add_rmsnorm_cluster_kernel(T* __restrict__ out, float* __restrict__ resid, const
     const int src = rows ? rows[r] : r;
     const int chunk = (hidden + TW_NORM_CLUSTER - 1) / TW_NORM_CLUSTER;
     const int c0 = rank * chunk, c1 = min(hidden, c0 + chunk);
-    float wv[TW_NORM_CMAXV];
+    float wv[TW_NORM_CMAXV], wv2[PAIR ? TW_NORM_CMAXV : 1];
 #pragma unroll
     for (int j = 0; j < TW_NORM_CMAXV; ++j) {
         const int i = c0 + threadIdx.x + j * TW_NORM_CTHREADS;
         wv[j] = i < c1 ? weight[i] : 0.f;
+        if constexpr (PAIR) wv2[j] = i < c1 && pair.out ? pair.weight[i] : 0.f;
     }
     tw_grid_wait();
     TW_TIMELINE_MARK();
@@ -183,7 +235,9 @@ add_rmsnorm_cluster_kernel(T* __restrict__ out, float* __restrict__ resid, const
     float* x = resid + (size_t)src * hidden;
     const T* d = delta ? delta + (size_t)src * hidden : nullptr;
     const float* ps = partial ? partial + (size_t)src * hidden : nullptr;
-    const bool has_delta = d || ps;
+    const T* d2 = PAIR && pair.delta ? pair.delta + (size_t)src * hidden : nullptr;
+    const float* ps2 = PAIR && pair.partial ? pair.partial + (size_t)src * hidden : nullptr;
+    const bool has_delta = d || ps || d2 || ps2;
     float v[TW_NORM_CMAXV];
     float ss = 0.f;
 #pragma unroll
@@ -191,37 +245,8 @@ add_rmsnorm_cluster_kernel(T* __restrict__ out, float* __restrict__ resid, const
         const int i = c0 + threadIdx.x + j * TW_NORM_CTHREADS;
         v[j] = 0.f;
         if (i < c1) {
-            float dv = 0.f;
-            if (d) {
-                dv = tw_to_float(d[i]);
-            } else if (ps) {
-                // The slices are summed in the order every consumer of a split product uses: whole groups of
-                // four into four sums by k mod 4, the rest into the first, then (s0 + s1) + (s2 + s3).  The
-                // first sixteen are loaded before anything is added, so that they are one round trip to L2
-                // and not one per group (this kernel is nothing but latency).
-                float t[16];
-#pragma unroll
-                for (int u = 0; u < 16; ++u) t[u] = u < nsplit ? ps[(size_t)u * split_stride + i] : 0.f;
-                const int full = nsplit & ~3;
-                float sum[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-                for (int u = 0; u < 16; ++u) {
-                    if (u < full) sum[u & 3] += t[u];
-                }
-                int k = 16;
-                for (; k + 4 <= nsplit; k += 4) {
-                    sum[0] += ps[(size_t)k * split_stride + i];
-                    sum[1] += ps[(size_t)(k + 1) * split_stride + i];
-                    sum[2] += ps[(size_t)(k + 2) * split_stride + i];
-                    sum[3] += ps[(size_t)(k + 3) * split_stride + i];
-                }
-#pragma unroll
-                for (int u = 0; u < 16; ++u) {
-                    if (u >= full && u < nsplit) sum[0] += t[u];
-                }
-                for (k = max(k, full); k < nsplit; ++k) sum[0] += ps[(size_t)k * split_stride + i];
-                dv = (sum[0] + sum[1]) + (sum[2] + sum[3]);
-            }
+            float dv = d ? tw_to_float(d[i]) : (ps ? tw_slices_ahead_at(ps, nsplit, split_stride, i) : 0.f);
+            if constexpr (PAIR) dv += d2 ? tw_to_float(d2[i]) : (ps2 ? tw_slices_ahead_at(ps2, pair.nsplit, pair.split_stride, i) : 0.f);
             v[j] = x[i] + dv * dscale;
             if (!rows && has_delta) x[i] = v[j];
             ss += v[j] * v[j];
@@ -240,7 +265,12 @@ add_rmsnorm_cluster_kernel(T* __restrict__ out, float* __restrict__ resid, const
 #pragma unroll
     for (int j = 0; j < TW_NORM_CMAXV; ++j) {
         const int i = c0 + threadIdx.x + j * TW_NORM_CTHREADS;
-        if (i < c1) o[i] = tw_from_float<T>((v[j] * inv) * wv[j]);
+        if (i < c1) {
+            o[i] = tw_from_float<T>((v[j] * inv) * wv[j]);
+            if constexpr (PAIR) {
+                if (pair.out) pair.out[(size_t)r * hidden + i] = tw_from_float<T>((v[j] * inv) * wv2[j]);
+            }
+        }
     }
 }
 
@@ -263,10 +293,11 @@ __device__ __forceinline__ void tw_store4(__nv_bfloat16* p, float4 v) {
 // Dense delta only; hidden a multiple of 4 and at most 4 * 256 * V4 wide.  V4 = float4 per thread: 4 for rows up
 // to 4,096 wide (half the registers, twice the blocks per SM), 8 up to 8,192.
 #define TW_NORM_V4 8
-template <typename T, int V4>
+template <typename T, int V4, bool PAIR>
 __global__ void __launch_bounds__(256)
 add_rmsnorm_vec4_kernel(T* __restrict__ out, float* __restrict__ resid, const T* __restrict__ delta,
-                        const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale) {
+                        const float* __restrict__ weight, float eps, int hidden, const int* __restrict__ rows, float dscale,
+                        TwNormPair<T> pair) {
     __shared__ float scratch[33];
     TW_TIMELINE_SCOPE(TW_K_NORM);
     tw_grid_wait();
@@ -284,8 +315,14 @@ add_rmsnorm_vec4_kernel(T* __restrict__ out, float* __restrict__ resid, const T*
         v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (i < n4) {
             v[j] = x4[i];
-            if (delta) {
-                const float4 d = tw_load4(delta + (size_t)src * hidden + 4 * i);
+            if (delta || (PAIR && pair.delta)) {
+                float4 d = delta ? tw_load4(delta + (size_t)src * hidden + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                if constexpr (PAIR) {
+                    if (pair.delta) {
+                        const float4 e = tw_load4(pair.delta + (size_t)src * hidden + 4 * i);
+                        d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
+                    }
+                }
                 v[j].x += d.x * dscale; v[j].y += d.y * dscale; v[j].z += d.z * dscale; v[j].w += d.w * dscale;
                 if (!rows) x4[i] = v[j];
             }
@@ -302,33 +339,40 @@ add_rmsnorm_vec4_kernel(T* __restrict__ out, float* __restrict__ resid, const T*
             const float4 w = w4[i];
             tw_store4(out + (size_t)r * hidden + 4 * i,
                       make_float4((v[j].x * inv) * w.x, (v[j].y * inv) * w.y, (v[j].z * inv) * w.z, (v[j].w * inv) * w.w));
+            if constexpr (PAIR) {
+                if (pair.out) {
+                    const float4 u = reinterpret_cast<const float4*>(pair.weight)[i];
+                    tw_store4(pair.out + (size_t)r * hidden + 4 * i,
+                              make_float4((v[j].x * inv) * u.x, (v[j].y * inv) * u.y, (v[j].z * inv) * u.z, (v[j].w * inv) * u.w));
+                }
+            }
         }
     }
 }
 
-template <typename T>
+template <typename T, bool PAIR>
 static int launch_add_rmsnorm(T* out, float* resid, const T* delta, const float* partial, int nsplit,
                               size_t split_stride, const float* weight, float eps, int n_rows, int hidden,
-                              const int* rows, float dscale, cudaStream_t stream) {
+                              const int* rows, float dscale, TwNormPair<T> pair, cudaStream_t stream) {
     if (n_rows <= 64 && hidden >= 1024 && hidden <= TW_NORM_CLUSTER * TW_NORM_CTHREADS * TW_NORM_CMAXV) {
-        return tw_launch(add_rmsnorm_cluster_kernel<T>, dim3(n_rows * TW_NORM_CLUSTER), dim3(TW_NORM_CTHREADS), 0, stream,
-                         TW_NORM_CLUSTER, out, resid, delta, partial, nsplit, split_stride, weight, eps, hidden, rows, dscale);
+        return tw_launch(add_rmsnorm_cluster_kernel<T, PAIR>, dim3(n_rows * TW_NORM_CLUSTER), dim3(TW_NORM_CTHREADS), 0, stream,
+                         TW_NORM_CLUSTER, out, resid, delta, partial, nsplit, split_stride, weight, eps, hidden, rows, dscale, pair);
     }
-    if (!partial && (hidden & 3) == 0 && hidden <= 4 * 256 * TW_NORM_V4) {
+    if (!partial && !(PAIR && pair.partial) && (hidden & 3) == 0 && hidden <= 4 * 256 * TW_NORM_V4) {
         if (hidden <= 4 * 256 * 4)
-            tw_launch(add_rmsnorm_vec4_kernel<T, 4>, dim3(n_rows), dim3(256), 0, stream, 1, out, resid, delta, weight, eps,
-                      hidden, rows, dscale);
+            tw_launch(add_rmsnorm_vec4_kernel<T, 4, PAIR>, dim3(n_rows), dim3(256), 0, stream, 1, out, resid, delta, weight, eps,
+                      hidden, rows, dscale, pair);
         else
-            tw_launch(add_rmsnorm_vec4_kernel<T, TW_NORM_V4>, dim3(n_rows), dim3(256), 0, stream, 1, out, resid, delta, weight,
-                      eps, hidden, rows, dscale);
+            tw_launch(add_rmsnorm_vec4_kernel<T, TW_NORM_V4, PAIR>, dim3(n_rows), dim3(256), 0, stream, 1, out, resid, delta, weight,
+                      eps, hidden, rows, dscale, pair);
         return TW_LAUNCH_CHECK();
     }
     if (hidden <= TW_NORM_THREADS * TW_NORM_MAXV)
-        tw_launch(add_rmsnorm_kernel<T, true>, dim3(n_rows), dim3(TW_NORM_THREADS), 0, stream, 1, out, resid, delta, partial, nsplit,
-                                                                            split_stride, weight, eps, hidden, rows, dscale);
+        tw_launch(add_rmsnorm_kernel<T, true, PAIR>, dim3(n_rows), dim3(TW_NORM_THREADS), 0, stream, 1, out, resid, delta, partial,
+                  nsplit, split_stride, weight, eps, hidden, rows, dscale, pair);
     else
-        tw_launch(add_rmsnorm_kernel<T, false>, dim3(n_rows), dim3(TW_NORM_THREADS), 0, stream, 1, out, resid, delta, partial, nsplit,
-                                                                             split_stride, weight, eps, hidden, rows, dscale);
+        tw_launch(add_rmsnorm_kernel<T, false, PAIR>, dim3(n_rows), dim3(TW_NORM_THREADS), 0, stream, 1, out, resid, delta, partial,
+                  nsplit, split_stride, weight, eps, hidden, rows, dscale, pair);
     return TW_LAUNCH_CHECK();
 }
 
@@ -338,10 +382,30 @@ TW_EXPORT int tw_add_rmsnorm(void* out, float* resid, const void* delta, const f
     if (n_rows <= 0) return 0;
     if (delta && partial) return (int)cudaErrorInvalidValue;
     if (dtype == TW_F32)
-        return launch_add_rmsnorm<float>((float*)out, resid, (const float*)delta, partial, nsplit, (size_t)split_stride,
-                                         weight, eps, n_rows, hidden, rows, delta_scale, stream);
-    return launch_add_rmsnorm<__nv_bfloat16>((__nv_bfloat16*)out, resid, (const __nv_bfloat16*)delta, partial, nsplit,
-                                             (size_t)split_stride, weight, eps, n_rows, hidden, rows, delta_scale, stream);
+        return launch_add_rmsnorm<float, false>((float*)out, resid, (const float*)delta, partial, nsplit, (size_t)split_stride,
+                                                weight, eps, n_rows, hidden, rows, delta_scale, TwNormPair<float>{}, stream);
+    return launch_add_rmsnorm<__nv_bfloat16, false>((__nv_bfloat16*)out, resid, (const __nv_bfloat16*)delta, partial, nsplit,
+                                                    (size_t)split_stride, weight, eps, n_rows, hidden, rows, delta_scale,
+                                                    TwNormPair<__nv_bfloat16>{}, stream);
+}
+
+// Two deltas in, two normalised copies out (see PAIR above); of each pair the second, or both deltas, may be absent.
+TW_EXPORT int tw_add_rmsnorm_pair(void* out, void* out2, float* resid, const void* delta, const float* partial, int nsplit,
+                                  long split_stride, const void* delta2, const float* partial2, int nsplit2, long split_stride2,
+                                  const float* weight, const float* weight2, float eps, int n_rows, int hidden, const int* rows,
+                                  float delta_scale, int dtype, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if ((delta && partial) || (delta2 && partial2) || (out2 && !weight2)) return (int)cudaErrorInvalidValue;
+    if (dtype == TW_F32)
+        return launch_add_rmsnorm<float, true>((float*)out, resid, (const float*)delta, partial, nsplit, (size_t)split_stride,
+                                               weight, eps, n_rows, hidden, rows, delta_scale,
+                                               TwNormPair<float>{(const float*)delta2, partial2, nsplit2, (size_t)split_stride2,
+                                                                 weight2, (float*)out2}, stream);
+    return launch_add_rmsnorm<__nv_bfloat16, true>(
+        (__nv_bfloat16*)out, resid, (const __nv_bfloat16*)delta, partial, nsplit, (size_t)split_stride, weight, eps, n_rows, hidden,
+        rows, delta_scale,
+        TwNormPair<__nv_bfloat16>{(const __nv_bfloat16*)delta2, partial2, nsplit2, (size_t)split_stride2, weight2, (__nv_bfloat16*)out2},
+        stream);
 }
 
 // ---------------------------------------------------------------------------
@@ -850,21 +914,23 @@ TW_EXPORT int tw_gate_mul(void* out, int out_stride, const void* x, int x_stride
 }
 
 // ---------------------------------------------------------------------------
-// Soft cap of fp32 logits in place: x <- cap * tanh(x / cap).
+// fp32 logits in place: x <- scale * x, then, with cap > 0, x <- cap * tanh(x / cap).
 // ---------------------------------------------------------------------------
-__global__ void softcap_kernel(float* __restrict__ x, long total, float cap) {
+__global__ void softcap_kernel(float* __restrict__ x, long total, float scale, float cap) {
     tw_grid_wait();
     tw_grid_launch_dependents();
     long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
     const long step = (long)gridDim.x * blockDim.x;
-    for (; idx < total; idx += step) x[idx] = cap * tanhf(x[idx] / cap);
+    for (; idx < total; idx += step) {
+        const float v = x[idx] * scale;
+        x[idx] = cap > 0.f ? cap * tanhf(v / cap) : v;
+    }
 }
 
-TW_EXPORT int tw_softcap(float* x, long long total, float cap, cudaStream_t stream) {
+TW_EXPORT int tw_softcap(float* x, long long total, float scale, float cap, cudaStream_t stream) {
     if (total <= 0) return 0;
-    if (!(cap > 0.f)) return (int)cudaErrorInvalidValue;
     const int blocks = (int)((total + 255) / 256 < 1184 ? (total + 255) / 256 : 1184);
-    return tw_launch(softcap_kernel, dim3(blocks), dim3(256), 0, stream, 1, x, (long)total, cap);
+    return tw_launch(softcap_kernel, dim3(blocks), dim3(256), 0, stream, 1, x, (long)total, scale, cap);
 }
 
 // ---------------------------------------------------------------------------
@@ -1146,7 +1212,8 @@ TW_EXPORT int tw_kv_store(const void* rows, int stride, int k_col, int v_col, co
 //   2. rotation by position of `rot_dims` values from column `rot_col` on (one span that all heads share, outside
 //      the normalised spans; pairs of neighbours or of halves), cos and sin multiplied by `magnitude`;
 //   3. the store of the key columns (from `k_col`) and, where the values have pages of their own, of the value
-//      columns (from `v_col`) into the token's place in its request's pages.
+//      columns (from `v_col`) into the token's place in its request's pages;
+//   4. gate_out[row, j] = sigmoid(value at gate_col + j) in fp32, j < gate_heads (a gate per head for the attention kernels).
 // Serves attention with normalised heads (spans: the query heads, the key heads; no rotation) and attention over
 // low-rank latents (spans: the query latent, the key/value latent; the shared rotated key part; one set of pages).
 // Everything between the loads and the stores is fp32; what is stored is what the rows hold afterwards, bit for bit.
@@ -1159,7 +1226,7 @@ norm_rotate_store_kernel(T* __restrict__ rows, int row_stride, NormSpans sp, T* 
                          int k_col, int v_col, const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                          const int* __restrict__ seq_slot, const int* __restrict__ block_table, int table_stride,
                          T* __restrict__ k_cache, T* __restrict__ v_cache, int Hkv, int Dk, int Dv, int page_size, int num_pages,
-                         int write_cache, int* status) {
+                         int write_cache, int gate_col, int gate_heads, float* __restrict__ gate_out, int* status) {
     tw_grid_wait();
     tw_grid_launch_dependents();
     const int n = blockIdx.x;
@@ -1275,6 +1342,8 @@ norm_rotate_store_kernel(T* __restrict__ rows, int row_stride, NormSpans sp, T* 
         row[a] = tw_from_float<T>(u * cs - v * sn);
         row[b] = tw_from_float<T>(v * cs + u * sn);
     }
+    for (int i = (int)blockDim.x - 1 - (int)threadIdx.x; i < gate_heads; i += blockDim.x)       // (from the threads the rotation left idle)
+        gate_out[(size_t)n * gate_heads + i] = 1.0f / (1.0f + expf(-tw_to_float(row[gate_col + i])));
     if (!write_cache) return;
     __syncthreads();            // the block's own writes to the row are visible to all of its threads from here on
     if (page < 0 || page >= num_pages) {
@@ -1315,8 +1384,10 @@ TW_EXPORT int tw_norm_rotate_store(void* rows, int row_stride, int n_tokens, int
                                    int rot_col, int rot_dims, const float* inv_freq, int interleaved, float magnitude, int k_col,
                                    int v_col, const int* positions, const int* seq_of_token, const int* seq_slot,
                                    const int* block_table, int table_stride, void* k_cache, void* v_cache, int Hkv, int Dk, int Dv,
-                                   int page_size, int num_pages, int write_cache, int dtype, int* status, cudaStream_t stream) {
+                                   int page_size, int num_pages, int write_cache, int gate_col, int gate_heads, float* gate_out, int dtype,
+                                   int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (gate_heads < 0 || (gate_heads && !gate_out)) return (int)cudaErrorInvalidValue;
     if (spans < 0 || spans > 2 || (spans >= 1 && (heads0 <= 0 || dim0 <= 0 || !weight0)) || (spans == 2 && (heads1 <= 0 || dim1 <= 0 || !weight1))
         || rot_dims < 0 || (rot_dims & 1) || (rot_dims && !inv_freq) || (write_cache && !k_cache))
         return (int)cudaErrorInvalidValue;
@@ -1340,11 +1411,11 @@ TW_EXPORT int tw_norm_rotate_store(void* rows, int row_stride, int n_tokens, int
         return tw_launch(norm_rotate_store_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, 1, (float*)rows, row_stride, sp,
                          (float*)dst0, eps, block_wide, 0, rot_col, rot_dims, inv_freq, interleaved, magnitude, k_col, v_col, positions, seq_of_token,
                          seq_slot, block_table, table_stride, (float*)k_cache, (float*)v_cache, Hkv, Dk, Dv, page_size, num_pages,
-                         write_cache, status);
+                         write_cache, gate_col, gate_heads, gate_out, status);
     return tw_launch(norm_rotate_store_kernel<__nv_bfloat16>, dim3(n_tokens), dim3(threads), 0, stream, 1, (__nv_bfloat16*)rows,
                      row_stride, sp, (__nv_bfloat16*)dst0, eps, block_wide, vec16, rot_col, rot_dims, inv_freq, interleaved, magnitude, k_col, v_col,
                      positions, seq_of_token, seq_slot, block_table, table_stride, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache,
-                     Hkv, Dk, Dv, page_size, num_pages, write_cache, status);
+                     Hkv, Dk, Dv, page_size, num_pages, write_cache, gate_col, gate_heads, gate_out, status);
 }
 
 // ---------------------------------------------------------------------------

@@ -19,6 +19,9 @@
 //   TW_REC_GLA         S <- diag(a) S + k v^T                o = S^T q          (gated linear attention)
 //                      a = sigmoid(z + b)^(1 / tau) per key channel from the projected z, evaluated as
 //                      exp(logsigmoid(z + b) / tau); 1 / tau arrives in `cap`, b in p0
+//   TW_REC_SSD         S <- e^(-r_h dt) S + dt k v^T         o = S^T q + u_h v  (the state-space form of linear attention)
+//                      dt = softplus(d + b_h) per head from the projected d, r_h = e^(A_h); A in p0, b in p1, the skip u
+//                      in p2.  q, k and v arrive as fp32 rows (here: convolved and activated), heads may share q and k
 //
 // One block per (head, request, slice of the columns of S): a thread owns a column of S in registers (TW_DK
 // values, a compile-time size; where that size is a multiple of 16 four or eight lanes share a column, a quarter or
@@ -43,7 +46,7 @@
 // same bits.
 #define TW_REC_SHARES ((TW_DK % 32 == 0) ? 8 : ((TW_DK % 16 == 0) ? 4 : 1))
 
-enum : int { TW_REC_RETENTION = 0, TW_REC_WKV = 1, TW_REC_MLSTM = 2, TW_REC_DELTA = 3, TW_REC_GLA = 4 };
+enum : int { TW_REC_RETENTION = 0, TW_REC_WKV = 1, TW_REC_MLSTM = 2, TW_REC_DELTA = 3, TW_REC_GLA = 4, TW_REC_SSD = 5 };
 
 struct RecArgs {
     float* out;                 // [rows, H * Dv] fp32
@@ -51,9 +54,10 @@ struct RecArgs {
     const void* q; int q_stride;        // rows of q (r), k, v: element type T, column h * D + i inside each
     const void* k; int k_stride;
     const void* v; int v_stride;
-    const float* wpre; int wpre_stride; // wkv, gla: d [rows, H * Dk] fp32;  mlstm: [rows, 2 H] fp32 (pi | pf);  delta: d [rows, H * Dk] or [rows, H]
-    const float* p0;            // wkv: w0 [H * Dk];  gla: b [H * Dk];  retention: decay [H];  mlstm: bias [2 H];  delta: A [H] (log of the rate)
-    const float* p1;            // wkv: u [H * Dk];  delta: b [H * Dk] or [H]
+    const float* wpre; int wpre_stride; // wkv, gla: d [rows, H * Dk] fp32;  mlstm: [rows, 2 H] fp32 (pi | pf);  delta: d [rows, H * Dk] or [rows, H];  ssd: d [rows, H]
+    const float* p0;            // wkv: w0 [H * Dk];  gla: b [H * Dk];  retention: decay [H];  mlstm: bias [2 H];  delta, ssd: A [H] (log of the rate)
+    const float* p1;            // wkv: u [H * Dk];  delta: b [H * Dk] or [H];  ssd: b [H]
+    const float* p2;            // ssd: the skip [H]
     const float* bpre; int bpre_stride; // delta: the write strength's pre-activation [rows, H] fp32
     int channel_decay;          // delta: a decay per key channel (else one per head)
     int qk_group;               // value heads that share a head of q and k (1: every head has its own)
@@ -102,7 +106,7 @@ linear_recurrence_kernel(RecArgs a) {
     const bool live = walks && j < cols;
     // a staged chunk: q [C][DK], k [C][DK], w [C][DK] (wkv) or gates [C][2] (mlstm), v [C][per]; two of them, so that
     // the rows of the next 16 tokens are staged while the state walks through these
-    const int extra = (MODE == TW_REC_WKV || MODE == TW_REC_GLA) ? C * DKP : (MODE == TW_REC_MLSTM ? 2 * C : (MODE == TW_REC_DELTA ? C * DKP + 2 * C : 0));
+    const int extra = (MODE == TW_REC_WKV || MODE == TW_REC_GLA) ? C * DKP : ((MODE == TW_REC_MLSTM || MODE == TW_REC_SSD) ? 2 * C : (MODE == TW_REC_DELTA ? C * DKP + 2 * C : 0));
     const int chunk_floats = 2 * C * DKP + extra + C * per;
     float* su = sm + 2 * chunk_floats;      // [DKP] bonus (wkv)
     const long long head_state = (long long)DK * cols + (MODE == TW_REC_MLSTM ? 1 : 0);
@@ -112,8 +116,9 @@ linear_recurrence_kernel(RecArgs a) {
     const T* __restrict__ gv = (const T*)a.v;
     const int half = a.rot_dims >> 1;
     const int hq = h / a.qk_group;      // the head of q and k this head reads
-    const float rate = MODE == TW_REC_DELTA ? expf(a.p0[h]) : 0.f;     // delta: the head's decay rate
-    const bool vec_rows = MODE == TW_REC_DELTA && sizeof(T) == 4 && (a.q_stride % 4) == 0 && (a.k_stride % 4) == 0
+    const float rate = (MODE == TW_REC_DELTA || MODE == TW_REC_SSD) ? expf(a.p0[h]) : 0.f;     // the head's decay rate
+    const float skip = MODE == TW_REC_SSD ? a.p2[h] : 0.f;
+    const bool vec_rows = (MODE == TW_REC_DELTA || MODE == TW_REC_SSD) && sizeof(T) == 4 && (a.q_stride % 4) == 0 && (a.k_stride % 4) == 0
                           && (reinterpret_cast<size_t>(a.q) % 16) == 0 && (reinterpret_cast<size_t>(a.k) % 16) == 0
                           && (!a.channel_decay || ((a.wpre_stride % 4) == 0 && (reinterpret_cast<size_t>(a.wpre) % 16) == 0
                                                    && (reinterpret_cast<size_t>(a.p1) % 16) == 0));
@@ -150,7 +155,7 @@ linear_recurrence_kernel(RecArgs a) {
         const int first = MODE == TW_REC_RETENTION ? a.rot_dims : 0;     // channels from here on are not rotated
         const int plain = DK - first;
         bool staged = false;
-        if constexpr (MODE == TW_REC_DELTA && sizeof(T) == 4 && KS > 1) {
+        if constexpr ((MODE == TW_REC_DELTA || MODE == TW_REC_SSD) && sizeof(T) == 4 && KS > 1) {
             if (vec_rows) {
                 // fp32 rows whose heads start on 16-byte boundaries: four channels per load, and all of a thread's
                 // loads of the chunk are under way before the first is used
@@ -163,7 +168,7 @@ linear_recurrence_kernel(RecArgs a) {
                     float4 kk = *reinterpret_cast<const float4*>((const float*)gk + row * a.k_stride + hq * DK + i);
                     qq.x *= a.q_scale; qq.y *= a.q_scale; qq.z *= a.q_scale; qq.w *= a.q_scale;
                     kk.x *= a.k_scale; kk.y *= a.k_scale; kk.z *= a.k_scale; kk.w *= a.k_scale;
-                    if (a.channel_decay) {
+                    if (MODE == TW_REC_DELTA && a.channel_decay) {
                         const float4 dd = *reinterpret_cast<const float4*>(a.wpre + row * a.wpre_stride + h * DK + i);
                         const float4 bb = *reinterpret_cast<const float4*>(a.p1 + h * DK + i);
                         float4 ww;
@@ -242,6 +247,13 @@ linear_recurrence_kernel(RecArgs a) {
                 sg[C + t] = 1.0f / (1.0f + expf(-a.bpre[row * a.bpre_stride + h]));
             }
         }
+        if (MODE == TW_REC_SSD) {
+            for (int t = tid; t < ct; t += nthreads) {
+                const float dt = tw_softplus(a.wpre[(size_t)(start + t0 + t) * a.wpre_stride + h] + a.p1[h]);
+                sw[2 * t] = expf(-rate * dt);
+                sw[2 * t + 1] = dt;
+            }
+        }
         for (int e = tid; e < ct * per; e += nthreads) {     // the block's own columns of v
             const int t = e / per, c = blockIdx.z * per + (e - t * per);
             if (c < Dv) sv[e] = tw_to_float(gv[(size_t)(start + t0 + t) * a.v_stride + h * Dv + c]);
@@ -296,6 +308,10 @@ linear_recurrence_kernel(RecArgs a) {
                     fa = expf(lf + m - m_new);
                     fb = expf(li - m_new) * vj;
                     m = m_new;
+                }
+                if (MODE == TW_REC_SSD) {
+                    fa = sw[2 * t];
+                    fb = sw[2 * t + 1] * vj;
                 }
                 const float* w = sw + t * DKP + ks * SEG;
                 const float* u = su + ks * SEG;
@@ -453,7 +469,7 @@ linear_recurrence_kernel(RecArgs a) {
                     if (MODE == TW_REC_MLSTM && j == Dv)
                         a.den[row * a.H + h] = fmaxf(fabsf(acc), expf(-m)) + 1e-6f;
                     else
-                        a.out[row * ((size_t)a.H * Dv) + (size_t)h * Dv + j] = acc;
+                        a.out[row * ((size_t)a.H * Dv) + (size_t)h * Dv + j] = MODE == TW_REC_SSD ? acc + skip * vj : acc;
                 }
             }
         }
@@ -491,7 +507,7 @@ static int launch_split(const RecArgs& a, int n_seqs, bool long_portions, cudaSt
     b.cols_per_block = per;
     const size_t chunk = 2 * TW_REC_CHUNK * DKP + (size_t)TW_REC_CHUNK * per
                          + ((MODE == TW_REC_WKV || MODE == TW_REC_GLA) ? TW_REC_CHUNK * DKP
-                            : (MODE == TW_REC_MLSTM ? 2 * TW_REC_CHUNK : (MODE == TW_REC_DELTA ? TW_REC_CHUNK * DKP + 2 * TW_REC_CHUNK : 0)));
+                            : ((MODE == TW_REC_MLSTM || MODE == TW_REC_SSD) ? 2 * TW_REC_CHUNK : (MODE == TW_REC_DELTA ? TW_REC_CHUNK * DKP + 2 * TW_REC_CHUNK : 0)));
     const size_t smem = (2 * chunk + DKP) * sizeof(float);
     if (smem > 48 * 1024) {
         const cudaError_t e = cudaFuncSetAttribute(linear_recurrence_kernel<T, MODE, KS>,
@@ -513,7 +529,7 @@ static int launch_recurrence(const RecArgs& a, int n_seqs, bool long_portions, c
 
 TW_EXPORT int tw_linear_recurrence(int mode, float* out, float* den, const void* q, int q_stride, const void* k, int k_stride,
                                    const void* v, int v_stride, const float* wpre, int wpre_stride, const float* p0,
-                                   const float* p1, const float* bpre, int bpre_stride, int channel_decay, int qk_group,
+                                   const float* p1, const float* p2, const float* bpre, int bpre_stride, int channel_decay, int qk_group,
                                    const float* inv_freq, int rot_dims, float q_scale, float k_scale,
                                    float cap, float* state, long long state_stride, const void* tail_src, int tail_stride,
                                    int tail_width, long long tail_offset, const int* positions, const int* seq_slot,
@@ -526,7 +542,7 @@ TW_EXPORT int tw_linear_recurrence(int mode, float* out, float* den, const void*
     RecArgs a;
     a.bpre = bpre; a.bpre_stride = bpre_stride; a.channel_decay = channel_decay; a.qk_group = qk_group;
     a.out = out; a.den = den; a.q = q; a.q_stride = q_stride; a.k = k; a.k_stride = k_stride; a.v = v; a.v_stride = v_stride;
-    a.wpre = wpre; a.wpre_stride = wpre_stride; a.p0 = p0; a.p1 = p1; a.inv_freq = inv_freq; a.rot_dims = inv_freq ? rot_dims : 0;
+    a.wpre = wpre; a.wpre_stride = wpre_stride; a.p0 = p0; a.p1 = p1; a.p2 = p2; a.inv_freq = inv_freq; a.rot_dims = inv_freq ? rot_dims : 0;
     a.k_scale = k_scale; a.q_scale = q_scale; a.cap = cap; a.state = state; a.state_stride = state_stride;
     a.tail_src = tail_src; a.tail_stride = tail_stride; a.tail_width = tail_width; a.tail_offset = tail_offset;
     a.positions = positions; a.seq_slot = seq_slot; a.seq_q_start = seq_q_start; a.seq_q_len = seq_q_len;
@@ -550,6 +566,9 @@ TW_EXPORT int tw_linear_recurrence(int mode, float* out, float* den, const void*
     case TW_REC_DELTA:
         if (!f32 || !bpre || !wpre || !p0 || !p1) return (int)cudaErrorInvalidValue;     // its rows are prepared in fp32 in every run type
         return launch_recurrence<float, TW_REC_DELTA>(a, n_seqs, lp, stream);
+    case TW_REC_SSD:
+        if (!f32 || !wpre || !p0 || !p1 || !p2) return (int)cudaErrorInvalidValue;
+        return launch_recurrence<float, TW_REC_SSD>(a, n_seqs, lp, stream);
     }
     return (int)cudaErrorInvalidValue;
 }

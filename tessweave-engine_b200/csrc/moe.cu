@@ -6,7 +6,9 @@
 //                    softmax over those alone; optionally one more dot product per token, sigmoid(ws . h), the
 //                    gate of an expert that every token uses.  With `scoring` 1: s = softmax(z) over every router
 //                    output, the `top` largest s + correction are chosen, and their weights are s * weight_scale
-//                    (not renormalised)
+//                    (not renormalised); with `scoring` 2 their weights are s / (sum of the chosen s + 1e-20) * weight_scale.
+//                    With `group_count` > 0 the outputs form that many equal groups of neighbours; a group counts as much
+//                    as its best output, and only outputs of the best `group_keep` groups may be chosen
 //   tw_moe_gate_up   act[token, j] = silu(Wg_e h) * (Wu_e h)          e = the j-th expert of the token
 //                    with `act` 1: g = min(Wg_e h, limit), u = clamp(Wu_e h, -limit, limit), g sigmoid(alpha g) (u + 1)
 //   tw_moe_up        act[token, j] = f(Wu_e h) for experts without a gate, f one of the activations of common.cuh
@@ -104,8 +106,8 @@ __global__ void __launch_bounds__(512)
 moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, float* __restrict__ shared_gate,
                  const T* __restrict__ h, int h_stride, const T* __restrict__ wr, const float* __restrict__ br,
                  const T* __restrict__ ws, int width, int E, int top, int scoring, const float* __restrict__ correction,
-                 float weight_scale) {
-    extern __shared__ float sm[];           // [width] the row, [E + 1] logits, [E] marks
+                 float weight_scale, int group_count, int group_keep) {
+    extern __shared__ float sm[];           // [width] the row, [E + 1] logits, [E] marks, [2 group_count]
     tw_grid_wait();
     tw_grid_launch_dependents();
     const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -119,31 +121,79 @@ moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, float* __
         if (lane == 0) z[e] = e < E ? d + (br ? br[e] : 0.f) : d;
     }
     __syncthreads();
-    if (threadIdx.x != 0) return;
-    if (ws && shared_gate) shared_gate[row] = 1.0f / (1.0f + expf(-z[E]));
-    // selection: `top` times the largest logit that is left; a row of NaN still names `top` different experts
+    if (warp != 0) return;
+    if (lane == 0 && ws && shared_gate) shared_gate[row] = 1.0f / (1.0f + expf(-z[E]));
     float* taken = z + E + 1;
-    for (int e = 0; e < E; ++e) taken[e] = 0.f;
-    if (scoring == 1) {
-        // scores over every output; the choice looks at score + correction, the weight is the plain score
+    if (scoring != 0) {
+        // scores over every output; the choice looks at score + correction, the weight is the plain score.  One warp: lane l
+        // holds outputs l, l + 32, ...; a choice is the largest value, the lowest index where values are equal
         float top_z = -INFINITY, den = 0.f;
-        for (int e = 0; e < E; ++e) top_z = fmaxf(top_z, z[e]);
-        for (int e = 0; e < E; ++e) { z[e] = expf(z[e] - top_z); den += z[e]; }
-        for (int e = 0; e < E; ++e) z[e] /= den;
-        for (int j = 0; j < top; ++j) {
-            int arg = -1;
+        for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, z[e]);
+        top_z = tw_warp_max(top_z);
+        for (int e = lane; e < E; e += 32) { z[e] = expf(z[e] - top_z); den += z[e]; }
+        den = tw_warp_sum(den);
+        for (int e = lane; e < E; e += 32) {
+            z[e] /= den;
+            taken[e] = group_count > 0 ? 1.f : 0.f;
+        }
+        __syncwarp();
+        // the largest of n values that are not marked in `mark`, by (value, lowest index); a row of NaN still names an index
+        auto pick = [&](int n, auto value, auto marked) -> int {
             float best = -INFINITY;
-            for (int e = 0; e < E; ++e) {
-                if (taken[e] != 0.f) continue;
-                const float c = z[e] + (correction ? correction[e] : 0.f);
+            int arg = -1;
+            for (int e = lane; e < n; e += 32) {
+                if (marked(e)) continue;
+                const float c = value(e);
                 if (arg < 0 || c > best) { arg = e; best = c; }
             }
-            taken[arg] = 1.f;
-            chosen[(size_t)row * top + j] = arg;
-            weight[(size_t)row * top + j] = z[arg] * weight_scale;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+                if (oa >= 0 && (arg < 0 || ob > best || (!(best > ob) && oa < arg))) { best = ob; arg = oa; }
+            }
+            return __shfl_sync(0xffffffffu, arg, 0);      // (values that are not ordered: all lanes take lane 0's)
+        };
+        if (group_count > 0) {
+            const int size = E / group_count;
+            float* group = taken + E;             // [group_count] the groups' best scores, [group_count] marks
+            float* closed = group + group_count;
+            for (int gr = lane; gr < group_count; gr += 32) {
+                float best = -INFINITY;
+                for (int e = gr * size; e < (gr + 1) * size; ++e) best = fmaxf(best, z[e]);
+                group[gr] = best;
+                closed[gr] = 0.f;
+            }
+            __syncwarp();
+            for (int k = 0; k < group_keep; ++k) {
+                const int gr = pick(group_count, [&](int e) { return group[e]; }, [&](int e) { return closed[e] != 0.f; });
+                __syncwarp();
+                for (int e = gr * size + lane; e < (gr + 1) * size; e += 32) taken[e] = 0.f;
+                if (lane == 0) closed[gr] = 1.f;
+                __syncwarp();
+            }
+        }
+        float sum = 0.f;
+        for (int j = 0; j < top; ++j) {
+            const int arg = pick(E, [&](int e) { return z[e] + (correction ? correction[e] : 0.f); }, [&](int e) { return taken[e] != 0.f; });
+            __syncwarp();
+            sum += z[arg];
+            if (lane == 0) {
+                taken[arg] = 1.f;
+                chosen[(size_t)row * top + j] = arg;
+                weight[(size_t)row * top + j] = z[arg] * weight_scale;
+            }
+            __syncwarp();
+        }
+        if (scoring == 2 && lane == 0) {
+            for (int j = 0; j < top; ++j)
+                weight[(size_t)row * top + j] = z[chosen[(size_t)row * top + j]] / (sum + 1e-20f) * weight_scale;
         }
         return;
     }
+    if (lane != 0) return;
+    // selection: `top` times the largest logit that is left; a row of NaN still names `top` different experts
+    for (int e = 0; e < E; ++e) taken[e] = 0.f;
     float best0 = 0.f, sum = 0.f;
     for (int j = 0; j < top; ++j) {
         int arg = -1;
@@ -164,19 +214,23 @@ moe_route_kernel(int* __restrict__ chosen, float* __restrict__ weight, float* __
 
 TW_EXPORT int tw_moe_route(int* chosen, float* weight, float* shared_gate, const void* h, int h_stride, const void* wr,
                            const float* br, const void* ws, int rows, int width, int E, int top, int scoring,
-                           const float* correction, float weight_scale, int dtype, cudaStream_t stream) {
+                           const float* correction, float weight_scale, int group_count, int group_keep, int dtype,
+                           cudaStream_t stream) {
     if (rows <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || scoring < 0 || scoring > 1) return (int)cudaErrorInvalidValue;
-    const size_t smem = ((size_t)width + 2 * E + 1) * sizeof(float);
+    if (E <= 0 || top <= 0 || top > E || scoring < 0 || scoring > 2) return (int)cudaErrorInvalidValue;
+    if (group_count < 0 || (group_count > 0 && (scoring == 0 || E % group_count || group_keep < 1 || group_keep > group_count
+                                                || group_keep * (E / group_count) < top)))
+        return (int)cudaErrorInvalidValue;
+    const size_t smem = ((size_t)width + 2 * E + 1 + 2 * group_count) * sizeof(float);
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     const int threads = 32 * min(16, max(4, E + 1));        // a warp per expert (and one for the shared gate), up to 16
     if (dtype == TW_F32)
         return tw_launch(moe_route_kernel<float>, dim3(rows), dim3(threads), smem, stream, 1, chosen, weight, shared_gate,
                          (const float*)h, h_stride, (const float*)wr, br, (const float*)ws, width, E, top, scoring, correction,
-                         weight_scale);
+                         weight_scale, group_count, group_keep);
     return tw_launch(moe_route_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), smem, stream, 1, chosen, weight, shared_gate,
                      (const __nv_bfloat16*)h, h_stride, (const __nv_bfloat16*)wr, br, (const __nv_bfloat16*)ws, width, E, top,
-                     scoring, correction, weight_scale);
+                     scoring, correction, weight_scale, group_count, group_keep);
 }
 
 #define TW_MOE_WARPS 8

@@ -406,6 +406,46 @@ def add_rmsnorm(out: torch.Tensor, resid: torch.Tensor, delta, weight: torch.Ten
     _check(code, "add_rmsnorm")
 
 
+def _delta_operand(delta, like: torch.Tensor, hidden: int, n_rows: int | None, what: str):
+    """(tensor or None, slices or None, number of slices, their stride) of a delta that a norm kernel adds."""
+    if isinstance(delta, SplitSum):
+        slices = delta.slices
+        _need(slices.dtype == torch.float32 and slices.shape[2] == hidden and slices[0].is_contiguous(),
+              f"{what}: split sum must be fp32 [slices, rows, hidden]")
+        return None, slices, slices.shape[0], slices.stride(0)
+    _need(delta is None or (delta.dtype == like.dtype and delta.is_contiguous() and delta.shape[1] == hidden
+                            and (n_rows is None or delta.shape[0] >= n_rows)), f"{what}: delta must match the output type and width")
+    return delta, None, 0, 0
+
+
+def add_rmsnorm_pair(out: torch.Tensor, out2: torch.Tensor | None, resid: torch.Tensor, delta, delta2, weight: torch.Tensor,
+                     weight2: torch.Tensor | None, eps: float, n_rows: int, rows: torch.Tensor | None = None,
+                     delta_scale: float = 1.0) -> None:
+    """resid += delta_scale * (delta + delta2) (in place, fp32), out = rmsnorm(resid) * weight and out2 = rmsnorm(resid) *
+    weight2: what a layer whose two sub-layers read one stream through norms of their own does between layers.  Each
+    delta as in ``add_rmsnorm`` and either may be None; ``out2`` None: one result.  ``rows`` as in ``add_rmsnorm``."""
+    hidden = resid.shape[1]
+    n_src = None if rows is not None else n_rows
+    d1, p1, n1, s1 = _delta_operand(delta, out, hidden, n_src, "rmsnorm pair")
+    d2, p2, n2, s2 = _delta_operand(delta2, out, hidden, n_src, "rmsnorm pair")
+    _cuda(out, out2, resid, d1, p1, d2, p2, weight, weight2, rows)
+    _need(resid.dtype == torch.float32 and resid.is_contiguous(), "rmsnorm pair: residual stream must be contiguous fp32")
+    _need((out2 is None) == (weight2 is None), "rmsnorm pair: a second result has a weight of its own")
+    for o, w in ((out, weight), (out2, weight2)):
+        _need(o is None or (o.is_contiguous() and o.dtype == out.dtype and o.shape[1] == hidden and o.shape[0] >= n_rows
+                            and w.dtype == torch.float32 and w.numel() == hidden and w.is_contiguous()),
+              "rmsnorm pair: results of one type and the stream's width, with fp32 weights")
+    if rows is not None:
+        _need(rows.dtype == torch.int32 and rows.numel() >= n_rows, "rmsnorm pair: rows must be int32")
+    else:
+        _need(resid.shape[0] >= n_rows, "rmsnorm pair: fewer residual rows than asked")
+    code = _fn("elementwise", "tw_add_rmsnorm_pair")(
+        _ptr(out), _ptr(out2), _ptr(resid), _ptr(d1), _ptr(p1), c_int(n1), c_long(s1), _ptr(d2), _ptr(p2), c_int(n2), c_long(s2),
+        _ptr(weight), _ptr(weight2), c_float(eps), c_int(n_rows), c_int(hidden), _ptr(rows), c_float(delta_scale),
+        c_int(dtype_code(out.dtype)), _stream())
+    _check(code, "add_rmsnorm_pair")
+
+
 def rope_kv_write(qkv: torch.Tensor, bias: torch.Tensor | None, positions: torch.Tensor, seq_of_token: torch.Tensor,
                   seq_slot: torch.Tensor, block_table: torch.Tensor, inv_freq: torch.Tensor | None,
                   k_pages: torch.Tensor, v_pages: torch.Tensor, n_tokens: int, n_q_heads: int, n_kv_heads: int,
@@ -500,13 +540,15 @@ def norm_rotate_store(rows: torch.Tensor, n_tokens: int, spans: list[tuple[int, 
                       positions: torch.Tensor, seq_of_token: torch.Tensor, seq_slot: torch.Tensor, block_table: torch.Tensor,
                       k_pages: torch.Tensor, v_pages: torch.Tensor | None, k_col: int, v_col: int, write_cache: bool,
                       status: torch.Tensor, dst0: torch.Tensor | None = None, rot_col: int = 0, rot_dims: int = 0,
-                      inv_freq: torch.Tensor | None = None, interleaved: bool = False, magnitude: float = 1.0) -> None:
+                      inv_freq: torch.Tensor | None = None, interleaved: bool = False, magnitude: float = 1.0,
+                      gate_col: int = 0, gate_out: torch.Tensor | None = None) -> None:
     """One pass over every token's projected row: the norms of ``spans`` (as ``span_rmsnorm``; span 0 goes to the
     contiguous rows ``dst0`` instead of in place where given), the rotation by position of ``rot_dims`` values from
     column ``rot_col`` on (``rotate_pairs`` on one span), and the store of the key columns (from ``k_col``) and value
-    columns (from ``v_col``; ``v_pages`` None: one set of pages) into the token's place in the pages."""
+    columns (from ``v_col``; ``v_pages`` None: one set of pages) into the token's place in the pages.  ``gate_out``
+    (fp32 [rows, heads], or None) receives the sigmoid of as many columns from ``gate_col`` on."""
     _need(len(spans) <= 2, "norm_rotate_store: at most two spans")
-    _cuda(rows, positions, seq_of_token, seq_slot, block_table, k_pages, v_pages, status, dst0, inv_freq, *(w for _, _, _, w in spans))
+    _cuda(rows, positions, seq_of_token, seq_slot, block_table, k_pages, v_pages, status, dst0, inv_freq, gate_out, *(w for _, _, _, w in spans))
     _need(rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[0] >= n_tokens and rows.dtype == k_pages.dtype and k_pages.is_contiguous(),
           "norm_rotate_store: rows of the pages' type, contiguous pages")
     for col, heads, dim, w in spans:
@@ -524,6 +566,9 @@ def norm_rotate_store(rows: torch.Tensor, n_tokens: int, spans: list[tuple[int, 
     _need(k_col + kv_heads * dk <= rows.shape[1] and (v_pages is None or v_col + kv_heads * dv <= rows.shape[1]),
           "norm_rotate_store: the key and value columns must lie inside the rows")
     _need(block_table.dtype == torch.int32 and block_table.is_contiguous(), "norm_rotate_store: bad block table")
+    _need(gate_out is None or (gate_out.dtype == torch.float32 and gate_out.is_contiguous() and gate_out.shape[0] >= n_tokens
+                               and 0 <= gate_col and gate_col + gate_out.shape[1] <= rows.shape[1]),
+          "norm_rotate_store: the gates must be contiguous fp32 rows, and their columns lie inside the rows")
     (c0, h0, d0, w0) = spans[0] if spans else (0, 0, 0, None)
     (c1, h1, d1, w1) = spans[1] if len(spans) == 2 else (0, 0, 0, None)
     code = _fn("elementwise", "tw_norm_rotate_store")(
@@ -531,8 +576,8 @@ def norm_rotate_store(rows: torch.Tensor, n_tokens: int, spans: list[tuple[int, 
         c_int(c1), c_int(h1), c_int(d1), _ptr(w1), c_float(eps), c_int(rot_col), c_int(rot_dims), _ptr(inv_freq),
         c_int(1 if interleaved else 0), c_float(magnitude), c_int(k_col), c_int(v_col), _ptr(positions), _ptr(seq_of_token),
         _ptr(seq_slot), _ptr(block_table), c_int(block_table.shape[1]), _ptr(k_pages), _ptr(v_pages), c_int(kv_heads), c_int(dk),
-        c_int(dv), c_int(k_pages.shape[2]), c_int(k_pages.shape[0]), c_int(1 if write_cache else 0), c_int(dtype_code(rows.dtype)),
-        _ptr(status), _stream())
+        c_int(dv), c_int(k_pages.shape[2]), c_int(k_pages.shape[0]), c_int(1 if write_cache else 0), c_int(gate_col),
+        c_int(0 if gate_out is None else gate_out.shape[1]), _ptr(gate_out), c_int(dtype_code(rows.dtype)), _ptr(status), _stream())
     _check(code, "norm_rotate_store")
 
 
@@ -551,11 +596,12 @@ def gate_mul(out: torch.Tensor, x: torch.Tensor, gate: torch.Tensor, act: int, n
     _check(code, "gate_mul")
 
 
-def softcap(logits: torch.Tensor, cap: float) -> None:
-    """logits <- cap * tanh(logits / cap), in place on contiguous fp32 rows."""
+def softcap(logits: torch.Tensor, cap: float | None, scale: float = 1.0) -> None:
+    """logits <- scale * logits, then (with a cap) logits <- cap * tanh(logits / cap), in place on contiguous fp32 rows."""
     _cuda(logits)
-    _need(logits.dtype == torch.float32 and logits.is_contiguous() and cap > 0, "softcap: contiguous fp32 logits and a positive cap")
-    code = _fn("elementwise", "tw_softcap")(_ptr(logits), ctypes.c_longlong(logits.numel()), c_float(cap), _stream())
+    _need(logits.dtype == torch.float32 and logits.is_contiguous() and (cap is None or cap > 0), "softcap: contiguous fp32 logits and a positive cap")
+    code = _fn("elementwise", "tw_softcap")(_ptr(logits), ctypes.c_longlong(logits.numel()), c_float(scale),
+                                            c_float(0.0 if cap is None else cap), _stream())
     _check(code, "softcap")
 
 
@@ -1430,7 +1476,7 @@ def gemm_tcgen05_stream(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, m: 
 # ---------------------------------------------------------------------------
 # pieces of mixers that are not attention over a cache: recurrences with a matrix state, token shift
 # ---------------------------------------------------------------------------
-RECURRENCE_RETENTION, RECURRENCE_WKV, RECURRENCE_MLSTM, RECURRENCE_DELTA, RECURRENCE_GLA = 0, 1, 2, 3, 4
+RECURRENCE_RETENTION, RECURRENCE_WKV, RECURRENCE_MLSTM, RECURRENCE_DELTA, RECURRENCE_GLA, RECURRENCE_SSD = 0, 1, 2, 3, 4, 5
 RECURRENCE_MAX_KEY_DIM = 256      # a thread keeps a column of the state in registers (beyond 128 it spills)
 
 
@@ -1448,7 +1494,8 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
                       pre: torch.Tensor | None = None, p0: torch.Tensor | None = None, p1: torch.Tensor | None = None,
                       inv_freq: torch.Tensor | None = None, rot_dims: int = 0, q_scale: float = 1.0, k_scale: float = 1.0,
                       cap: float = 1.0, tail: torch.Tensor | None = None, tail_offset: int = 0, max_q_len: int = 1 << 30,
-                      write_pre: torch.Tensor | None = None, channel_decay: bool = False, qk_group: int = 1) -> None:
+                      write_pre: torch.Tensor | None = None, channel_decay: bool = False, qk_group: int = 1,
+                      p2: torch.Tensor | None = None) -> None:
     """Walk every request's rows of the step through its matrix state (csrc/linear_recurrence.cu): ``out`` fp32
     [rows, heads * value_dim] receives the raw outputs, ``den`` fp32 [rows, heads] the mLSTM denominators.  q, k, v are
     column slices of the projected rows (heads side by side).  ``pre``: fp32 rows the rule needs beside them (wkv:
@@ -1460,8 +1507,14 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
     ``channel_decay``, else [rows, heads]), ``p0`` the log of each head's rate [heads], ``p1`` the decay's bias (of
     ``pre``'s width), ``write_pre`` the write strength before its sigmoid, fp32 [rows, heads]; ``qk_group`` value heads
     share a head of q and k.  Gated linear attention takes ``pre`` the projected decay [rows, heads * key_dim], ``p0`` its
-    bias and ``cap`` the exponent 1 / tau of the sigmoid."""
-    _cuda(out, den, q, k, v, state, positions, seq_slot, seq_q_start, seq_q_len, pre, p0, p1, inv_freq, tail, write_pre)
+    bias and ``cap`` the exponent 1 / tau of the sigmoid.  The state-space rule takes fp32 q, k, v that are ready to use,
+    ``pre`` the projected step size [rows, heads], ``p0`` the log of each head's rate, ``p1`` the step size's bias and ``p2``
+    the skip, each [heads]; ``qk_group`` as in the delta rule."""
+    _cuda(out, den, q, k, v, state, positions, seq_slot, seq_q_start, seq_q_len, pre, p0, p1, p2, inv_freq, tail, write_pre)
+    _need(mode != RECURRENCE_SSD or (q.dtype == torch.float32 and pre is not None and pre.stride(1) == 1 and pre.shape[1] >= heads
+                                     and all(p is not None and p.numel() == heads and p.is_contiguous() for p in (p0, p1, p2))
+                                     and qk_group >= 1 and heads % qk_group == 0),
+          "recurrence: the state-space rule needs fp32 rows, a projected step size, and a rate, bias and skip per head")
     if mode == RECURRENCE_DELTA:
         width = heads * key_dim if channel_decay else heads
         _need(q.dtype == torch.float32 and pre is not None and p0 is not None and p1 is not None and write_pre is not None
@@ -1473,7 +1526,7 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
     _need(q.dtype == k.dtype == v.dtype and q.stride(1) == k.stride(1) == v.stride(1) == 1, "recurrence: q, k, v of one type, unit column stride")
     _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1, "recurrence: state must be fp32 [slots, numel]")
     _need(0 < key_dim <= 256 and 0 < value_dim <= 256, "recurrence: head sizes must lie in 1..256")
-    for t in (pre, p0, p1, inv_freq, den):
+    for t in (pre, p0, p1, p2, inv_freq, den):
         _need(t is None or t.dtype == torch.float32, "recurrence: constants, gates and denominators are fp32")
     _need(mode != RECURRENCE_MLSTM or (den is not None and pre is not None and p0 is not None), "recurrence: mlstm needs gates and a denominator buffer")
     _need(mode != RECURRENCE_WKV or (pre is not None and p0 is not None and p1 is not None and key_dim == value_dim), "recurrence: wkv needs decay rows, offset and bonus")
@@ -1483,7 +1536,7 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
           "recurrence: gated linear attention needs the projected decay rows, their bias and a positive exponent")
     code = _fn("linear_recurrence", "tw_linear_recurrence", {"TW_DK": key_dim})(
         c_int(mode), _ptr(out), _ptr(den), _ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)),
-        _ptr(pre), c_int(0 if pre is None else pre.stride(0)), _ptr(p0), _ptr(p1), _ptr(write_pre),
+        _ptr(pre), c_int(0 if pre is None else pre.stride(0)), _ptr(p0), _ptr(p1), _ptr(p2), _ptr(write_pre),
         c_int(0 if write_pre is None else write_pre.stride(0)), c_int(1 if channel_decay else 0), c_int(qk_group),
         _ptr(inv_freq), c_int(rot_dims),
         c_float(q_scale), c_float(k_scale), c_float(cap), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(tail),
@@ -1511,6 +1564,23 @@ def head_norm_gate(out: torch.Tensor, raw: torch.Tensor, den: torch.Tensor | Non
         _ptr(out), c_int(out.stride(0)), _ptr(raw), _ptr(den), _ptr(weight), _ptr(gate), c_int(0 if gate is None else gate.stride(0)),
         c_int(act), c_float(eps), c_int(n_rows), c_int(heads), c_int(value_dim), c_int(dtype_code(out.dtype)), _stream())
     _check(code, "head_norm_gate")
+
+
+def gate_part_norm(out: torch.Tensor, raw: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, act: int, eps: float, n_rows: int,
+                   parts: int) -> None:
+    """u = raw * act(gate) (fp32 ``raw`` [rows, width], ``gate`` a column slice of rows of the output's type); each of the
+    ``parts`` equal parts of a row of u is divided by its own root mean square; times ``weight`` (fp32 [width])."""
+    _cuda(out, raw, weight, gate)
+    width = raw.shape[1]
+    _need(raw.dtype == torch.float32 and raw.is_contiguous() and parts >= 1 and width % parts == 0, "gate_part_norm: raw must be fp32 rows of equal parts")
+    _need(out.stride(1) == 1 and out.shape[1] == width and gate.dtype == out.dtype and gate.stride(1) == 1 and gate.shape[1] == width
+          and min(out.shape[0], raw.shape[0], gate.shape[0]) >= n_rows, "gate_part_norm: gate and output rows of one type and raw's width")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == width, "gate_part_norm: weight fp32 [width]")
+    _need(act in (GATE_SILU, GATE_SIGMOID), "gate_part_norm: the activation is silu or sigmoid")
+    code = _fn("recurrent", "tw_gate_part_norm")(
+        _ptr(out), c_int(out.stride(0)), _ptr(raw), _ptr(weight), _ptr(gate), c_int(gate.stride(0)), c_int(act), c_float(eps),
+        c_int(n_rows), c_int(width), c_int(parts), c_int(dtype_code(out.dtype)), _stream())
+    _check(code, "gate_part_norm")
 
 
 def token_shift_mix(out: torch.Tensor, h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, state_offset: int,
@@ -1611,15 +1681,22 @@ def kv_store(rows: torch.Tensor, k_col: int, v_col: int, positions: torch.Tensor
 # ---------------------------------------------------------------------------
 def moe_route(chosen: torch.Tensor, weight: torch.Tensor, shared_gate: torch.Tensor | None, h: torch.Tensor, w_router: torch.Tensor,
               b_router: torch.Tensor | None, w_shared_gate: torch.Tensor | None, n_rows: int, top: int,
-              score_all: bool = False, correction: torch.Tensor | None = None, weight_scale: float = 1.0) -> None:
+              score_all: bool = False, correction: torch.Tensor | None = None, weight_scale: float = 1.0,
+              renormalise: bool = False, groups: tuple[int, int] | None = None) -> None:
     """Per row: the ``top`` experts with the largest fp32 logits ``w_router h + b_router`` (int32 [rows, top]), the
     softmax over those logits alone (fp32 [rows, top]), and ``sigmoid(w_shared_gate . h)`` (fp32 [rows]) if asked.
     With ``score_all`` the scores are the softmax over every router output, the choice goes by score + ``correction``
-    (fp32 [outputs], may be None) and the weights are the chosen scores times ``weight_scale``, not renormalised."""
+    (fp32 [outputs], may be None) and the weights are the chosen scores times ``weight_scale``, not renormalised -- or, with ``renormalise``, the chosen scores over their
+    sum (+ 1e-20) times ``weight_scale``.  ``groups`` = (count, keep): the outputs form ``count`` equal groups of neighbours
+    and only those of the ``keep`` groups with the largest best score may be chosen."""
     _cuda(chosen, weight, shared_gate, h, w_router, b_router, w_shared_gate, correction)
     experts, width = w_router.shape
     _need(correction is None or (score_all and correction.dtype == torch.float32 and correction.numel() == experts
                                  and correction.is_contiguous()), "moe_route: the correction is fp32 [router outputs] and goes with score_all")
+    count, keep = groups if groups is not None else (0, 0)
+    _need((groups is None and not renormalise) or score_all, "moe_route: groups and renormalised weights go with score_all")
+    _need(groups is None or (0 < keep <= count and experts % count == 0 and keep * (experts // count) >= top),
+          "moe_route: the kept groups must be some of equal groups, and hold enough outputs")
     _need(chosen.dtype == torch.int32 and weight.dtype == torch.float32 and chosen.is_contiguous() and weight.is_contiguous()
           and chosen.shape[1] == weight.shape[1] == top and chosen.shape[0] >= n_rows, "moe_route: chosen int32 / weight fp32 [rows, top]")
     _need(h.stride(1) == 1 and h.shape[1] == width and h.dtype == w_router.dtype and w_router.is_contiguous() and 0 < top <= experts,
@@ -1630,7 +1707,8 @@ def moe_route(chosen: torch.Tensor, weight: torch.Tensor, shared_gate: torch.Ten
         "moe_route: the shared gate needs a vector of the activations' type and an fp32 output")
     code = _fn("moe", "tw_moe_route")(_ptr(chosen), _ptr(weight), _ptr(shared_gate), _ptr(h), c_int(h.stride(0)), _ptr(w_router),
                                       _ptr(b_router), _ptr(w_shared_gate), c_int(n_rows), c_int(width), c_int(experts), c_int(top),
-                                      c_int(1 if score_all else 0), _ptr(correction), c_float(weight_scale),
+                                      c_int((2 if renormalise else 1) if score_all else 0), _ptr(correction), c_float(weight_scale),
+                                      c_int(count), c_int(keep),
                                       c_int(dtype_code(h.dtype)), _stream())
     _check(code, "moe_route")
 
@@ -1827,15 +1905,16 @@ SHORT_CONV_MAX_TAPS = 17
 def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, state_offset: int,
                seq_of_token: torch.Tensor, seq_slot: torch.Tensor, seq_q_start: torch.Tensor, n_rows: int,
                unit_heads: int = 0, unit_dim: int = 0, scaled_heads: int = 0, head_scale: float = 1.0, unit_eps: float = 0.0,
-               move_single: torch.Tensor | None = None) -> None:
-    """out[t, c] = silu(sum_j w[c, j] x[t - (taps - 1) + j, c]) in fp32 [rows, channels]: a causal convolution over the
+               move_single: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
+    """out[t, c] = silu([bias[c] +] sum_j w[c, j] x[t - (taps - 1) + j, c]) in fp32 [rows, channels]: a causal convolution over the
     rows of each request, per channel (the last tap is the row's own).  The taps - 1 rows before a request's first row of
     this step are read from its state (fp32, [channels, taps - 1] at ``state_offset``; zeros at a request's start).  The
     first ``unit_heads`` heads of ``unit_dim`` channels are then scaled to x / sqrt(sum x^2 + unit_eps), the first
     ``scaled_heads`` of those also by ``head_scale``.  ``short_conv_state`` moves the state on afterwards; with
     ``move_single`` (the requests' row counts of this step, int32) the kernel itself moves on the state of every request
     that brings one row, and ``short_conv_state(..., skip_single=True)`` is needed only for the others."""
-    _cuda(out, x, w, state, seq_of_token, seq_slot, seq_q_start, move_single)
+    _cuda(out, x, w, state, seq_of_token, seq_slot, seq_q_start, move_single, bias)
+    _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == w.shape[0]), "short_conv: the bias must be fp32 [channels]")
     _need(move_single is None or move_single.dtype == torch.int32, "short_conv: the row counts must be int32")
     channels, taps = w.shape
     _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == channels and out.shape[0] >= n_rows,
@@ -1846,7 +1925,7 @@ def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch
           and state_offset + channels * (taps - 1) <= state.shape[1], "short_conv: the state must be fp32 [slots, numel] with room for the taps")
     _need(0 <= scaled_heads <= unit_heads and unit_heads * unit_dim <= channels, "short_conv: the unit heads exceed the channels")
     code = _fn("recurrent", "tw_short_conv")(
-        _ptr(out), _ptr(x), c_int(x.stride(0)), _ptr(w), c_int(taps), _ptr(state), ctypes.c_longlong(state.stride(0)),
+        _ptr(out), _ptr(x), c_int(x.stride(0)), _ptr(w), _ptr(bias), c_int(taps), _ptr(state), ctypes.c_longlong(state.stride(0)),
         ctypes.c_longlong(state_offset), _ptr(seq_of_token), _ptr(seq_slot), _ptr(seq_q_start), _ptr(move_single),
         c_int(0 if move_single is None else 1), c_int(n_rows), c_int(channels),
         c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(head_scale), c_float(unit_eps), c_int(dtype_code(x.dtype)), _stream())

@@ -224,6 +224,105 @@ TW_EXPORT int tw_head_norm_gate(void* out, int out_stride, const float* raw, con
 }
 
 // ---------------------------------------------------------------------------
+// Gate first, then the norm: u = raw * act(gate); every row's u is cut into `parts` equal parts, and each part is divided
+// by its own root mean square, out = T(u / sqrt(mean_part(u^2) + eps) * weight).  act: 1 silu, 2 sigmoid.  fp32 until the
+// one rounding.  A block per (row, part); parts of up to 8,192 values on 16-byte boundaries are held in registers, others
+// are read and gated twice.
+// ---------------------------------------------------------------------------
+__device__ __forceinline__ float tw_gated(float y, float g, int act) {
+    const float sg = 1.0f / (1.0f + expf(-g));
+    return y * (act == 1 ? g * sg : sg);
+}
+__device__ __forceinline__ float4 tw_rec_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 tw_rec_load4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void tw_rec_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void tw_rec_store4(__nv_bfloat16* p, float4 v) {
+    uint2 raw;
+    *reinterpret_cast<__nv_bfloat162*>(&raw.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&raw.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+template <typename T, int V4>       // V4: groups of four values a thread keeps; 0: nothing is kept
+__global__ void __launch_bounds__(256)
+gate_part_norm_kernel(T* __restrict__ out, int out_stride, const float* __restrict__ raw, const float* __restrict__ weight,
+                      const T* __restrict__ gate, int gate_stride, int act, float eps, int width, int part) {
+    __shared__ float scratch[33];
+    tw_grid_wait();
+    tw_grid_launch_dependents();
+    const int row = blockIdx.x, c0 = blockIdx.y * part;
+    const float* r = raw + (size_t)row * width + c0;
+    const T* g = gate + (size_t)row * gate_stride + c0;
+    const float* w = weight + c0;
+    T* o = out + (size_t)row * out_stride + c0;
+    float ss = 0.f;
+    if constexpr (V4 > 0) {
+        const int n4 = part >> 2;
+        float4 u[V4];
+#pragma unroll
+        for (int j = 0; j < V4; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            u[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i < n4) {
+                const float4 y = tw_rec_load4(r + 4 * i), z = tw_rec_load4(g + 4 * i);
+                u[j] = make_float4(tw_gated(y.x, z.x, act), tw_gated(y.y, z.y, act), tw_gated(y.z, z.z, act), tw_gated(y.w, z.w, act));
+                ss += u[j].x * u[j].x + u[j].y * u[j].y + u[j].z * u[j].z + u[j].w * u[j].w;
+            }
+        }
+        const float inv = 1.0f / sqrtf(tw_block_sum(ss, scratch) / (float)part + eps);
+#pragma unroll
+        for (int j = 0; j < V4; ++j) {
+            const int i = threadIdx.x + j * blockDim.x;
+            if (i < n4) {
+                const float4 k = tw_rec_load4(w + 4 * i);
+                tw_rec_store4(o + 4 * i, make_float4(u[j].x * inv * k.x, u[j].y * inv * k.y, u[j].z * inv * k.z, u[j].w * inv * k.w));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < part; i += blockDim.x) {
+            const float u = tw_gated(r[i], tw_to_float(g[i]), act);
+            ss += u * u;
+        }
+        const float inv = 1.0f / sqrtf(tw_block_sum(ss, scratch) / (float)part + eps);
+        for (int i = threadIdx.x; i < part; i += blockDim.x)
+            o[i] = tw_from_float<T>(tw_gated(r[i], tw_to_float(g[i]), act) * inv * w[i]);
+    }
+}
+
+template <typename T>
+static int launch_gate_part_norm(T* out, int out_stride, const float* raw, const float* weight, const T* gate, int gate_stride,
+                                 int act, float eps, int rows, int width, int parts, cudaStream_t stream) {
+    const int part = width / parts;
+    auto a16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    const bool vec = (part & 3) == 0 && (width & 3) == 0 && (gate_stride & 3) == 0 && (out_stride & 3) == 0 && a16(raw) && a16(weight)
+                     && a16(gate) && a16(out);
+    const dim3 grid(rows, parts);
+    if (vec && part <= 4 * 64)
+        return tw_launch(gate_part_norm_kernel<T, 1>, grid, dim3(64), 0, stream, 1, out, out_stride, raw, weight, gate, gate_stride, act, eps, width, part);
+    if (vec && part <= 4 * 256 * 2)
+        return tw_launch(gate_part_norm_kernel<T, 2>, grid, dim3(256), 0, stream, 1, out, out_stride, raw, weight, gate, gate_stride, act, eps, width, part);
+    if (vec && part <= 4 * 256 * 8)
+        return tw_launch(gate_part_norm_kernel<T, 8>, grid, dim3(256), 0, stream, 1, out, out_stride, raw, weight, gate, gate_stride, act, eps, width, part);
+    return tw_launch(gate_part_norm_kernel<T, 0>, grid, dim3(part <= 128 ? 64 : 256), 0, stream, 1, out, out_stride, raw, weight, gate, gate_stride,
+                     act, eps, width, part);
+}
+
+TW_EXPORT int tw_gate_part_norm(void* out, int out_stride, const float* raw, const float* weight, const void* gate, int gate_stride,
+                                int act, float eps, int rows, int width, int parts, int dtype, cudaStream_t stream) {
+    if (rows <= 0) return 0;
+    if (width <= 0 || parts <= 0 || width % parts || act < 1 || act > 2) return (int)cudaErrorInvalidValue;
+    if (dtype == TW_F32)
+        return launch_gate_part_norm<float>((float*)out, out_stride, raw, weight, (const float*)gate, gate_stride, act, eps, rows, width, parts, stream);
+    return launch_gate_part_norm<__nv_bfloat16>((__nv_bfloat16*)out, out_stride, raw, weight, (const __nv_bfloat16*)gate, gate_stride, act, eps,
+                                                rows, width, parts, stream);
+}
+
+// ---------------------------------------------------------------------------
 // Token shift: out[m][row] = h[row] + (h[row - 1] - h[row]) * mu[m] for `n_mix` blends of a row with the row
 // before it in the same request.  A request's first row of a step takes the row the step before left in the
 // request's state (zeros at the very first token).  fp32 arithmetic, rounded once.
@@ -332,7 +431,7 @@ TW_EXPORT int tw_tanh_rows(void* x, long long count, int dtype, cudaStream_t str
 
 // ---------------------------------------------------------------------------
 // Short causal convolution over time, per channel, with silu, for the packed rows a recurrence reads:
-//   y[t, c] = silu(sum_j w[c, j] x[t - (taps - 1) + j, c]),   the last tap is the row's own, zeros before a request's start.
+//   y[t, c] = silu(bias[c] + sum_j w[c, j] x[t - (taps - 1) + j, c])  (bias may be null),   the last tap is the row's own, zeros before a request's start.
 // The taps - 1 rows before a request's first row of this step come from the request's state (fp32, channel-major:
 // state[offset + c * (taps - 1) + j], j = 0 the oldest), which tw_short_conv_state moves on afterwards.  Behind the
 // convolution the first `unit_heads` heads of `unit_dim` channels are scaled to unit length, x / sqrt(sum x^2 + unit_eps),
@@ -340,7 +439,7 @@ TW_EXPORT int tw_tanh_rows(void* x, long long count, int dtype, cudaStream_t str
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, int taps,
+short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias, int taps,
                   float* __restrict__ state, long long state_stride, long long state_offset,
                   const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                   const int* __restrict__ seq_q_len, int move_single, int channels, int chunk, int unit_heads, int unit_dim,
@@ -359,7 +458,7 @@ short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride
     // them moves them on itself (the oldest input leaves, the row's own joins), and the step needs no second kernel.
     const bool move = move_single && seq_q_len[s] == 1 && taps > 1;
     for (int c = c0 + threadIdx.x; c < c1; c += blockDim.x) {
-        float acc = 0.f;
+        float acc = bias ? bias[c] : 0.f;
         float* tc = tail + (size_t)c * (taps - 1);
         for (int j = 0; j < taps; ++j) {
             const int back = taps - 1 - j;               // how many rows before this one
@@ -396,7 +495,7 @@ short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256)
 short_conv_rows_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w,
-                       float* __restrict__ state, long long state_stride, long long state_offset,
+                       const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
                        const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                        const int* __restrict__ seq_q_len, int move_single, int n_rows, int channels, int chunk, int unit_heads,
                        int unit_dim, int scaled_heads, float head_scale, float unit_eps) {
@@ -411,6 +510,7 @@ short_conv_rows_kernel(float* __restrict__ out, const T* __restrict__ x, int x_s
         float wt[TAPS], xw[TAPS];
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) wt[j] = w[(size_t)c * TAPS + j];
+        const float b = bias ? bias[c] : 0.f;
         // xw[j] is the input TAPS - 1 - j rows before the current one (whichever request that row belongs to)
 #pragma unroll
         for (int j = 0; j + 1 < TAPS; ++j) {
@@ -430,7 +530,7 @@ short_conv_rows_kernel(float* __restrict__ out, const T* __restrict__ x, int x_s
                 const int r = row - seq_q_start[s];          // rows of this request before this one in the step
                 float* tc = state + (size_t)seq_slot[s] * state_stride + state_offset + (size_t)c * (TAPS - 1);
                 const bool move = move_single && TAPS > 1 && seq_q_len[s] == 1;
-                float acc = 0.f;
+                float acc = b;
 #pragma unroll
                 for (int j = 0; j < TAPS; ++j) {
                     const int back = TAPS - 1 - j;
@@ -495,7 +595,7 @@ __global__ void short_conv_state_kernel(const T* __restrict__ x, int x_stride, i
 }
 
 template <typename T>
-static int launch_short_conv(float* out, const T* x, int x_stride, const float* w, int taps, float* state, long long state_stride,
+static int launch_short_conv(float* out, const T* x, int x_stride, const float* w, const float* bias, int taps, float* state, long long state_stride,
                              long long state_offset, const int* seq_of_token, const int* seq_slot, const int* seq_q_start,
                              const int* seq_q_len, int move_single, int n_rows, int channels, int unit_heads, int unit_dim,
                              int scaled_heads, float head_scale, float unit_eps, cudaStream_t stream) {
@@ -517,7 +617,7 @@ static int launch_short_conv(float* out, const T* x, int x_stride, const float* 
                                                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rsmem);             \
                 if (e != cudaSuccess) return (int)e;                                                                             \
             }                                                                                                                    \
-            return tw_launch(short_conv_rows_kernel<T, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, state,    \
+            return tw_launch(short_conv_rows_kernel<T, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, bias, state, \
                              state_stride, state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows,   \
                              channels, chunk, unit_heads, unit_dim, scaled_heads, head_scale, unit_eps);                         \
         }
@@ -530,14 +630,14 @@ static int launch_short_conv(float* out, const T* x, int x_stride, const float* 
 #undef TW_CONV_ROWS_LAUNCH
     }
     const dim3 grid(n_rows, (channels + chunk - 1) / chunk);
-    return tw_launch(short_conv_kernel<T>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, taps, state, state_stride,
+    return tw_launch(short_conv_kernel<T>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, bias, taps, state, state_stride,
                      state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, channels, chunk, unit_heads,
                      unit_dim, scaled_heads, head_scale, unit_eps);
 }
 
 // seq_q_len with move_single: requests that bring one row have their state moved on by this kernel (and
 // tw_short_conv_state is then told to skip them).
-TW_EXPORT int tw_short_conv(float* out, const void* x, int x_stride, const float* w, int taps, float* state,
+TW_EXPORT int tw_short_conv(float* out, const void* x, int x_stride, const float* w, const float* bias, int taps, float* state,
                             long long state_stride, long long state_offset, const int* seq_of_token, const int* seq_slot,
                             const int* seq_q_start, const int* seq_q_len, int move_single, int n_rows, int channels,
                             int unit_heads, int unit_dim, int scaled_heads, float head_scale, float unit_eps, int dtype,
@@ -545,10 +645,10 @@ TW_EXPORT int tw_short_conv(float* out, const void* x, int x_stride, const float
     if (n_rows <= 0 || channels <= 0) return 0;
     if (taps < 1 || taps > 17 || unit_heads * unit_dim > channels || (move_single && !seq_q_len)) return (int)cudaErrorInvalidValue;
     if (dtype == TW_F32)
-        return launch_short_conv<float>(out, (const float*)x, x_stride, w, taps, state, state_stride, state_offset, seq_of_token,
+        return launch_short_conv<float>(out, (const float*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token,
                                         seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels, unit_heads, unit_dim,
                                         scaled_heads, head_scale, unit_eps, stream);
-    return launch_short_conv<__nv_bfloat16>(out, (const __nv_bfloat16*)x, x_stride, w, taps, state, state_stride, state_offset,
+    return launch_short_conv<__nv_bfloat16>(out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset,
                                             seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels,
                                             unit_heads, unit_dim, scaled_heads, head_scale, unit_eps, stream);
 }

@@ -606,7 +606,7 @@ def dugudra_kernel_table(config: dict, batch: int, context: int, prefill_tokens:
             [(lambda v=v, i=i: lat.prepare(ctx, projs[i % len(projs)], v, True)) for i, v in enumerate(views)],
             m * (lat.in_width + lat.q_rank + Dl + Hq * (2 * lat.q_head + Dl)) * 2 + maps,
             2.0 * m * Hq * lat.q_head * (lat.q_rank + Dl), note="the two products are the library's")
-        ql = lat.prepare(ctx, projs[0], views[0], True).clone()
+        ql = lat.prepare(ctx, projs[0], views[0], True)[0].clone()
         outs = [torch.empty(m, lat.q_size, device=dev, dtype=bf) for _ in range(2)]
         if phase == "decode":
             nbytes, flops = m * seen * per_key + m * 2 * lat.q_size * 2, 2.0 * m * Hq * 2 * Dl * seen

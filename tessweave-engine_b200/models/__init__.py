@@ -7,5 +7,6 @@ from . import sapatar  # noqa: F401  (registers "Sapatar")
 from . import nufatar  # noqa: F401  (registers "Nufatar")
 from . import dugudra  # noqa: F401  (registers "Dugudra")
 from . import varivik  # noqa: F401  (registers "Varivik")
+from . import bavetar  # noqa: F401  (registers "Bavetar")
 
 __all__ = ["LayerSpec", "ModelSpec", "ScheduleEntry", "Model"]

@@ -34,7 +34,7 @@ def mixer_spec(cfg: DugudraConfig, layer: DugudraLayer, where: str) -> PartSpec:
         return PartSpec("latent_attention", {
             "hidden": cfg.width, "n_heads": m.heads, "head_dim": m.dim, "rot_dim": m.rot_dim, "v_head_dim": m.vdim,
             "q_rank": m.q_rank, "kv_rank": m.kv_rank, "scale": m.scale, "eps": cfg.norm_eps, "window": m.window,
-            "position": position, "output_gate": True})
+            "position": position, "gate": "values"})
     if isinstance(m, GlaConfig):
         if m.decay_rank is None:
             raise ValueError(f"{where}: the inner size of the decay projection is known neither from 'decay_rank' nor from a checkpoint")

@@ -25,6 +25,7 @@ from typing import Any, Callable
 
 import torch
 
+from ..csrc import ops
 from ..csrc.ops import SplitSum
 
 
@@ -287,6 +288,13 @@ def dense_delta(ctx: "StepContext", delta, dtype: torch.dtype, name: str = "delt
     return delta
 
 
+@dataclass(frozen=True)
+class DeltaPair:
+    """Two pending deltas (each a tensor or a ``SplitSum``) of sub-layers that read the same stream: their sum joins it."""
+    first: object
+    second: object
+
+
 class Embedding(Part):
     """Turns the token ids of a step into the rows of the residual stream."""
 
@@ -309,15 +317,21 @@ class Head(Part):
 class Norm(Part):
     """out = norm(resid [+ delta]); updates the fp32 residual stream in place.
 
-    ``delta`` is None, a tensor of the activation type, or a ``SplitSum``.  A norm whose kernel adds
-    the slices itself sets ``accepts_split_sum``; callers go through ``apply``, which adds them up
-    first for a norm that does not."""
+    ``delta`` is None, a tensor of the activation type, a ``SplitSum``, or a ``DeltaPair`` of those.  A norm whose
+    kernel adds the slices itself sets ``accepts_split_sum``, one whose kernel adds two deltas at once
+    ``accepts_delta_pair``; callers go through ``apply``, which adds them up first for a norm that does not."""
     accepts_split_sum = False
+    accepts_delta_pair = False
 
     def apply(self, ctx: "StepContext", out: torch.Tensor, resid: torch.Tensor, delta, n_rows: int,
               rows: torch.Tensor | None = None, delta_scale: float = 1.0) -> None:
         """``delta_scale``: the delta is multiplied by it (in fp32) as it joins the stream; a norm that cannot do
         that implements ``forward`` without the argument and is only ever asked for a scale of 1."""
+        if isinstance(delta, DeltaPair) and not self.accepts_delta_pair:
+            if delta_scale != 1.0:
+                raise RuntimeError("a pair of deltas with a factor needs a norm whose kernel adds both")
+            ops.add_delta(resid, delta.first, ctx.n_tokens)
+            delta = delta.second
         if not self.accepts_split_sum:
             delta = dense_delta(ctx, delta, out.dtype)
         if delta_scale == 1.0:
@@ -328,6 +342,13 @@ class Norm(Part):
     def forward(self, ctx: "StepContext", out: torch.Tensor, resid: torch.Tensor, delta, n_rows: int,
                 rows: torch.Tensor | None = None, delta_scale: float = 1.0) -> None:
         raise NotImplementedError
+
+    def apply_twice(self, ctx: "StepContext", out: torch.Tensor, other: "Norm", other_out: torch.Tensor, resid: torch.Tensor,
+                    delta, n_rows: int, delta_scale: float = 1.0) -> None:
+        """The delta joins the stream, and both this norm and ``other`` write their rows of it.  A kind whose kernel does
+        both in one pass overrides this."""
+        self.apply(ctx, out, resid, delta, n_rows, delta_scale=delta_scale)
+        other.apply(ctx, other_out, resid, None, n_rows)
 
     def add_normed(self, ctx: "StepContext", resid: torch.Tensor, delta, n_rows: int,
                    copy: torch.Tensor | None = None) -> None:
@@ -403,7 +424,7 @@ class Block(Part):
 
 @dataclass
 class ResidualStream:
-    """The fp32 residual rows plus a delta (tensor or ``SplitSum``) the next norm still has to add.
+    """The fp32 residual rows plus a delta (tensor, ``SplitSum`` or ``DeltaPair``) the next norm still has to add.
     ``rounded``: the same rows (without the pending delta) in the activation type, if the part that wrote
     them last made that copy; whoever changes ``resid`` without renewing it sets it to None.
     ``copies``: fp32 [rows, copies, width] when a block keeps several parallel copies of the stream instead of

@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .base import (Block, PartSpec, ResidualStream, Runtime, StepContext, WeightDecl, build_part, dense_delta, join_name,
+from .base import (Block, DeltaPair, PartSpec, ResidualStream, Runtime, StepContext, WeightDecl, build_part, dense_delta, join_name,
                    register_part, unscaled_pending)
 
 
@@ -222,34 +222,41 @@ class HyperPreNormBlock(ArrangedBlock):
 
 @register_part("block", "parallel_pre_norm")
 class ParallelPreNormBlock(ArrangedBlock):
-    """x = x + (mixer(norm1(x)) + feed_forward(norm1(x))): one norm, and both sub-layers read its output.
-    ``feed_forward`` may be None: the layer then has its mixer only.
+    """x = x + (mixer(norm1(x)) + feed_forward(norm1(x))): both sub-layers read the same x, through one norm, or, with
+    ``norm2``, through a norm each: x = x + (mixer(norm1(x)) + feed_forward(norm2(x))).  ``feed_forward`` may be None:
+    the layer then has its mixer only (a checkpoint's tensor for its ``norm2`` is skipped).
 
-    The mixer's delta is added to the fp32 residual rows right away (nothing reads them before the next norm); the
-    feed-forward's is left pending, so the next norm's kernel adds it while it normalises.
+    Both deltas are left pending as a pair, so that the next norm's kernel adds them while it normalises; where a layer
+    has two norms, that kernel writes both results of the row it holds.
     """
 
-    ROLES = ("norm1", "mixer", "feed_forward")
+    ROLES = ("norm1", "mixer", "norm2", "feed_forward")
 
     def __init__(self, runtime: Runtime, hidden: int, norm1: PartSpec, mixer: PartSpec, feed_forward: PartSpec | None = None,
-                 names: dict[str, str] | None = None):
+                 names: dict[str, str] | None = None, norm2: PartSpec | None = None):
         super().__init__(runtime, hidden, names)
         self.norm1 = build_part("norm", norm1, runtime)
         self.mixer = build_part("mixer", mixer, runtime)
+        self.norm2 = build_part("norm", norm2, runtime) if norm2 is not None and feed_forward is not None else None
+        self.unused_norm2 = norm2 is not None and feed_forward is None
         self.feed_forward = build_part("feed_forward", feed_forward, runtime) if feed_forward is not None else None
         self.graph_safe = all(p.graph_safe for p in self.parts().values())
+
+    def redundant_names(self) -> list[str]:
+        return super().redundant_names() + ([self.names["norm2"]] if self.unused_norm2 else [])
 
     def forward(self, ctx: StepContext, stream: ResidualStream, cache, write_cache: bool) -> None:
         n, dt = ctx.n_tokens, self.runtime.dtype
         stream.rounded = None
         h = ctx.workspace.get("block.h", (n, self.hidden), dt)
-        self.norm1.apply(ctx, h, stream.resid, stream.pending, n, delta_scale=stream.pending_scale)
+        if self.norm2 is None:
+            h2 = h
+            self.norm1.apply(ctx, h, stream.resid, stream.pending, n, delta_scale=stream.pending_scale)
+        else:
+            h2 = ctx.workspace.get("block.h2", (n, self.hidden), dt)
+            self.norm1.apply_twice(ctx, h, self.norm2, h2, stream.resid, stream.pending, n, delta_scale=stream.pending_scale)
         stream.pending_scale = 1.0
         ctx.upcoming_weights = self.feed_forward.streamed_first() if self.feed_forward is not None else None
         delta = self.mixer.forward(ctx, h, cache, write_cache)
         ctx.upcoming_weights = None
-        if self.feed_forward is None:
-            stream.pending = delta
-            return
-        ops.add_delta(stream.resid, delta, n)
-        stream.pending = self.feed_forward.forward(ctx, h)
+        stream.pending = delta if self.feed_forward is None else DeltaPair(delta, self.feed_forward.forward(ctx, h2))

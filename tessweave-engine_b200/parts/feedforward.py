@@ -172,7 +172,9 @@ class RoutedExperts(FeedForward):
 
     Options of other designs.  ``score_all``: the scores are s = softmax(z) over *every* router output, the ``top``
     outputs with the largest s + ``correction`` (a stored fp32 vector named by ``correction``, or none) are chosen, and
-    the weights are their s times ``weight_scale``, not renormalised.  ``identity`` n: the router has n outputs more
+    the weights are their s times ``weight_scale``, not renormalised; with ``renormalise`` they are divided by their sum
+    (+ 1e-20) first.  ``groups`` (``count``, ``keep``): the outputs form ``count`` equal groups of neighbours, a group counts
+    as much as its best score, and only outputs of the ``keep`` best groups can be chosen.  ``identity`` n: the router has n outputs more
     than there are experts; such an output is an expert without tensors whose result is the token's row itself.
     ``activation``: ``{"kind": "clamped", "limit": l, "alpha": a}`` makes an expert's inner rows
     g sigmoid(a g) (u + 1) with g = min(Wg h, l), u = clamp(Wu h, -l, l) instead of silu(Wg h) (Wu h).  ``{"kind":
@@ -185,14 +187,23 @@ class RoutedExperts(FeedForward):
     def __init__(self, runtime: Runtime, hidden: int, experts: int, top: int, intermediate: int,
                  shared: PartSpec | None = None, shared_gate: bool = False, router_bias: bool = True,
                  names: dict[str, str] | None = None, score_all: bool = False, correction: str | None = None,
-                 weight_scale: float = 1.0, identity: int = 0, activation: dict | None = None):
+                 weight_scale: float = 1.0, identity: int = 0, activation: dict | None = None, renormalise: bool = False,
+                 groups: dict | None = None):
         super().__init__(runtime)
         if min(hidden, experts, top, intermediate) <= 0 or identity < 0 or top > experts + identity:
             raise ValueError("routed_experts: sizes must be positive and top at most the number of router outputs")
         if shared_gate and shared is None:
             raise ValueError("routed_experts: a gate of the shared expert needs a shared expert")
-        if (correction is not None or weight_scale != 1.0) and not score_all:
-            raise ValueError("routed_experts: a correction of the choice and a scale of the weights go with score_all")
+        if (correction is not None or weight_scale != 1.0 or renormalise or groups is not None) and not score_all:
+            raise ValueError("routed_experts: a correction of the choice, a scale of the weights, renormalised weights and groups "
+                             "go with score_all")
+        self.renormalise = bool(renormalise)
+        self.groups = (int(groups["count"]), int(groups["keep"])) if groups is not None else None
+        if self.groups is not None:
+            count, keep = self.groups
+            if not 0 < keep <= count or (experts + identity) % count or keep * ((experts + identity) // count) < top:
+                raise ValueError(f"routed_experts: {count} equal groups of {experts + identity} outputs, of which {keep} hold at "
+                                 f"least {top}, are not possible")
         self.hidden, self.experts, self.top, self.intermediate = hidden, experts, top, intermediate
         self.identity, self.outputs = int(identity), experts + int(identity)
         self.score_all, self.weight_scale = bool(score_all), float(weight_scale)
@@ -254,7 +265,8 @@ class RoutedExperts(FeedForward):
         gate = ws.get("moe.shared_gate", (n,), torch.float32) if self.w_shared_gate is not None else None
         ops.moe_route(chosen, weight, gate, h, self.w_router, self.b_router,
                       self.w_shared_gate.view(-1) if self.w_shared_gate is not None else None, n, self.top,
-                      score_all=self.score_all, correction=self.correction, weight_scale=self.weight_scale)
+                      score_all=self.score_all, correction=self.correction, weight_scale=self.weight_scale,
+                      renormalise=self.renormalise, groups=self.groups)
         return chosen, weight, gate
 
     def forward(self, ctx: StepContext, h: torch.Tensor):

@@ -20,6 +20,11 @@ class LatentAttention(PagedSoftmaxMixer):
         s_h(i, j) = (a_h(i) . k_h(j) + b_h(i) . r(j)) * scale        over the keys the window lets i see
         o_h = sum_j softmax_j(s_h) v_h(j);   delta = Wo (o * sigmoid(Wg h))                   (the gate is optional)
 
+    ``gate``: "values" (Wg has a row per value of every head, as above), "heads" (one row per head: head h's output is
+    multiplied by sigmoid(Wg h)_h) or None.  A gate per head is a number the attention kernels multiply by in their
+    epilogue: it commutes with the head's value map.  ``sink`` (a tensor name): a learned number per head whose
+    exponential joins the softmax's denominator -- it has no key and no value, is not scaled and counts once.
+
     Neither k_h nor v_h is ever formed.  Because k_h is linear in c, a_h . k_h(j) = (Wuk_h^T a_h) . c(j): the query is
     carried into the latent space once per token, and then every head is an ordinary attention head of size
     kv_rank + rot_dim whose keys are the rows [c | r] of ONE key/value head and whose values are the same rows (the
@@ -39,8 +44,8 @@ class LatentAttention(PagedSoftmaxMixer):
              "gate": "g", "out": "o"}
 
     def __init__(self, runtime: Runtime, hidden: int, n_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, q_rank: int,
-                 kv_rank: int, scale: float, eps: float, position: PartSpec, window: int | None = None, output_gate: bool = True,
-                 names: dict[str, str] | None = None):
+                 kv_rank: int, scale: float, eps: float, position: PartSpec, window: int | None = None, gate: str | None = "values",
+                 sink: str | None = None, names: dict[str, str] | None = None):
         super().__init__(runtime)
         if min(hidden, n_heads, head_dim, v_head_dim, q_rank, kv_rank) <= 0 or rot_dim < 0 or rot_dim % 2:
             raise ValueError("latent_attention: sizes must be positive and the rotated part even")
@@ -60,13 +65,21 @@ class LatentAttention(PagedSoftmaxMixer):
         self.v_dim, self.same_dims = self.head_dim, True
         self.q_size = n_heads * self.head_dim
         self.window, self.scale = window, float(scale)
-        self.sink = self.bias_rows = self.bias_by_distance = None
+        if gate not in ("values", "heads", None):
+            raise ValueError(f"latent_attention: the gate is per 'values', per 'heads' or None, not {gate!r}")
+        self.bias_rows = self.bias_by_distance = None
+        self.sink_name = sink
+        self.sink = runtime.empty(n_heads, dtype=torch.float32) if sink is not None else None
         self.score_terms = True                              # the values are the keys
-        self.has_gate = bool(output_gate)
+        self.gate = gate
         self.out_size = n_heads * v_head_dim
-        # rows [Wdq; Wdkv; Wg]: one product reads h
-        self.in_width = q_rank + self.head_dim + (self.out_size if self.has_gate else 0)
+        # rows [Wdq; Wdkv; Wg], one product reads h; with a gate per head the rows end on a 16-byte boundary
+        self.gate_size = {"values": self.out_size, "heads": n_heads, None: 0}[gate]
+        self.in_width = q_rank + self.head_dim + self.gate_size
+        if gate == "heads":
+            self.in_width = -(-self.in_width // 8) * 8
         self.w_in = runtime.empty(self.in_width, hidden)
+        self.w_in[q_rank + self.head_dim + self.gate_size:].zero_()
         self.w_uq = runtime.empty(n_heads * self.q_head, q_rank)
         self.q_norm_w = runtime.empty(q_rank, dtype=torch.float32)
         self.c_norm_w = runtime.empty(kv_rank, dtype=torch.float32)
@@ -87,8 +100,10 @@ class LatentAttention(PagedSoftmaxMixer):
                  WeightDecl(nm["uk"], (H * self.plain_dim, self.kv_rank), dest=self.to_latent[:, :self.plain_dim, :self.kv_rank]),
                  WeightDecl(nm["uv"], (H * self.value_dim, self.kv_rank), dest=self.w_uv),
                  WeightDecl(nm["out"], (hid, self.out_size), dest=self.w_o)]
-        if self.has_gate:
-            decls.append(WeightDecl(nm["gate"], (self.out_size, hid), dest=self.w_in[b:]))
+        if self.gate is not None:
+            decls.append(WeightDecl(nm["gate"], (self.gate_size, hid), dest=self.w_in[b:b + self.gate_size]))
+        if self.sink is not None:
+            decls.append(WeightDecl(self.sink_name, (H,), role="vector", init="wide_normal", dest=self.sink))
         return decls
 
     def cache_need(self) -> PagedKV:
@@ -118,40 +133,42 @@ class LatentAttention(PagedSoftmaxMixer):
         ops.rotate_pairs(rows, ctx.positions, ctx.seq_of_token, plan.inv_freq, ctx.n_tokens, n_heads, head_dim, plan.rot_dims,
                          plan.interleaved, magnitude=plan.magnitude, first=first)
 
-    def prepare(self, ctx: StepContext, proj: torch.Tensor, cache: PagedView, write_cache: bool) -> torch.Tensor:
-        """Norms, rotation, the store of [c | r], and the queries in the latent space: [rows, H * (kv_rank + rot_dim)]."""
+    def prepare(self, ctx: StepContext, proj: torch.Tensor, cache: PagedView, write_cache: bool):
+        """Norms, rotation, the store of [c | r], and the queries in the latent space: (those, [rows, H * (kv_rank +
+        rot_dim)]; the heads' gates fp32 [rows, H], or None)."""
         n, ws, dt, H = ctx.n_tokens, ctx.workspace, self.runtime.dtype, self.n_heads
         a = self.q_rank
         # one pass over a token's row: both latents' norms (the query latent into rows of its own, which the next
         # product reads), the rotation of the shared key part, the store of [c | r]
         plan = self._plan()
         cq = ws.get("latent.cq", (n, a), dt)
+        gates = ws.get("latent.gates", (n, H), torch.float32) if self.gate == "heads" else None
         ops.norm_rotate_store(proj, n, [(0, 1, self.q_rank, self.q_norm_w), (a, 1, self.kv_rank, self.c_norm_w)], self.eps,
                               ctx.positions, ctx.seq_of_token, ctx.seq_slot, cache.block_table, cache.k_pages, None, a, a,
                               write_cache, ctx.status, dst0=cq, rot_col=a + self.kv_rank, rot_dims=self.rot_dim,
                               inv_freq=plan.inv_freq if plan is not None else None,
                               interleaved=plan.interleaved if plan is not None else False,
-                              magnitude=plan.magnitude if plan is not None else 1.0)
+                              magnitude=plan.magnitude if plan is not None else 1.0, gate_col=a + self.head_dim, gate_out=gates)
         q = linear(ctx, "latent.q", cq, self.w_uq)
         self._rotate(ctx, q, H, self.q_head, self.plain_dim)
         ql = ws.get("latent.q_latent", (n, self.q_size), dt)
         configure_matmul_precision()
         ops.note_call("library batched product")
         torch.bmm(q.view(n, H, self.q_head).transpose(0, 1), self.to_latent, out=ql.view(n, H, self.head_dim).transpose(0, 1))
-        return ql
+        return ql, gates
 
     def attend(self, ctx: StepContext, proj: torch.Tensor, cache: PagedView, write_cache: bool) -> torch.Tensor:
         """The heads' results after their value maps and the gate: [rows, H * v_head_dim]."""
         n, ws, dt, H = ctx.n_tokens, ctx.workspace, self.runtime.dtype, self.n_heads
-        ql = self.prepare(ctx, proj, cache, write_cache)
+        ql, gates = self.prepare(ctx, proj, cache, write_cache)
         mixed = ws.get("latent.mixed", (n, self.q_size), dt)
-        self._attend(ctx, mixed, ql, cache)
+        self._attend(ctx, mixed, ql, cache, gate=gates)
         out = ws.get("latent.out", (n, self.out_size), dt)
         ops.note_call("library batched product")
         torch.bmm(mixed.view(n, H, self.head_dim)[:, :, :self.kv_rank].transpose(0, 1),
                   self.w_uv.view(H, self.value_dim, self.kv_rank).transpose(1, 2),
                   out=out.view(n, H, self.value_dim).transpose(0, 1))
-        if self.has_gate:
+        if self.gate == "values":
             ops.gate_mul(out, out, proj[:, self.q_rank + self.head_dim:], ops.GATE_SIGMOID, n)
         return out
 

@@ -4,7 +4,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .base import Norm, Runtime, StepContext, WeightDecl, register_part
+from .base import DeltaPair, Norm, Runtime, StepContext, WeightDecl, register_part
 
 
 @register_part("norm", "rmsnorm")
@@ -18,6 +18,7 @@ class RMSNorm(Norm):
     around zero and the norm multiplies by ``1 + w`` (the one is added once, in fp32, when the weights are in).
     """
     accepts_split_sum = True
+    accepts_delta_pair = True
 
     def __init__(self, runtime: Runtime, size: int, eps: float, weight_name: str = "weight", unit_offset: bool = False):
         super().__init__(runtime)
@@ -38,7 +39,18 @@ class RMSNorm(Norm):
             torch.add(self._stored, 1.0, out=self.weight)
 
     def forward(self, ctx: StepContext, out, resid, delta, n_rows, rows=None, delta_scale: float = 1.0) -> None:
+        if isinstance(delta, DeltaPair):
+            ops.add_rmsnorm_pair(out, None, resid, delta.first, delta.second, self.weight, None, self.eps, n_rows, rows,
+                                 delta_scale=delta_scale)
+            return
         ops.add_rmsnorm(out, resid, delta, self.weight, self.eps, n_rows, rows, delta_scale=delta_scale)
+
+    def apply_twice(self, ctx: StepContext, out, other, other_out, resid, delta, n_rows, delta_scale: float = 1.0) -> None:
+        if not (isinstance(other, RMSNorm) and other.eps == self.eps):
+            super().apply_twice(ctx, out, other, other_out, resid, delta, n_rows, delta_scale)
+            return
+        first, second = (delta.first, delta.second) if isinstance(delta, DeltaPair) else (delta, None)
+        ops.add_rmsnorm_pair(out, other_out, resid, first, second, self.weight, other.weight, self.eps, n_rows, delta_scale=delta_scale)
 
     def add_normed(self, ctx: StepContext, resid, delta, n_rows, copy=None) -> None:
         ops.rmsnorm_to_residual(resid, delta, self.weight, self.eps, n_rows, copy)

@@ -453,3 +453,83 @@ class GatedLinearAttention(MatrixStateMixer):
         raw, _ = self._recur(ctx, proj[:, :a], proj[:, a:2 * a], proj[:, 2 * a:2 * a + b], cache, write_cache,
                              pre=decay, p0=self.b_a2, q_scale=self.key_dim ** -0.5, cap=1.0 / self.tau)
         return self._finish(ctx, raw, None, self.norm_per_head, proj[:, 2 * a + b:])
+
+
+@register_part("mixer", "mamba2")
+class Mamba2(MatrixStateMixer):
+    """State-space duality (Mamba-2): a matrix state whose decay and write strength come from one step size per head.
+
+        [z | x | B | C | d] = W h            z, x: n_heads heads of value_dim; B, C: n_groups heads of state_dim; d: one per head
+        x, B, C: a causal convolution over time per channel (``conv_taps`` taps and a bias, zeros before the start), then silu
+        dt = softplus(d + dt_bias);  S <- exp(-exp(A_log) dt) S + dt B x^T;  y = S^T C + D x        fp32, S zero at the start
+        u = y * silu(z); each of ``norm_groups`` equal parts of u over its own root mean square; delta = (u * norm) Wo^T
+
+    Head h reads group h // (n_heads / n_groups) of B and C.  In the terms of the other rules B is the key, C the query
+    and x the value.  The state slot holds S of every head and, behind them, the last ``conv_taps - 1`` inputs of every
+    convolved channel, so a request may be cut into steps anywhere.  W is one tensor; its last rows (d), which enter the
+    recurrence, are a product of their own with an fp32 result.
+    ``names``: in, conv, conv_bias, dt_bias, rate_log, skip, norm, out.
+    """
+
+    rule = ops.RECURRENCE_SSD
+    NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "rate_log": "A_log", "skip": "D",
+             "norm": "norm", "out": "o"}
+
+    def __init__(self, runtime: Runtime, hidden: int, n_heads: int, value_dim: int, state_dim: int, n_groups: int, conv_taps: int,
+                 norm_groups: int, eps: float, names: dict[str, str] | None = None):
+        super().__init__(runtime)
+        self._sizes(hidden, n_heads, state_dim, value_dim, eps)
+        if n_groups <= 0 or n_heads % n_groups:
+            raise ValueError("mamba2: n_heads must be a multiple of n_groups")
+        if not 1 <= conv_taps <= ops.SHORT_CONV_MAX_TAPS:
+            raise ValueError(f"mamba2: conv_taps must lie in 1..{ops.SHORT_CONV_MAX_TAPS}")
+        if norm_groups <= 0 or self.v_size % norm_groups:
+            raise ValueError("mamba2: norm_groups must divide n_heads * value_dim")
+        self.names = {**self.NAMES, **(names or {})}
+        self.n_groups, self.taps, self.norm_groups = int(n_groups), int(conv_taps), int(norm_groups)
+        self.qk_size = n_groups * state_dim                      # (the base class counted a q/k head per value head)
+        self.conv_channels = self.v_size + 2 * self.qk_size
+        self.conv_offset = self.state_numel                      # where the convolution's last inputs sit in a slot
+        self.state_numel += self.conv_channels * (self.taps - 1)
+        self.row_size = self.v_size + self.conv_channels         # [z | x | B | C]
+        self.w_in = runtime.empty(self.row_size + n_heads, hidden)
+        self.conv = runtime.empty(self.conv_channels, self.taps, dtype=torch.float32)
+        self.conv_bias, self.norm = (runtime.empty(n, dtype=torch.float32) for n in (self.conv_channels, self.v_size))
+        self.rate_log, self.dt_bias, self.skip = (runtime.empty(n_heads, dtype=torch.float32) for _ in range(3))
+        self.w_o = runtime.empty(hidden, self.v_size)
+
+    def weights(self) -> list[WeightDecl]:
+        nm, H = self.names, self.n_heads
+        return [WeightDecl(nm["in"], (self.row_size + H, self.hidden), dest=self.w_in),
+                WeightDecl(nm["conv"], (self.conv_channels, self.taps), role="vector", init="wide_normal", dest=self.conv),
+                WeightDecl(nm["conv_bias"], (self.conv_channels,), role="vector", init="normal", dest=self.conv_bias),
+                WeightDecl(nm["dt_bias"], (H,), role="vector", init="wide_normal", dest=self.dt_bias),
+                WeightDecl(nm["rate_log"], (H,), role="vector", init="wide_normal", dest=self.rate_log),
+                WeightDecl(nm["skip"], (H,), role="vector", init="one_plus_normal", dest=self.skip),
+                WeightDecl(nm["norm"], (self.v_size,), role="vector", init="one_plus_normal", dest=self.norm),
+                WeightDecl(nm["out"], (self.hidden, self.v_size), dest=self.w_o)]
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, cache, write_cache: bool):
+        cache = self._check(cache)
+        raw, proj = self.recur(ctx, h, cache, write_cache)
+        out = ctx.workspace.get("recurrence.out", (ctx.n_tokens, self.v_size), self.runtime.dtype)
+        ops.gate_part_norm(out, raw, self.norm, proj[:, :self.v_size], ops.GATE_SILU, self.eps, ctx.n_tokens, self.norm_groups)
+        return linear(ctx, "mixer.delta", out, self.w_o, allow_split=True)
+
+    def recur(self, ctx: StepContext, h: torch.Tensor, cache: StateView, write_cache: bool):
+        """(y fp32 [rows, heads * value_dim], the projected rows [z | x | B | C]); the requests' states move on."""
+        n, ws = ctx.n_tokens, ctx.workspace
+        b, a, C = self.v_size, self.qk_size, self.conv_channels
+        proj = linear(ctx, "mamba2.in", h, self.w_in[:self.row_size])
+        step = linear(ctx, "mamba2.step", h, self.w_in[self.row_size:], out_dtype=torch.float32)
+        mixed = proj[:, b:]
+        ready = ws.get("mamba2.ready", (n, C), torch.float32)
+        ops.short_conv(ready, mixed, self.conv, cache.state, self.conv_offset, ctx.seq_of_token, ctx.seq_slot, ctx.seq_q_start, n,
+                       move_single=ctx.seq_q_len if write_cache else None, bias=self.conv_bias)
+        if write_cache and self.taps > 1 and not ctx.decode_only:
+            # (a request that brings one row had its state moved on by the convolution itself)
+            ops.short_conv_state(mixed, self.taps, C, cache.state, self.conv_offset, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
+                                 ctx.n_seqs, skip_single=True)
+        raw, _ = self._recur(ctx, ready[:, b + a:], ready[:, b:b + a], ready[:, :b], cache, write_cache, pre=step,
+                             p0=self.rate_log, p1=self.dt_bias, p2=self.skip, qk_group=self.n_heads // self.n_groups)
+        return raw, proj
