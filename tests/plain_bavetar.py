@@ -210,3 +210,11 @@ def read_folder(folder, dtype=torch.float64):
 def logits_of(folder, tokens, dtype=torch.float64) -> torch.Tensor:
     cfg, w = read_folder(folder, dtype)
     return forward(cfg, w, tokens)
+
+
+def greedy(folder, prompt, steps):
+    cfg, w = read_folder(folder, torch.float64)
+    ids = list(prompt)
+    for _ in range(steps):
+        ids.append(int(torch.argmax(forward(cfg, w, ids)[-1])))
+    return ids[len(prompt):]

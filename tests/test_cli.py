@@ -333,3 +333,47 @@ def test_generate_varivik_as_a_user_starts_it(tmp_path):
     assert proc.returncode == 0, proc.stderr[-3000:]
     got = [int(t) for t in proc.stdout.strip().split(",")]
     assert got == plain_varivik.greedy(folder, prompt, 8)
+
+
+# ---------------------------------------------------------------------------
+# the Bavetar decoder through the same command line
+# ---------------------------------------------------------------------------
+def test_doctor_and_inspect_know_bavetar(tmp_path):
+    from tiny_bavetar import BAVETAR_A
+    assert "Bavetar" in json.loads(run_cli("doctor").stdout)["architectures"]
+    config = tmp_path / "config.json"
+    config.write_text(json.dumps(BAVETAR_A))
+    folder = tmp_path / "model"
+    assert run_cli("init", folder, "--config", config, "--seed", 2, "--init-std", 0.1).returncode == 0
+    proc = run_cli("inspect", folder, "--kv-blocks", 10, "--block-size", 8)
+    assert proc.returncode == 0, proc.stderr
+    out = json.loads(proc.stdout)
+    mixers = [layer["mixer"] for layer in BAVETAR_A["layers"]]
+    assert out["layers_in_schedule"] == len(mixers)
+    assert out["kv_bf16_bytes"] == sum(m["kv_rank"] + m["rot_dim"] for m in mixers if "kv_rank" in m) * 2 * 10 * 8
+    assert out["state_bytes_per_request"] == 4 * sum(
+        m["heads"] * m["state"] * m["vdim"] + (m["heads"] * m["vdim"] + 2 * m["groups"] * m["state"]) * (m["conv"] - 1)
+        for m in mixers if "state" in m)
+    bad = tmp_path / "bad"
+    bad.mkdir()
+    (bad / "config.json").write_text(json.dumps({**BAVETAR_A, "layers": [{**BAVETAR_A["layers"][0], "type": "conv"}]}))
+    proc = run_cli("inspect", bad)
+    assert proc.returncode != 0 and "not implemented" in proc.stderr
+
+
+@pytest.mark.gpu
+def test_generate_bavetar_as_a_user_starts_it(tmp_path):
+    """init -> generate --prompt-ids in float32 -> the plain implementation's greedy continuation."""
+    import plain_bavetar
+    from tiny_bavetar import BAVETAR_D
+    config = tmp_path / "config.json"
+    config.write_text(json.dumps(BAVETAR_D))
+    folder = tmp_path / "model"
+    assert run_cli("init", folder, "--config", config, "--seed", 11, "--init-std", 0.25).returncode == 0
+    prompt = [5, 17, 3, 20, 41, 7, 50, 10, 23]
+    proc = run_cli("generate", folder, "--prompt-ids", ",".join(map(str, prompt)), "--dtype", "float32", "--max-tokens", 8,
+                   "--ignore-eos", "--log", tmp_path / "runs" / "engine.jsonl", "--block-size", 8, "--kv-blocks", 32,
+                   "--prefill-chunk", 4, "--max-context", 256)
+    assert proc.returncode == 0, proc.stderr[-3000:]
+    got = [int(t) for t in proc.stdout.strip().split(",")]
+    assert got == plain_bavetar.greedy(folder, prompt, 8)

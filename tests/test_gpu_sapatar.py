@@ -90,7 +90,7 @@ def test_hyper_connection_pass(dtype, copies, width):
 
 
 def run_state_mixer(rt, mixer, hidden, plain_fn, lengths=(223, 9), plan=((7, 0), (1, 4), (2, 1), (0, 1), (150, 3), (63, 0)),
-                    loud_row=None):
+                    loud_row=None, bf16=3e-2):
     """A mixer with a fixed-size state, cut into steps (down to one row, up to 150), two requests side by side in
     slots 2 and 0; against the plain mixer on each whole sequence.  ``loud_row``: that row of request a is twelve
     times as large as the others, so that what it leaves in the state outweighs everything else for as long as the
@@ -112,8 +112,8 @@ def run_state_mixer(rt, mixer, hidden, plain_fn, lengths=(223, 9), plan=((7, 0),
         out = dense_delta(ctx, mixer.forward(ctx, rows, view, True), dtype).float().cpu()
         got_a.append(out[:na]); got_b.append(out[na:na + nb])
         at[2] += na; at[0] += nb
-    close(torch.cat(got_a), want_a, dtype, "request a")
-    close(torch.cat(got_b), want_b, dtype, "request b")
+    close(torch.cat(got_a), want_a, dtype, "request a", bf16=bf16)
+    close(torch.cat(got_b), want_b, dtype, "request b", bf16=bf16)
     assert float(state[1].abs().max()) == 0.0          # nobody's slot
 
 
