@@ -9,6 +9,7 @@ decode through the Python entry point, prefill of 2,048 tokens, and decode at ba
     python bench.py --design nufatar          # the same for the Nufatar decoder (beside Sapatar and Qwen2)
     python bench.py --design dugudra          # the same for the Dugudra decoder (beside Sapatar and Qwen2)
     python bench.py --design varivik          # the same for the Varivik decoder (beside Sapatar and Qwen2)
+    python bench.py --design bavetar          # the same for the Bavetar decoder (beside Dugudra and Qwen2)
 
 The default run has the layer sizes of the Qwen2.5-7B-sized benchmark configuration with
 random weights (N(0, 0.02), drawn on the device), a batch of 8 and a context of 4,096 tokens.
@@ -356,7 +357,7 @@ def workload_run(name: str, layers: int | None) -> dict:
 
 
 def design_run(args, pk: dict, pk_source: str) -> dict:
-    """``--design linurax|sapatar|nufatar|dugudra|varivik``: that decoder and the Qwen2 decoder at the layer sizes of the benchmark
+    """``--design linurax|sapatar|nufatar|dugudra|varivik|bavetar``: that decoder and the Qwen2 decoder at the layer sizes of the benchmark
     configuration (``--layers`` of them, default 8 here), random weights: a prompt step of 2,048 tokens, decode at
     batch 1 and ``--batch`` with ``--context`` keys, and the design's own kernels alone."""
     import torch
@@ -369,12 +370,14 @@ def design_run(args, pk: dict, pk_source: str) -> dict:
               "prefill_tokens": PREFILL_TOKENS, "peaks": pk, "peaks_source": pk_source, "dtype": "bf16",
               "data": "synthetic: random weights, uniform random token ids", "sizes": {}}
     like = {"linurax": db.linurax_config_like, "sapatar": db.sapatar_config_like, "nufatar": db.nufatar_config_like,
-            "dugudra": db.dugudra_config_like, "varivik": db.varivik_config_like}[args.design]
+            "dugudra": db.dugudra_config_like, "varivik": db.varivik_config_like, "bavetar": db.bavetar_config_like}[args.design]
     for name, qwen in sizes.items():
         entry = {}
         beside = [("qwen2", dict(qwen, num_hidden_layers=layers))]
         if args.design in ("nufatar", "dugudra", "varivik"):      # the closest design in the tree: windowed attention, matrix memories, experts
             beside.insert(0, ("sapatar", db.sapatar_config_like(qwen, layers)))
+        if args.design == "bavetar":       # the closest design: latent attention, a matrix state per head, routed experts
+            beside.insert(0, ("dugudra", db.dugudra_config_like(qwen, layers)))
         for design, config in [(args.design, like(qwen, layers))] + beside:
             model = db.build(config)
             t = db.step_times(model, args.batch, args.context, PREFILL_TOKENS, PAGE_SIZE)
@@ -392,6 +395,11 @@ def design_run(args, pk: dict, pk_source: str) -> dict:
                                        pk["hbm_gbs"], pk["bf16_tflops"], PAGE_SIZE)
         rows += db.sapatar_kernel_table(db.sapatar_config_like(BENCH_CONFIG, 4), args.batch, args.context, PREFILL_TOKENS,
                                         pk["hbm_gbs"], pk["bf16_tflops"])
+    elif args.design == "bavetar":
+        rows = db.bavetar_kernel_table(db.bavetar_config_like(BENCH_CONFIG, 4), args.batch, args.context, PREFILL_TOKENS,
+                                       pk["hbm_gbs"], pk["bf16_tflops"], PAGE_SIZE)
+        rows += db.dugudra_kernel_table(db.dugudra_config_like(BENCH_CONFIG, 4), args.batch, args.context, PREFILL_TOKENS,
+                                        pk["hbm_gbs"], pk["bf16_tflops"], PAGE_SIZE)
     elif args.design == "varivik":
         rows = db.varivik_kernel_table(db.varivik_config_like(BENCH_CONFIG, 4), args.batch, args.context, PREFILL_TOKENS,
                                        pk["hbm_gbs"], pk["bf16_tflops"], PAGE_SIZE, value_dims=(None, BENCH_CONFIG["head_dim"] // 2))
@@ -511,7 +519,7 @@ def main() -> int:
     ap.add_argument("--timeline", action="store_true",
                     help="record one decode step block by block on the device (kernels compiled with their recorder) "
                          "and print its launches in time order; for looking at, not a measurement")
-    ap.add_argument("--design", choices=["linurax", "sapatar", "nufatar", "dugudra", "varivik"], default=None,
+    ap.add_argument("--design", choices=["linurax", "sapatar", "nufatar", "dugudra", "varivik", "bavetar"], default=None,
                     help="another design beside the Qwen2 decoder at equal layer sizes: prompt and decode throughput of "
                          "both, and the design's own kernels with their rooflines (a record of its own; the default "
                          "workload and its JSON line are not touched)")

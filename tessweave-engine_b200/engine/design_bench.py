@@ -819,3 +819,153 @@ def varivik_kernel_table(config: dict, batch: int, context: int, prefill_tokens:
     if int(status) != 0:
         raise RuntimeError(f"a kernel reported status {int(status)} during the kernel table")
     return rows
+
+
+# ---------------------------------------------------------------------------
+# the Bavetar decoder
+# ---------------------------------------------------------------------------
+def bavetar_config_like(qwen: dict, layers: int) -> dict:
+    """A Bavetar config.json with the sizes of the Qwen2 configuration ``qwen``: layers [mamba2 + experts, latent
+    attention + dense, mamba2 + dense, latent attention + experts] in turn.  The recurrence is twice the residual width
+    in heads of 64 with states of 128, eight groups (as many parts in its norm) and four taps; the latent attention has
+    Qwen2's query heads of its head size and half as many rotated values more, a query latent of 1,536 and cached rows of
+    192 + 64 values; the dense feed-forward has as many weights in its two matrices as Qwen2's three; eight experts of a
+    quarter of Qwen2's feed-forward in four groups, three chosen from three of them."""
+    heads, dim, width, ff = (qwen[k] for k in ("num_attention_heads", "head_dim", "hidden_size", "intermediate_size"))
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 3, "scale": 1.5, "groups": {"count": 4, "keep": 3}}}
+    latent = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "q_rank": 1536, "kv_rank": 256 - dim // 2,
+              "scale": (dim + dim // 2) ** -0.5, "rot": {"dims": dim // 2, "base": qwen["rope_theta"]}}
+    mamba = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    pattern = [{"type": "mamba2", "mixer": mamba, "mlp": moe}, {"type": "latent_attention", "mixer": latent, "mlp": dense},
+               {"type": "mamba2", "mixer": mamba, "mlp": dense}, {"type": "latent_attention", "mixer": latent, "mlp": moe}]
+    return {"architecture": "Bavetar", "vocab": qwen["vocab_size"], "width": width, "norm": {"eps": qwen["rms_norm_eps"]},
+            "logit_scale": 0.5, "logit_softcap": 30.0, "layers": [pattern[i % 4] for i in range(layers)]}
+
+
+def bavetar_kernel_table(config: dict, batch: int, context: int, prefill_tokens: int, hbm_gbs: float, tflops: float,
+                         page_size: int = 16) -> list[dict]:
+    """The Bavetar kernels alone, each inside a CUDA graph with operands rotated beyond L2, for a decode step of
+    ``batch`` rows and a prompt step: latent attention (preparation, attention with a sink and gates), the convolution,
+    the state-space recurrence, the gated norm of parts, the norm of two deltas with two results, both feed-forwards.
+    fraction = max(bytes / HBM peak, FLOPs / tensor peak) / time."""
+    import tessweave_engine_b200 as tw
+    from ..config.bavetar_config import DenseConfig
+    from ..models.bavetar import feed_forward_spec, mixer_spec
+    from ..parts.base import DeltaPair
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    rt = Runtime(dev, bf)
+    cfg, _ = tw.resolve(config)
+    W = cfg.width
+    layer_of = {l.type: l for l in cfg.layers}
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    rows: list[dict] = []
+
+    def add(name, m, thunks, nbytes, flops, reps=4, note=""):
+        kernel = _kernels_of(thunks[0])
+        us = _graph_us(thunks, reps)
+        floor = max(nbytes / (hbm_gbs * 1e9), flops / (tflops * 1e12)) * 1e6
+        rows.append({"op": name, "rows": m, "kernel": kernel, "us": round(us, 2), "mbytes": round(nbytes / 1e6, 2),
+                     "gflop": round(flops / 1e9, 2), "floor_us": round(floor, 2), "frac": round(floor / us, 3),
+                     "bound": "hbm" if nbytes / (hbm_gbs * 1e9) >= flops / (tflops * 1e12) else "tensor", "note": note})
+
+    for m, phase in ((batch, "decode"), (prefill_tokens, "prefill")):
+        requests = batch if phase == "decode" else 1
+        per = m // requests
+        kv_tokens = context if phase == "decode" else m
+        ctx = _context(rt, Workspace(dev), status, [context - 1] * m if phase == "decode" else list(range(m)),
+                       [r for r in range(requests) for _ in range(per)], list(range(requests)), [r * per for r in range(requests)],
+                       [per] * requests, [context] * requests if phase == "decode" else [m])
+        # ---- latent attention
+        lat = build_part("mixer", mixer_spec(cfg, layer_of["latent_attention"]), rt)
+        _fill(lat)
+        Hq, Dl, blocks = lat.n_heads, lat.head_dim, -(-kv_tokens // page_size)
+        caches = []
+        for _ in range(_copies(requests * blocks * page_size * Dl * 2)):
+            cache = CacheManager([(lat.cache_need(), None)], page_size, requests * blocks, requests, kv_tokens, bf, dev, prefix_cache=False)
+            for g in cache.groups:
+                g.k.normal_(0, 0.5)
+            for _r in range(requests):
+                cache.ensure(cache.admit(None), kv_tokens)
+            cache.sync_tables()
+            caches.append(cache)
+        views = [c.view(0) for c in caches]
+        projs = [torch.randn(m, lat.in_width, device=dev, dtype=bf) for _ in range(_copies(m * lat.in_width * 2) if phase == "prefill" else 1)]
+        add(f"{phase}: latent norms + rotation + store + gates, query product, rotation, queries into the latent space", m,
+            [(lambda v=v, i=i: lat.prepare(ctx, projs[i % len(projs)], v, True)) for i, v in enumerate(views)],
+            m * (lat.in_width + lat.q_rank + Dl + Hq * (2 * lat.q_head + Dl)) * 2 + Hq * (lat.q_head * lat.q_rank + lat.q_head * Dl) * 2,
+            2.0 * m * Hq * lat.q_head * (lat.q_rank + Dl), note="the two products are the library's")
+        ql, gates = (t.clone() for t in lat.prepare(ctx, projs[0], views[0], True))
+        outs = [torch.empty(m, lat.q_size, device=dev, dtype=bf) for _ in range(2)]
+        if phase == "decode":
+            nbytes, flops = m * kv_tokens * Dl * 2 + m * 2 * lat.q_size * 2, 2.0 * m * Hq * 2 * Dl * kv_tokens
+        else:
+            nbytes, flops = m * (2 * lat.q_size + Dl) * 2, 2.0 * Hq * 2 * Dl * _visible_pairs(m, None)
+        add(f"{phase}: attention of {Hq} heads over {kv_tokens} cached rows of {Dl} values, sink, gates", m,
+            [(lambda v=v, i=i: lat._attend(ctx, outs[i % 2], ql, v, gate=gates)) for i, v in enumerate(views)], nbytes, flops,
+            reps=2 if phase == "prefill" else 4)
+        del caches, views, projs, lat, ql, outs, gates
+        torch.cuda.empty_cache()
+        # ---- the recurrence and what stands around it
+        mam = build_part("mixer", mixer_spec(cfg, layer_of["mamba2"]), rt)
+        _fill(mam)
+        H, N, Dv, C, taps = mam.n_heads, mam.key_dim, mam.value_dim, mam.conv_channels, mam.taps
+        sets = []
+        for _ in range(_copies(max(requests * mam.state_numel * 8, m * C * 6))):
+            sets.append((torch.randn(m, mam.row_size, device=dev, dtype=bf), torch.empty(m, C, device=dev), torch.zeros(requests, mam.state_numel, device=dev),
+                         torch.randn(m, H, device=dev), torch.empty(m, mam.v_size, device=dev), torch.empty(m, mam.v_size, device=dev, dtype=bf)))
+        moved = ctx.seq_q_len if phase == "decode" else None
+        add(f"{phase}: convolution of {taps} taps over {C} channels", m,
+            [(lambda s=s: ops.short_conv(s[1], s[0][:, mam.v_size:], mam.conv, s[2], mam.conv_offset, ctx.seq_of_token, ctx.seq_slot,
+                                         ctx.seq_q_start, m, bias=mam.conv_bias, move_single=moved)) for s in sets],
+            m * C * 6 + requests * C * (taps - 1) * 8, 0.0, reps=8)
+        a, b = mam.qk_size, mam.v_size
+        state_bytes = 2 * requests * H * N * Dv * 4
+        add(f"{phase}: state-space recurrence, {H} heads of {N} x {Dv}, {mam.n_groups} groups", m,
+            [(lambda s=s: mam.walk(ctx, s[1], s[3], StateView(s[2]), True)) for s in sets],
+            m * C * 4 + m * b * 4 + m * H * 4 + state_bytes, 0.0, reps=2 if phase == "prefill" else 8,
+            note=f"{4.0 * m * H * N * Dv / 1e9:.2f} GFLOP in the token-by-token form")
+        add(f"{phase}: gate and norm of {mam.norm_groups} parts", m,
+            [(lambda s=s: ops.gate_part_norm(s[5], s[4], mam.norm, s[0][:, :b], ops.GATE_SILU, 1e-6, m, mam.norm_groups)) for s in sets],
+            m * b * 8, 0.0, reps=8)
+        del sets, mam
+        torch.cuda.empty_cache()
+        # ---- the norm between layers: two deltas in, two results out
+        norms = [build_part("norm", tw.PartSpec("rmsnorm", {"size": W, "eps": cfg.norm_eps, "weight_name": ""}), rt) for _ in range(2)]
+        for norm in norms:
+            _fill(norm)
+        sets = [(torch.randn(m, W, device=dev), *(torch.randn(m, W, device=dev, dtype=bf) for _ in range(4))) for _ in range(_copies(m * W * 16))]
+        add(f"{phase}: residual add of two deltas + two RMSNorms", m,
+            [(lambda s=s: norms[0].apply_twice(ctx, s[3], norms[1], s[4], s[0], DeltaPair(s[1], s[2]), m)) for s in sets],
+            m * W * (4 + 4 + 2 * 4), 0.0, reps=8)
+        del sets
+        # ---- feed-forwards
+        hs = [torch.randn(m, W, device=dev, dtype=bf) for _ in range(4)]
+        mlp = next(l.mlp for l in cfg.layers if isinstance(l.mlp, DenseConfig))
+        parts = [build_part("feed_forward", feed_forward_spec(cfg, mlp), rt) for _ in range(2)]
+        for part in parts:
+            _fill(part)
+        add(f"{phase}: dense feed-forward (up, square of relu, down)", m,
+            [(lambda p=p, i=i: p.forward(ctx, hs[i % 4])) for i, p in enumerate(parts)],
+            2 * mlp.ff * W * 2 + m * (2 * W + 2 * mlp.ff) * 2, 2.0 * m * 2 * mlp.ff * W, reps=3)
+        del parts
+        torch.cuda.empty_cache()
+        mlp = next(l.mlp for l in cfg.layers if l.mlp is not None and not isinstance(l.mlp, DenseConfig))
+        parts = []
+        for _ in range(_copies(mlp.experts * 3 * mlp.ff * W * 2) if phase == "decode" else 2):
+            part = build_part("feed_forward", feed_forward_spec(cfg, mlp), rt)
+            _fill(part)
+            part.w_router.normal_(0, 0.5)
+            parts.append(part)
+        touched = min(mlp.experts, m * mlp.top)
+        add(f"{phase}: router over {mlp.experts} experts in {mlp.groups[0]} groups, {mlp.top} chosen", m,
+            [(lambda p=p, i=i: p.route(ctx, hs[i % 4])) for i, p in enumerate(parts)], m * W * 2 + mlp.experts * W * 2, 0.0, reps=8)
+        add(f"{phase}: router, the chosen experts and the weighted sum", m,
+            [(lambda p=p, i=i: p.forward(ctx, hs[i % 4])) for i, p in enumerate(parts)],
+            touched * 3 * mlp.ff * W * 2 + m * W * 4, 2.0 * m * mlp.top * 3 * mlp.ff * W, reps=2,
+            note="bytes: the matrices of the experts a step of this size touches at most, once")
+        del parts, hs
+        torch.cuda.empty_cache()
+    if int(status) != 0:
+        raise RuntimeError(f"a kernel reported status {int(status)} during the kernel table")
+    return rows

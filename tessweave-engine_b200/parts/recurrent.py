@@ -519,7 +519,7 @@ class Mamba2(MatrixStateMixer):
     def recur(self, ctx: StepContext, h: torch.Tensor, cache: StateView, write_cache: bool):
         """(y fp32 [rows, heads * value_dim], the projected rows [z | x | B | C]); the requests' states move on."""
         n, ws = ctx.n_tokens, ctx.workspace
-        b, a, C = self.v_size, self.qk_size, self.conv_channels
+        b, C = self.v_size, self.conv_channels
         proj = linear(ctx, "mamba2.in", h, self.w_in[:self.row_size])
         step = linear(ctx, "mamba2.step", h, self.w_in[self.row_size:], out_dtype=torch.float32)
         mixed = proj[:, b:]
@@ -530,6 +530,11 @@ class Mamba2(MatrixStateMixer):
             # (a request that brings one row had its state moved on by the convolution itself)
             ops.short_conv_state(mixed, self.taps, C, cache.state, self.conv_offset, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
                                  ctx.n_seqs, skip_single=True)
+        return self.walk(ctx, ready, step, cache, write_cache), proj
+
+    def walk(self, ctx: StepContext, ready: torch.Tensor, step: torch.Tensor, cache: StateView, write_cache: bool) -> torch.Tensor:
+        """y of the rows [x | B | C], which are convolved and activated, and their projected step sizes."""
+        b, a = self.v_size, self.qk_size
         raw, _ = self._recur(ctx, ready[:, b + a:], ready[:, b:b + a], ready[:, :b], cache, write_cache, pre=step,
                              p0=self.rate_log, p1=self.dt_bias, p2=self.skip, qk_group=self.n_heads // self.n_groups)
-        return raw, proj
+        return raw
