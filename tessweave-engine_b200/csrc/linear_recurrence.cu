@@ -21,7 +21,7 @@
 //                      exp(logsigmoid(z + b) / tau); 1 / tau arrives in `cap`, b in p0
 //   TW_REC_SSD         S <- e^(-r_h dt) S + dt k v^T         o = S^T q + u_h v  (the state-space form of linear attention)
 //                      dt = softplus(d + b_h) per head from the projected d, r_h = e^(A_h); A in p0, b in p1, the skip u
-//                      in p2.  q, k and v arrive as fp32 rows (here: convolved and activated), heads may share q and k
+//                      in p2.  q, k and v arrive ready to use (here: convolved and activated), heads may share q and k
 //
 // One block per (head, request, slice of the columns of S): a thread owns a column of S in registers (TW_DK
 // values, a compile-time size; where that size is a multiple of 16 four or eight lanes share a column, a quarter or
@@ -567,8 +567,9 @@ TW_EXPORT int tw_linear_recurrence(int mode, float* out, float* den, const void*
         if (!f32 || !bpre || !wpre || !p0 || !p1) return (int)cudaErrorInvalidValue;     // its rows are prepared in fp32 in every run type
         return launch_recurrence<float, TW_REC_DELTA>(a, n_seqs, lp, stream);
     case TW_REC_SSD:
-        if (!f32 || !wpre || !p0 || !p1 || !p2) return (int)cudaErrorInvalidValue;
-        return launch_recurrence<float, TW_REC_SSD>(a, n_seqs, lp, stream);
+        if (!wpre || !p0 || !p1 || !p2) return (int)cudaErrorInvalidValue;
+        return f32 ? launch_recurrence<float, TW_REC_SSD>(a, n_seqs, lp, stream)
+                   : launch_recurrence<__nv_bfloat16, TW_REC_SSD>(a, n_seqs, lp, stream);
     }
     return (int)cudaErrorInvalidValue;
 }

@@ -1507,14 +1507,14 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
     ``channel_decay``, else [rows, heads]), ``p0`` the log of each head's rate [heads], ``p1`` the decay's bias (of
     ``pre``'s width), ``write_pre`` the write strength before its sigmoid, fp32 [rows, heads]; ``qk_group`` value heads
     share a head of q and k.  Gated linear attention takes ``pre`` the projected decay [rows, heads * key_dim], ``p0`` its
-    bias and ``cap`` the exponent 1 / tau of the sigmoid.  The state-space rule takes fp32 q, k, v that are ready to use,
+    bias and ``cap`` the exponent 1 / tau of the sigmoid.  The state-space rule takes q, k, v that are ready to use,
     ``pre`` the projected step size [rows, heads], ``p0`` the log of each head's rate, ``p1`` the step size's bias and ``p2``
     the skip, each [heads]; ``qk_group`` as in the delta rule."""
     _cuda(out, den, q, k, v, state, positions, seq_slot, seq_q_start, seq_q_len, pre, p0, p1, p2, inv_freq, tail, write_pre)
-    _need(mode != RECURRENCE_SSD or (q.dtype == torch.float32 and pre is not None and pre.stride(1) == 1 and pre.shape[1] >= heads
+    _need(mode != RECURRENCE_SSD or (pre is not None and pre.stride(1) == 1 and pre.shape[1] >= heads
                                      and all(p is not None and p.numel() == heads and p.is_contiguous() for p in (p0, p1, p2))
                                      and qk_group >= 1 and heads % qk_group == 0),
-          "recurrence: the state-space rule needs fp32 rows, a projected step size, and a rate, bias and skip per head")
+          "recurrence: the state-space rule needs a projected step size, and a rate, bias and skip per head")
     if mode == RECURRENCE_DELTA:
         width = heads * key_dim if channel_decay else heads
         _need(q.dtype == torch.float32 and pre is not None and p0 is not None and p1 is not None and write_pre is not None
@@ -1544,6 +1544,57 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
         _ptr(positions), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), c_int(n_seqs), c_int(heads), c_int(key_dim),
         c_int(value_dim), c_int(1 if write_state else 0), c_int(max_q_len), c_int(dtype_code(q.dtype)), _stream())
     _check(code, "linear_recurrence")
+
+
+STATE_SPACE_CHUNK_STATES = (16, 32, 64, 128, 256)
+STATE_SPACE_CHUNK_MIN_TOKENS = 17       # portions of a chunk of the token-by-token kernel and less stay there
+
+
+def state_space_chunks_supported(dtype: torch.dtype, state_dim: int, value_dim: int, channels: int, max_q_len: int) -> bool:
+    """Whether a step whose longest portion has ``max_q_len`` tokens runs the state-space recurrence in chunks on the
+    tensor cores: bfloat16 rows, state sizes and values the tiles take, and more than a few tokens.
+    TESSWEAVE_STATE_SPACE=tokens|chunks forces one of the two (the latter only for sizes the kernel takes)."""
+    import os
+    if dtype != torch.bfloat16 or state_dim not in STATE_SPACE_CHUNK_STATES or value_dim % 16 or channels % 8:
+        return False
+    forced = os.environ.get("TESSWEAVE_STATE_SPACE")
+    if forced in ("tokens", "chunks"):
+        return forced == "chunks"
+    return max_q_len >= STATE_SPACE_CHUNK_MIN_TOKENS
+
+
+def state_space_slice(heads: int, n_seqs: int, value_dim: int, sms: int = 148) -> int:
+    """Values of a head that a block of the chunked kernel serves: 64 where they divide, less where that would leave more
+    than half of the SMs without a block (a slice repeats the products that do not depend on the values)."""
+    sizes = [d for d in (64, 32, 16) if value_dim % d == 0]
+    for d in sizes:
+        if heads * n_seqs * (value_dim // d) > sms // 2 or d == sizes[-1]:
+            return d
+    raise KernelError(f"the chunked state-space kernel takes values in multiples of 16, not {value_dim}")
+
+
+def state_space_chunks(out: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pre: torch.Tensor, rate_log: torch.Tensor,
+                       dt_bias: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, seq_slot: torch.Tensor, seq_q_start: torch.Tensor,
+                       seq_q_len: torch.Tensor, n_seqs: int, heads: int, state_dim: int, value_dim: int, qk_group: int,
+                       write_state: bool = True, slice_dim: int | None = None) -> None:
+    """``linear_recurrence`` with the state-space rule over portions of a prompt, 64 tokens at a time on the tensor cores
+    (csrc/state_space.cu): same operands and state, bfloat16 q, k, v."""
+    _cuda(out, q, k, v, pre, rate_log, dt_bias, skip, state, seq_slot, seq_q_start, seq_q_len)
+    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == heads * value_dim, "state_space_chunks: out must be fp32 [rows, H * Dv]")
+    _need(all(t.dtype == torch.bfloat16 and t.stride(1) == 1 for t in (q, k, v)) and heads % qk_group == 0
+          and q.shape[1] == k.shape[1] == heads // qk_group * state_dim and v.shape[1] == heads * value_dim,
+          "state_space_chunks: q, k, v must be bf16 rows of their heads")
+    _need(pre.dtype == torch.float32 and pre.stride(1) == 1 and pre.shape[1] >= heads
+          and all(p.dtype == torch.float32 and p.numel() == heads and p.is_contiguous() for p in (rate_log, dt_bias, skip)),
+          "state_space_chunks: fp32 step sizes [rows, H] and constants [H]")
+    _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1 and state.shape[1] >= heads * state_dim * value_dim,
+          "state_space_chunks: the state must be fp32 [slots, numel]")
+    code = _fn("state_space", "tw_state_space_chunks", {"TW_DK": state_dim})(
+        _ptr(out), _ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)), _ptr(pre), c_int(pre.stride(0)),
+        _ptr(rate_log), _ptr(dt_bias), _ptr(skip), _ptr(state), ctypes.c_longlong(state.stride(0)), _ptr(seq_slot), _ptr(seq_q_start),
+        _ptr(seq_q_len), c_int(n_seqs), c_int(heads), c_int(state_dim), c_int(value_dim), c_int(qk_group),
+        c_int(slice_dim or state_space_slice(heads, n_seqs, value_dim)), c_int(1 if write_state else 0), _stream())
+    _check(code, "state_space_chunks")
 
 
 GATE_NONE, GATE_SILU, GATE_SIGMOID = 0, 1, 2
@@ -1906,7 +1957,7 @@ def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch
                seq_of_token: torch.Tensor, seq_slot: torch.Tensor, seq_q_start: torch.Tensor, n_rows: int,
                unit_heads: int = 0, unit_dim: int = 0, scaled_heads: int = 0, head_scale: float = 1.0, unit_eps: float = 0.0,
                move_single: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
-    """out[t, c] = silu([bias[c] +] sum_j w[c, j] x[t - (taps - 1) + j, c]) in fp32 [rows, channels]: a causal convolution over the
+    """out[t, c] = silu([bias[c] +] sum_j w[c, j] x[t - (taps - 1) + j, c]) as fp32 or bf16 rows [rows, channels]: a causal convolution over the
     rows of each request, per channel (the last tap is the row's own).  The taps - 1 rows before a request's first row of
     this step are read from its state (fp32, [channels, taps - 1] at ``state_offset``; zeros at a request's start).  The
     first ``unit_heads`` heads of ``unit_dim`` channels are then scaled to x / sqrt(sum x^2 + unit_eps), the first
@@ -1917,8 +1968,8 @@ def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == w.shape[0]), "short_conv: the bias must be fp32 [channels]")
     _need(move_single is None or move_single.dtype == torch.int32, "short_conv: the row counts must be int32")
     channels, taps = w.shape
-    _need(out.dtype == torch.float32 and out.is_contiguous() and out.shape[1] == channels and out.shape[0] >= n_rows,
-          "short_conv: the result must be contiguous fp32 [rows, channels]")
+    _need(out.dtype in (torch.float32, x.dtype) and out.is_contiguous() and out.shape[1] == channels and out.shape[0] >= n_rows,
+          "short_conv: the result must be contiguous [rows, channels], in fp32 or x's type")
     _need(x.stride(1) == 1 and x.shape[1] >= channels and x.shape[0] >= n_rows, "short_conv: bad input rows")
     _need(w.dtype == torch.float32 and w.is_contiguous() and 1 <= taps <= SHORT_CONV_MAX_TAPS, "short_conv: taps must be fp32 [channels, 1..17]")
     _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
@@ -1928,7 +1979,8 @@ def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch
         _ptr(out), _ptr(x), c_int(x.stride(0)), _ptr(w), _ptr(bias), c_int(taps), _ptr(state), ctypes.c_longlong(state.stride(0)),
         ctypes.c_longlong(state_offset), _ptr(seq_of_token), _ptr(seq_slot), _ptr(seq_q_start), _ptr(move_single),
         c_int(0 if move_single is None else 1), c_int(n_rows), c_int(channels),
-        c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(head_scale), c_float(unit_eps), c_int(dtype_code(x.dtype)), _stream())
+        c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(head_scale), c_float(unit_eps), c_int(dtype_code(x.dtype)),
+        c_int(dtype_code(out.dtype)), _stream())
     _check(code, "short_conv")
 
 

@@ -435,11 +435,11 @@ TW_EXPORT int tw_tanh_rows(void* x, long long count, int dtype, cudaStream_t str
 // The taps - 1 rows before a request's first row of this step come from the request's state (fp32, channel-major:
 // state[offset + c * (taps - 1) + j], j = 0 the oldest), which tw_short_conv_state moves on afterwards.  Behind the
 // convolution the first `unit_heads` heads of `unit_dim` channels are scaled to unit length, x / sqrt(sum x^2 + unit_eps),
-// the first `scaled_heads` of them also multiplied by `head_scale`.  One block per row; the result is fp32.
+// the first `scaled_heads` of them also multiplied by `head_scale`.  One block per row; the result is fp32, or (OT) rounded to bf16.
 // ---------------------------------------------------------------------------
-template <typename T>
+template <typename T, typename OT>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias, int taps,
+short_conv_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias, int taps,
                   float* __restrict__ state, long long state_stride, long long state_offset,
                   const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                   const int* __restrict__ seq_q_len, int move_single, int channels, int chunk, int unit_heads, int unit_dim,
@@ -470,7 +470,7 @@ short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride
     }
     __syncthreads();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
-    float* orow = out + (size_t)row * channels;
+    OT* orow = out + (size_t)row * channels;
     const int unit_end = unit_heads * unit_dim;
     if (c0 < unit_end) {
         const int h0 = c0 / unit_dim, h1 = min(unit_heads, (c1 + unit_dim - 1) / unit_dim);
@@ -480,10 +480,10 @@ short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride
             for (int d = lane; d < unit_dim; d += 32) ss += y[d] * y[d];
             ss = tw_warp_sum(ss);
             const float f = (head < scaled_heads ? head_scale : 1.0f) / sqrtf(ss + unit_eps);
-            for (int d = lane; d < unit_dim; d += 32) orow[head * unit_dim + d] = y[d] * f;
+            for (int d = lane; d < unit_dim; d += 32) orow[head * unit_dim + d] = tw_from_float<OT>(y[d] * f);
         }
     }
-    for (int c = max(c0, unit_end) + threadIdx.x; c < c1; c += blockDim.x) orow[c] = sy[c - c0];
+    for (int c = max(c0, unit_end) + threadIdx.x; c < c1; c += blockDim.x) orow[c] = tw_from_float<OT>(sy[c - c0]);
 }
 
 // The same for steps with many rows and at most TW_CONV_FAST_TAPS taps: a block serves `rows_per_block` consecutive rows
@@ -492,9 +492,9 @@ short_conv_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride
 // are added in the same order as above, so both kernels give the same bits.
 #define TW_CONV_FAST_TAPS 4
 #define TW_CONV_ROWS 8
-template <typename T, int TAPS>
+template <typename T, typename OT, int TAPS>
 __global__ void __launch_bounds__(256)
-short_conv_rows_kernel(float* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w,
+short_conv_rows_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w,
                        const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
                        const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                        const int* __restrict__ seq_q_len, int move_single, int n_rows, int channels, int chunk, int unit_heads,
@@ -558,16 +558,92 @@ short_conv_rows_kernel(float* __restrict__ out, const T* __restrict__ x, int x_s
         for (int d = lane; d < unit_dim; d += 32) ss += y[d] * y[d];
         ss = tw_warp_sum(ss);
         const float f = (head < scaled_heads ? head_scale : 1.0f) / sqrtf(ss + unit_eps);
-        float* orow = out + (size_t)(row0 + i) * channels;
-        for (int d = lane; d < unit_dim; d += 32) orow[head * unit_dim + d] = y[d] * f;
+        OT* orow = out + (size_t)(row0 + i) * channels;
+        for (int d = lane; d < unit_dim; d += 32) orow[head * unit_dim + d] = tw_from_float<OT>(y[d] * f);
     }
     const int p0 = max(c0, unit_end);
     if (p0 < c1) {
         const int span = c1 - p0;
         for (int e = threadIdx.x; e < nr * span; e += blockDim.x) {
             const int i = e / span, c = p0 + (e - i * span);
-            if (seq_of_token[row0 + i] >= 0) out[(size_t)(row0 + i) * channels + c] = sy[i * chunk + (c - c0)];
+            if (seq_of_token[row0 + i] >= 0) out[(size_t)(row0 + i) * channels + c] = tw_from_float<OT>(sy[i * chunk + (c - c0)]);
         }
+    }
+}
+
+// bf16 in and out, no unit heads, four taps or fewer, channels in groups of eight on 16-byte boundaries: a thread serves
+// eight channels of TW_CONV_WIDE_ROWS consecutive rows with 16-byte accesses, the inputs of the rows before in registers.
+#define TW_CONV_WIDE_ROWS 16
+#define TW_CONV_WIDE_THREADS 128
+__device__ __forceinline__ void tw_unpack8(uint4 raw, float (&f)[8]) {
+    const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const float2 u = __bfloat1622float2(p[e]);
+        f[2 * e] = u.x; f[2 * e + 1] = u.y;
+    }
+}
+template <int TAPS>
+__global__ void __launch_bounds__(TW_CONV_WIDE_THREADS)
+short_conv_wide_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, int x_stride, const float* __restrict__ w,
+                       const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
+                       const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
+                       const int* __restrict__ seq_q_len, int move_single, int n_rows, int channels) {
+    constexpr int R = TW_CONV_WIDE_ROWS, P = TAPS - 1;
+    tw_grid_wait();
+    tw_grid_launch_dependents();
+    const int c = (blockIdx.y * TW_CONV_WIDE_THREADS + threadIdx.x) * 8;
+    if (c >= channels) return;
+    const int row0 = blockIdx.x * R, nr = min(R, n_rows - row0);
+    float wt[8][TAPS], b[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c + e) * TAPS + j];
+        b[e] = bias ? bias[c + e] : 0.f;
+    }
+    uint4 xr[P + R];                     // the rows before (whichever request they belong to), then the block's own
+#pragma unroll
+    for (int i = 0; i < P + R; ++i) {
+        const int rr = row0 - P + i;
+        xr[i] = rr >= 0 && i - P < nr ? *reinterpret_cast<const uint4*>(x + (size_t)rr * x_stride + c) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        if (i >= nr) break;
+        const int row = row0 + i;
+        const int s = seq_of_token[row];
+        if (s < 0) continue;
+        const int r = row - seq_q_start[s];          // rows of this request before this one in the step
+        float acc[8], in[TAPS][8];
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) tw_unpack8(xr[i + j], in[j]);
+        if (r < P) {                                 // taps that reach into what the request's state keeps
+            float* tail = state + (size_t)seq_slot[s] * state_stride + state_offset + (size_t)c * P;
+            const bool move = move_single && seq_q_len[s] == 1;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+#pragma unroll
+                for (int j = 0; j < P; ++j)
+                    if (P - j > r) in[j][e] = tail[e * P + r + j];
+                if (move) {
+#pragma unroll
+                    for (int j = 1; j < TAPS; ++j) tail[e * P + j - 1] = in[j][e];
+                }
+            }
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            acc[e] = b[e];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc[e] += wt[e][j] * in[j][e];
+            acc[e] = acc[e] / (1.0f + expf(-acc[e]));
+        }
+        uint4 packed;
+        __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&packed);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) q[e] = __floats2bfloat162_rn(acc[2 * e], acc[2 * e + 1]);
+        *reinterpret_cast<uint4*>(out + (size_t)row * channels + c) = packed;
     }
 }
 
@@ -594,17 +670,30 @@ __global__ void short_conv_state_kernel(const T* __restrict__ x, int x_stride, i
     for (int j = 0; j < keep; ++j) tail[j] = fresh[j];
 }
 
-template <typename T>
-static int launch_short_conv(float* out, const T* x, int x_stride, const float* w, const float* bias, int taps, float* state, long long state_stride,
+template <typename T, typename OT>
+static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, const float* bias, int taps, float* state, long long state_stride,
                              long long state_offset, const int* seq_of_token, const int* seq_slot, const int* seq_q_start,
                              const int* seq_q_len, int move_single, int n_rows, int channels, int unit_heads, int unit_dim,
                              int scaled_heads, float head_scale, float unit_eps, cudaStream_t stream) {
+    if constexpr (sizeof(T) == 2 && sizeof(OT) == 2) {
+        if (unit_heads == 0 && n_rows >= 4 * TW_CONV_WIDE_ROWS && taps >= 2 && taps <= 4 && (channels & 7) == 0 && (x_stride & 7) == 0
+            && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
+            const dim3 wgrid((n_rows + TW_CONV_WIDE_ROWS - 1) / TW_CONV_WIDE_ROWS, (channels / 8 + TW_CONV_WIDE_THREADS - 1) / TW_CONV_WIDE_THREADS);
+#define TW_CONV_WIDE_LAUNCH(TAPS)                                                                                                 \
+            return tw_launch(short_conv_wide_kernel<TAPS>, wgrid, dim3(TW_CONV_WIDE_THREADS), 0, stream, 1, out, x, x_stride, w, bias,  \
+                             state, state_stride, state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels);
+            if (taps == 2) { TW_CONV_WIDE_LAUNCH(2) }
+            if (taps == 3) { TW_CONV_WIDE_LAUNCH(3) }
+            TW_CONV_WIDE_LAUNCH(4)
+#undef TW_CONV_WIDE_LAUNCH
+        }
+    }
     // about 512 channels per block, in whole unit heads while there are any (a head larger than that has a block of its own)
     int chunk = 512;
     if (unit_heads > 0 && unit_dim > 0) chunk = unit_dim * (unit_dim >= 512 ? 1 : 512 / unit_dim);
     const size_t smem = (size_t)chunk * sizeof(float);
     if (smem > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(short_conv_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        const cudaError_t e = cudaFuncSetAttribute(short_conv_kernel<T, OT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
     if (n_rows >= 8 * TW_CONV_ROWS && taps <= TW_CONV_FAST_TAPS && smem * TW_CONV_ROWS <= 96 * 1024) {
@@ -613,11 +702,11 @@ static int launch_short_conv(float* out, const T* x, int x_stride, const float* 
 #define TW_CONV_ROWS_LAUNCH(TAPS)                                                                                                \
         {                                                                                                                        \
             if (rsmem > 48 * 1024) {                                                                                             \
-                const cudaError_t e = cudaFuncSetAttribute(short_conv_rows_kernel<T, TAPS>,                                      \
+                const cudaError_t e = cudaFuncSetAttribute(short_conv_rows_kernel<T, OT, TAPS>,                                      \
                                                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rsmem);             \
                 if (e != cudaSuccess) return (int)e;                                                                             \
             }                                                                                                                    \
-            return tw_launch(short_conv_rows_kernel<T, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, bias, state, \
+            return tw_launch(short_conv_rows_kernel<T, OT, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, bias, state, \
                              state_stride, state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows,   \
                              channels, chunk, unit_heads, unit_dim, scaled_heads, head_scale, unit_eps);                         \
         }
@@ -630,25 +719,29 @@ static int launch_short_conv(float* out, const T* x, int x_stride, const float* 
 #undef TW_CONV_ROWS_LAUNCH
     }
     const dim3 grid(n_rows, (channels + chunk - 1) / chunk);
-    return tw_launch(short_conv_kernel<T>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, bias, taps, state, state_stride,
+    return tw_launch(short_conv_kernel<T, OT>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, bias, taps, state, state_stride,
                      state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, channels, chunk, unit_heads,
                      unit_dim, scaled_heads, head_scale, unit_eps);
 }
 
 // seq_q_len with move_single: requests that bring one row have their state moved on by this kernel (and
 // tw_short_conv_state is then told to skip them).
-TW_EXPORT int tw_short_conv(float* out, const void* x, int x_stride, const float* w, const float* bias, int taps, float* state,
+TW_EXPORT int tw_short_conv(void* out, const void* x, int x_stride, const float* w, const float* bias, int taps, float* state,
                             long long state_stride, long long state_offset, const int* seq_of_token, const int* seq_slot,
                             const int* seq_q_start, const int* seq_q_len, int move_single, int n_rows, int channels,
                             int unit_heads, int unit_dim, int scaled_heads, float head_scale, float unit_eps, int dtype,
-                            cudaStream_t stream) {
+                            int out_dtype, cudaStream_t stream) {
     if (n_rows <= 0 || channels <= 0) return 0;
     if (taps < 1 || taps > 17 || unit_heads * unit_dim > channels || (move_single && !seq_q_len)) return (int)cudaErrorInvalidValue;
     if (dtype == TW_F32)
-        return launch_short_conv<float>(out, (const float*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token,
+        return out_dtype != TW_F32 ? (int)cudaErrorInvalidValue : launch_short_conv<float, float>((float*)out, (const float*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token,
                                         seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels, unit_heads, unit_dim,
                                         scaled_heads, head_scale, unit_eps, stream);
-    return launch_short_conv<__nv_bfloat16>(out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset,
+    if (out_dtype != TW_F32)
+        return launch_short_conv<__nv_bfloat16, __nv_bfloat16>(
+            (__nv_bfloat16*)out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token, seq_slot,
+            seq_q_start, seq_q_len, move_single, n_rows, channels, unit_heads, unit_dim, scaled_heads, head_scale, unit_eps, stream);
+    return launch_short_conv<__nv_bfloat16, float>((float*)out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset,
                                             seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels,
                                             unit_heads, unit_dim, scaled_heads, head_scale, unit_eps, stream);
 }

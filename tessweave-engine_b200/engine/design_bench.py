@@ -911,20 +911,20 @@ def bavetar_kernel_table(config: dict, batch: int, context: int, prefill_tokens:
         _fill(mam)
         H, N, Dv, C, taps = mam.n_heads, mam.key_dim, mam.value_dim, mam.conv_channels, mam.taps
         sets = []
-        for _ in range(_copies(max(requests * mam.state_numel * 8, m * C * 6))):
-            sets.append((torch.randn(m, mam.row_size, device=dev, dtype=bf), torch.empty(m, C, device=dev), torch.zeros(requests, mam.state_numel, device=dev),
+        for _ in range(_copies(max(requests * mam.state_numel * 8, m * C * 4))):
+            sets.append((torch.randn(m, mam.row_size, device=dev, dtype=bf), torch.empty(m, C, device=dev, dtype=bf), torch.zeros(requests, mam.state_numel, device=dev),
                          torch.randn(m, H, device=dev), torch.empty(m, mam.v_size, device=dev), torch.empty(m, mam.v_size, device=dev, dtype=bf)))
         moved = ctx.seq_q_len if phase == "decode" else None
         add(f"{phase}: convolution of {taps} taps over {C} channels", m,
             [(lambda s=s: ops.short_conv(s[1], s[0][:, mam.v_size:], mam.conv, s[2], mam.conv_offset, ctx.seq_of_token, ctx.seq_slot,
                                          ctx.seq_q_start, m, bias=mam.conv_bias, move_single=moved)) for s in sets],
-            m * C * 6 + requests * C * (taps - 1) * 8, 0.0, reps=8)
+            m * C * 4 + requests * C * (taps - 1) * 8, 0.0, reps=8)
         a, b = mam.qk_size, mam.v_size
         state_bytes = 2 * requests * H * N * Dv * 4
         add(f"{phase}: state-space recurrence, {H} heads of {N} x {Dv}, {mam.n_groups} groups", m,
             [(lambda s=s: mam.walk(ctx, s[1], s[3], StateView(s[2]), True)) for s in sets],
-            m * C * 4 + m * b * 4 + m * H * 4 + state_bytes, 0.0, reps=2 if phase == "prefill" else 8,
-            note=f"{4.0 * m * H * N * Dv / 1e9:.2f} GFLOP in the token-by-token form")
+            m * C * 2 + m * b * 4 + m * H * 4 + state_bytes, 0.0 if phase == "decode" else 4.0 * m * H * N * Dv, reps=2 if phase == "prefill" else 8,
+            note="FLOPs of the token-by-token form")
         add(f"{phase}: gate and norm of {mam.norm_groups} parts", m,
             [(lambda s=s: ops.gate_part_norm(s[5], s[4], mam.norm, s[0][:, :b], ops.GATE_SILU, 1e-6, m, mam.norm_groups)) for s in sets],
             m * b * 8, 0.0, reps=8)

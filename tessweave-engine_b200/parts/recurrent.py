@@ -523,7 +523,7 @@ class Mamba2(MatrixStateMixer):
         proj = linear(ctx, "mamba2.in", h, self.w_in[:self.row_size])
         step = linear(ctx, "mamba2.step", h, self.w_in[self.row_size:], out_dtype=torch.float32)
         mixed = proj[:, b:]
-        ready = ws.get("mamba2.ready", (n, C), torch.float32)
+        ready = ws.get("mamba2.ready", (n, C), self.runtime.dtype)
         ops.short_conv(ready, mixed, self.conv, cache.state, self.conv_offset, ctx.seq_of_token, ctx.seq_slot, ctx.seq_q_start, n,
                        move_single=ctx.seq_q_len if write_cache else None, bias=self.conv_bias)
         if write_cache and self.taps > 1 and not ctx.decode_only:
@@ -533,8 +533,16 @@ class Mamba2(MatrixStateMixer):
         return self.walk(ctx, ready, step, cache, write_cache), proj
 
     def walk(self, ctx: StepContext, ready: torch.Tensor, step: torch.Tensor, cache: StateView, write_cache: bool) -> torch.Tensor:
-        """y of the rows [x | B | C], which are convolved and activated, and their projected step sizes."""
+        """y of the rows [x | B | C], which are convolved and activated, and their projected step sizes: portions of a
+        prompt in chunks on the tensor cores (bfloat16, sizes that kernel takes), everything else token by token."""
         b, a = self.v_size, self.qk_size
+        if (ops.state_space_chunks_supported(ready.dtype, self.key_dim, self.value_dim, self.conv_channels, ctx.max_q_len)
+                and self.state_numel % 2 == 0):
+            raw = ctx.workspace.get("recurrence.raw", (ctx.n_tokens, b), torch.float32)
+            ops.state_space_chunks(raw, ready[:, b + a:], ready[:, b:b + a], ready[:, :b], step, self.rate_log, self.dt_bias, self.skip,
+                                   cache.state, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len, ctx.n_seqs, self.n_heads, self.key_dim,
+                                   self.value_dim, self.n_heads // self.n_groups, write_cache)
+            return raw
         raw, _ = self._recur(ctx, ready[:, b + a:], ready[:, b:b + a], ready[:, :b], cache, write_cache, pre=step,
                              p0=self.rate_log, p1=self.dt_bias, p2=self.skip, qk_group=self.n_heads // self.n_groups)
         return raw

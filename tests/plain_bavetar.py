@@ -96,12 +96,15 @@ def state_space_recurrence(x, b, c, dt, rate, skip):
     return y
 
 
-def mixer_mamba2(h, w, p, m, eps):
+def mixer_mamba2(h, w, p, m, eps, stored=lambda t: t):
+    """``stored``: what is done to the projected rows (without the step sizes) and to the convolved rows between two steps
+    of the computation -- nothing, or a rounding to the type they are kept in."""
     T = h.shape[0]
     H, Dv, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
     inner = H * Dv
     z, xbc, dt = torch.split(h @ w[p + "in"].T, [inner, inner + 2 * G * N, H], dim=-1)
-    xbc = causal_convolution(xbc, w[p + "conv"], w[p + "conv.b"])
+    z, xbc = stored(z), stored(xbc)
+    xbc = stored(causal_convolution(xbc, w[p + "conv"], w[p + "conv.b"]))
     x, b, c = torch.split(xbc, [inner, G * N, G * N], dim=-1)
     per = H // G
     b = b.reshape(T, G, N).repeat_interleave(per, dim=1)

@@ -248,6 +248,66 @@ def test_state_space_mixer_alone(dtype, shape):
     run_state_mixer(rt, mixer, hidden, lambda h, pos: plain.mixer_mamba2(h, wd, "p.", layer["mixer"], 1e-5))
 
 
+def stored_as(dtype):
+    """The rounding of rows kept in ``dtype``, for the plain mixer: where sums over keys cancel (a state of one loud token, a
+    step size of a hundred) rounding the rows alone moves an output by several per cent."""
+    return (lambda t: t) if dtype == torch.float32 else (lambda t: t.to(torch.bfloat16).double())
+
+
+def walk_by_hand(x, b, c, dt, rate, skip, S):
+    """The recurrence from a given state, in float64: (y, the state behind the last token)."""
+    y = torch.empty_like(x)
+    for t in range(x.shape[0]):
+        S = torch.exp(-rate * dt[t])[:, None, None] * S + (dt[t][:, None] * b[t])[:, :, None] * x[t][:, None, :]
+        y[t] = torch.einsum("hnv,hn->hv", S, c[t]) + skip[:, None] * x[t]
+    return y, S
+
+
+@pytest.mark.parametrize("heads,groups,state,vdim,slice_dim", [
+    (4, 2, 16, 16, 16), (3, 1, 16, 64, 64), (2, 2, 32, 32, 32), (4, 1, 32, 48, 16), (6, 3, 64, 64, 64), (2, 1, 64, 64, 32), (3, 3, 64, 32, 16),
+    (2, 1, 128, 64, 64), (4, 2, 128, 128, 64), (2, 1, 128, 96, 32), (1, 1, 128, 16, 16), (2, 1, 256, 64, 64), (2, 2, 256, 32, 32)])
+def test_recurrence_in_chunks_on_the_tensor_cores(heads, groups, state, vdim, slice_dim):
+    """Six requests side by side of 1 to 200 tokens (chunk borders on both sides), states that are not zero at the start,
+    fast and slow heads, slots in another order than the requests; outputs and states against a walk in float64, to far
+    below what a bfloat16 rounding of state, decays or step sizes would leave."""
+    g = torch.Generator().manual_seed(state + vdim)
+    lens = [64, 1, 65, 200, 63, 2]
+    slots = [3, 0, 6, 2, 5, 1]
+    T, N, channels = sum(lens), state, heads * vdim + 2 * groups * state
+    rows = torch.randn(T, channels, generator=g).to(torch.bfloat16)
+    pre = torch.randn(T, heads, generator=g)
+    rate_log, bias, skip = (torch.randn(heads, generator=g) * 1.5 - off for off in (1.0, 1.0, 0.0))
+    init = torch.randn(7, heads * N * vdim + 6, generator=g)
+    st = init.cuda().clone()
+    out = torch.full((T, heads * vdim), float("nan"), device="cuda")
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")     # noqa: E731
+    starts = [sum(lens[:i]) for i in range(len(lens))]
+    dev = rows.cuda()
+    hv, gn = heads * vdim, groups * N
+    args = (dev[:, hv + gn:], dev[:, hv:hv + gn], dev[:, :hv], pre.cuda(), rate_log.cuda(), bias.cuda(), skip.cuda())
+    ops.state_space_chunks(out, *args, st, i32(slots), i32(starts), i32(lens), len(lens), heads, N, vdim, heads // groups, True, slice_dim=slice_dim)
+    kept = init.cuda().clone()
+    again = torch.empty_like(out)
+    ops.state_space_chunks(again, *args, kept, i32(slots), i32(starts), i32(lens), len(lens), heads, N, vdim, heads // groups, False, slice_dim=slice_dim)
+    assert torch.equal(again, out) and torch.equal(kept.cpu(), init)              # without the write the slots stay as they were
+    d = rows.double()
+    x, b, c = d[:, :hv].view(T, heads, vdim), d[:, hv:hv + gn].view(T, groups, N), d[:, hv + gn:].view(T, groups, N)
+    b, c = (t.repeat_interleave(heads // groups, dim=1) for t in (b, c))
+    dt = plain.softplus(pre.double() + bias.double())
+    got, got_state = out.cpu().double(), st.cpu().double()
+    for n, slot, at in zip(lens, slots, starts):
+        one = slice(at, at + n)
+        S0 = init[slot, :heads * N * vdim].double().view(heads, N, vdim)
+        y, S = walk_by_hand(x[one], b[one], c[one], dt[one], torch.exp(rate_log.double()), skip.double(), S0)
+        for h in range(heads):
+            scale = float(y[:, h].abs().max())
+            assert float((got[one].view(n, heads, vdim)[:, h] - y[:, h]).abs().max()) <= 1e-4 * scale, (n, h)
+            state_got = got_state[slot, :heads * N * vdim].view(heads, N, vdim)[h]
+            assert float((state_got - S[h]).abs().max()) <= 1e-4 * float(S[h].abs().max()), (n, h)
+        assert torch.equal(got_state[slot, heads * N * vdim:], init[slot, heads * N * vdim:].double())     # what lies behind the heads
+    assert torch.equal(got_state[4], init[4].double())                           # nobody's slot
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("vdim,state", [(16, 16), (64, 128), (64, 64), (32, 32)])
 @pytest.mark.parametrize("loud_row", [0, 3, 149])
@@ -264,8 +324,40 @@ def test_state_keeps_one_token_from_far_back(dtype, vdim, state, loud_row):
     set_weight(mixer, w, "dt_bias", torch.full((heads,), -1.0))
     set_weight(mixer, w, "D", torch.zeros(heads))
     wd = {k: v.double() for k, v in named(w).items()}
-    run_state_mixer(rt, mixer, hidden, lambda h, pos: plain.mixer_mamba2(h, wd, "p.", layer["mixer"], 1e-5), loud_row=loud_row,
-                    bf16=6e-2)                # (what rounding the projected rows to bfloat16 does to the plain mixer here: 4 %)
+    run_state_mixer(rt, mixer, hidden, lambda h, pos: plain.mixer_mamba2(h, wd, "p.", layer["mixer"], 1e-5, stored_as(dtype)),
+                    loud_row=loud_row, bf16=1.5e-2)
+
+
+@pytest.mark.parametrize("channels,taps,with_bias", [(256, 4, True), (1032, 3, True), (64, 2, False), (40, 4, True), (2056, 4, False), (48, 1, True), (20, 4, True)])
+@pytest.mark.parametrize("out_dtype", DTYPES)
+def test_convolution_over_mixed_rows(channels, taps, with_bias, out_dtype):
+    """bfloat16 rows of nine requests of 1 to 70 rows with padding rows in between, every request with inputs kept from
+    before; single rows move their state on.  Channels in eights (16-byte accesses) and not."""
+    g = torch.Generator().manual_seed(channels + taps)
+    lens = [1, 2, 3, 17, 1, 70, 4, 33, 1]
+    rows, seq_of, starts = [], [], []
+    for i, n in enumerate(lens):
+        starts.append(len(seq_of))
+        seq_of += [i] * n + [-1] * (i % 3)
+    T = len(seq_of)
+    x = torch.randn(T, channels + 8, generator=g).to(torch.bfloat16)
+    w, bias = torch.randn(channels, taps, generator=g), torch.randn(channels, generator=g) if with_bias else None
+    slots = [8, 3, 5, 0, 7, 1, 6, 2, 4]
+    state = torch.randn(9, 5 + channels * (taps - 1), generator=g)
+    st = state.cuda().clone()
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")     # noqa: E731
+    out = torch.full((T, channels), float("nan"), dtype=out_dtype, device="cuda")
+    dev = x.cuda()
+    ops.short_conv(out, dev[:, 8:], w.cuda(), st, 5, i32(seq_of), i32(slots), i32(starts), T, move_single=i32(lens),
+                   bias=None if bias is None else bias.cuda())
+    got, after = out.float().cpu(), st.cpu()
+    for n, slot, at in zip(lens, slots, starts):
+        kept = state[slot, 5:].view(channels, taps - 1).T.double()
+        seq = torch.cat([kept, x[at:at + n, 8:].double()])
+        y = sum(seq[j:j + n] * w[:, j].double() for j in range(taps)) + (0 if bias is None else bias.double())
+        close(got[at:at + n], plain.silu(y).float(), out_dtype, f"request of {n} rows", bf16=5e-3)
+        want = seq[1:].T.reshape(-1).float() if n == 1 and taps > 1 else state[slot, 5:]
+        assert torch.equal(after[slot, 5:], want) and torch.equal(after[slot, :5], state[slot, :5])
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -301,8 +393,8 @@ def test_decays_at_their_extremes(dtype, extreme):
     a, b = {"fast": (5.0, 3.0), "slow": (-12.0, -6.0), "large": (-1.0, 100.0)}[extreme]
     set_weight(mixer, w, "A_log", torch.tensor([a, a - 2.0])); set_weight(mixer, w, "dt_bias", torch.tensor([b, b + 0.5]))
     wd = {k: v.double() for k, v in named(w).items()}
-    run_state_mixer(rt, mixer, hidden, lambda h, pos: plain.mixer_mamba2(h, wd, "p.", layer["mixer"], 1e-5),
-                    bf16=0.1)                 # (what rounding the projected rows to bfloat16 does to the plain mixer here: 7 %)
+    run_state_mixer(rt, mixer, hidden, lambda h, pos: plain.mixer_mamba2(h, wd, "p.", layer["mixer"], 1e-5, stored_as(dtype)),
+                    bf16=1.5e-2)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
