@@ -28,7 +28,7 @@
 // Every wait on an mbarrier is bounded; a wait that runs out sets TW_ERR_WAIT in the status
 // word, every role stops, the block waits (bounded) for its copies in flight, frees its tensor
 // memory and returns.
-#include "tcgen05.cuh"
+#include "tcgen05_softmax.cuh"
 
 #ifndef TW_HEAD_DIM
 #define TW_HEAD_DIM 128
@@ -76,40 +76,6 @@ __device__ long long g_trace[TRACE_ROLES * TRACE_TILES * TRACE_SLOTS];
 #else
 #define TW_TRACE_AT(role, tile, slot) do {} while (0)
 #endif
-
-__device__ __forceinline__ float ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float max3(float a, float b, float c) {
-    float d;
-    asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-    return d;
-}
-// (a0, a1) * b + c and (a0, a1) + (b0, b1) as one packed instruction each
-__device__ __forceinline__ float2 fma2(float a0, float a1, float b, float c) {
-    float2 d;
-    asm("{\n\t.reg .b64 ra, rb, rc, rd;\n\t"
-        "mov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %4};\n\tmov.b64 rc, {%5, %5};\n\t"
-        "fma.rn.f32x2 rd, ra, rb, rc;\n\t"
-        "mov.b64 {%0, %1}, rd;\n\t}"
-        : "=f"(d.x), "=f"(d.y) : "f"(a0), "f"(a1), "f"(b), "f"(c));
-    return d;
-}
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-    float2 d;
-    asm("{\n\t.reg .b64 ra, rb, rd;\n\t"
-        "mov.b64 ra, {%2, %3};\n\tmov.b64 rb, {%4, %5};\n\t"
-        "add.rn.f32x2 rd, ra, rb;\n\t"
-        "mov.b64 {%0, %1}, rd;\n\t}"
-        : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
-    return d;
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<uint32_t*>(&v);
-}
 
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,

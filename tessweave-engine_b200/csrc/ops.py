@@ -808,12 +808,21 @@ def prefer_tcgen05_attention(dtype: torch.dtype, head_dim: int, page_size: int, 
     return max_q_len >= TCGEN05_ATTENTION_MIN_TOKENS
 
 
-def decode_splits(n_seqs: int, n_kv_heads: int, group: int, max_kv_len: int) -> int:
+def decode_blocks_per_sm(v_dim: int) -> int:
+    """How many blocks of the split-KV kernel that loads keys through registers an SM holds: four, or as many as the
+    shared memory of their value stages (three stages of 64 padded rows) leaves room for."""
+    return max(1, min(4, 227 * 1024 // (3 * 64 * (v_dim + 8) * 2 + 4096)))
+
+
+def decode_splits(n_seqs: int, n_kv_heads: int, group: int, max_kv_len: int, v_dim: int = 128) -> int:
     """How many slices the keys of a request are cut into, so that the launch fills the GPU.
     Up to 16 slices merge inside a thread-block cluster, which saves 2-3 us over the merge through
     scratch memory; clusters of 15 and 16 are only placed well when there are few of them, so with many
     (request, head) groups 15 and 16 slices become 14 (measured on B200, batch 8, 4 key/value heads,
-    4096 keys, a whole decode step: 3.61 ms with 13 or 14 slices, 3.64 with 12, 3.94 with 16, 4.02 with 15)."""
+    4096 keys, a whole decode step: 3.61 ms with 13 or 14 slices, 3.64 with 12, 3.94 with 16, 4.02 with 15).
+    Values of more than 128 leave fewer blocks on an SM, and a launch of more blocks than fit at once pays for every
+    further one (28 heads over cached rows of 256 values, batch 8, 4,096 keys, the kernel alone: 29.6 us with 8 slices on
+    256 blocks, 46 to 62 with 9 to 16)."""
     import os
     forced = os.environ.get("TESSWEAVE_DECODE_SPLITS")
     if forced:
@@ -821,17 +830,18 @@ def decode_splits(n_seqs: int, n_kv_heads: int, group: int, max_kv_len: int) -> 
     head_tiles = (group + 7) // 8
     tiles = max(1, -(-max_kv_len // 64))
     groups = max(1, n_seqs * n_kv_heads * head_tiles)
-    # the kernel fits four blocks on an SM; aim at a little under one full wave of blocks
-    room = 7 * _SM_COUNT // 2
+    # the kernel fits four blocks on an SM (fewer with wide values); aim at a little under one full wave of blocks
+    fits = decode_blocks_per_sm(v_dim)
+    room, full = 7 * fits * _SM_COUNT // 8, 15 * fits * _SM_COUNT // 16
     target = max(1, (room + groups // 2) // groups)        # rounded: 1.9 blocks' worth of room is two slices
     if target > 4 and target * groups > room:
         # clusters of five and more blocks are no longer all placed at once when the launch has more than 3.5 blocks
         # per SM (batch 12, 4 key/value heads, a whole decode step: 3.81 ms with 10 slices, 4.21 with 11)
         target = max(4, room // groups)
-    elif 1 < target <= 4 and target * groups > 15 * _SM_COUNT // 4:
+    elif 1 < target <= 4 and target * groups > full:
         # small clusters fill the SMs a little further (batch 44: 528 blocks of 3 slices, 5.23 ms against 5.51 with 2),
         # but not to the last slot (batch 48: 576 blocks, 6.56 ms against 5.59 with 2)
-        target = max(1, (15 * _SM_COUNT // 4) // groups)
+        target = max(1, full // groups)
     nsplit = max(1, min(tiles, target, 128, DECODE_SCRATCH_UNITS // max(1, n_seqs)))
     if 16 < nsplit <= 64 and max_kv_len <= 8192:
         # up to 8,192 keys the merge inside a cluster beats more slices merged through scratch memory (4,096 keys:
@@ -1183,6 +1193,50 @@ def attention_prefill_tcgen05(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_sl
         c_int(n_seqs), c_int(max_q_len), c_int(n_q_heads), c_int(n_kv_heads), c_int(k_pages.shape[2]),
         c_int(k_pages.shape[0]), c_int(window), c_float(scale), c_int(1 if skip_single else 0), _ptr(gate), _ptr(status), _stream())
     _check(code, "attention_prefill_tcgen05")
+
+
+LATENT_TCGEN05_MIN_TOKENS = 64
+
+
+def latent_tcgen05_key_tile(page_size: int) -> int | None:
+    """Keys per tile of the latent tcgen05 attention for pages of this size, or None: a tile is a whole number of pages (at
+    most 32), or a page a whole number of tiles."""
+    if page_size >= 4 and 96 % page_size == 0:
+        return 96
+    return 64 if page_size >= 4 and page_size % 64 == 0 else None
+
+
+def prefer_latent_tcgen05(dtype: torch.dtype, head_dim: int, page_size: int, max_q_len: int) -> bool:
+    """Whether a step whose longest portion has ``max_q_len`` tokens runs attention whose values are the keys on the tcgen05
+    kernel: bfloat16 and cached rows in multiples of 16 values up to 256.  TESSWEAVE_PREFILL_ATTENTION=mma|tcgen05 forces one
+    of the two (the latter only for shapes the kernel takes)."""
+    import os
+    if dtype != torch.bfloat16 or head_dim % 16 or not 16 <= head_dim <= 256 or latent_tcgen05_key_tile(page_size) is None:
+        return False
+    forced = os.environ.get("TESSWEAVE_PREFILL_ATTENTION")
+    if forced in ("mma", "tcgen05"):
+        return forced == "tcgen05"
+    return max_q_len >= LATENT_TCGEN05_MIN_TOKENS
+
+
+def attention_latent_tcgen05(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, pages, n_seqs, max_q_len, n_q_heads,
+                             n_kv_heads, head_dim, v_cols, window, scale, skip_single, status, sink: torch.Tensor | None = None,
+                             gate: torch.Tensor | None = None) -> None:
+    """Prompt attention whose values are the leading ``v_cols`` values of the keys, on the tcgen05 tensor cores
+    (csrc/attention_latent_tcgen05.cu).  Of a head's ``head_dim`` outputs the first ``v_cols`` (rounded up to 16) are
+    written.  ``sink``, ``gate`` and ``window`` as for ``attention_decode``."""
+    _cuda(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, pages, status, sink, gate)
+    _gate_check(gate, 0, n_q_heads)
+    _attn_common_checks(out, q, block_table, pages, pages, n_q_heads, n_kv_heads, head_dim)
+    _score_terms_checks(sink, None, n_q_heads)
+    tile = latent_tcgen05_key_tile(pages.shape[2])
+    _need(tile is not None and 0 < v_cols <= head_dim and scale > 0, "attention_latent_tcgen05: a page size, value columns or a scale the kernel does not take")
+    code = _fn("attention_latent_tcgen05", "tw_attn_latent_tc5", {"TW_HEAD_DIM": head_dim, "TW_V_COLS": -(-v_cols // 16) * 16, "TW_KEY_TILE": tile})(
+        _ptr(out), c_int(out.stride(0)), _ptr(q), c_int(q.stride(0)), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(seq_slot),
+        _ptr(block_table), c_int(block_table.shape[1]), _ptr(pages), c_int(n_seqs), c_int(max_q_len), c_int(n_q_heads), c_int(n_kv_heads),
+        c_int(pages.shape[2]), c_int(pages.shape[0]), c_int(window), c_float(scale), c_int(1 if skip_single else 0), _ptr(sink), _ptr(gate),
+        _ptr(status), _stream())
+    _check(code, "attention_latent_tcgen05")
 
 
 def attention_prefill(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, k_pages, v_pages, n_seqs,
@@ -1971,12 +2025,12 @@ def short_conv(out: torch.Tensor, x: torch.Tensor, w: torch.Tensor, state: torch
     _need(out.dtype in (torch.float32, x.dtype) and out.is_contiguous() and out.shape[1] == channels and out.shape[0] >= n_rows,
           "short_conv: the result must be contiguous [rows, channels], in fp32 or x's type")
     _need(x.stride(1) == 1 and x.shape[1] >= channels and x.shape[0] >= n_rows, "short_conv: bad input rows")
-    _need(w.dtype == torch.float32 and w.is_contiguous() and 1 <= taps <= SHORT_CONV_MAX_TAPS, "short_conv: taps must be fp32 [channels, 1..17]")
+    _need(w.dtype == torch.float32 and 1 <= taps <= SHORT_CONV_MAX_TAPS, "short_conv: taps must be fp32 [channels, 1..17]")
     _need(state.dtype == torch.float32 and state.dim() == 2 and state.stride(1) == 1
           and state_offset + channels * (taps - 1) <= state.shape[1], "short_conv: the state must be fp32 [slots, numel] with room for the taps")
     _need(0 <= scaled_heads <= unit_heads and unit_heads * unit_dim <= channels, "short_conv: the unit heads exceed the channels")
     code = _fn("recurrent", "tw_short_conv")(
-        _ptr(out), _ptr(x), c_int(x.stride(0)), _ptr(w), _ptr(bias), c_int(taps), _ptr(state), ctypes.c_longlong(state.stride(0)),
+        _ptr(out), _ptr(x), c_int(x.stride(0)), _ptr(w), c_int(w.stride(0)), c_int(w.stride(1)), _ptr(bias), c_int(taps), _ptr(state), ctypes.c_longlong(state.stride(0)),
         ctypes.c_longlong(state_offset), _ptr(seq_of_token), _ptr(seq_slot), _ptr(seq_q_start), _ptr(move_single),
         c_int(0 if move_single is None else 1), c_int(n_rows), c_int(channels),
         c_int(unit_heads), c_int(unit_dim), c_int(scaled_heads), c_float(head_scale), c_float(unit_eps), c_int(dtype_code(x.dtype)),

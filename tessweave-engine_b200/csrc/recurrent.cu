@@ -431,7 +431,7 @@ TW_EXPORT int tw_tanh_rows(void* x, long long count, int dtype, cudaStream_t str
 
 // ---------------------------------------------------------------------------
 // Short causal convolution over time, per channel, with silu, for the packed rows a recurrence reads:
-//   y[t, c] = silu(bias[c] + sum_j w[c, j] x[t - (taps - 1) + j, c])  (bias may be null),   the last tap is the row's own, zeros before a request's start.
+//   y[t, c] = silu(bias[c] + sum_j w[c, j] x[t - (taps - 1) + j, c])  (bias may be null; w[c, j] at w[c * w_c + j * w_j]),   the last tap is the row's own, zeros before a request's start.
 // The taps - 1 rows before a request's first row of this step come from the request's state (fp32, channel-major:
 // state[offset + c * (taps - 1) + j], j = 0 the oldest), which tw_short_conv_state moves on afterwards.  Behind the
 // convolution the first `unit_heads` heads of `unit_dim` channels are scaled to unit length, x / sqrt(sum x^2 + unit_eps),
@@ -439,7 +439,7 @@ TW_EXPORT int tw_tanh_rows(void* x, long long count, int dtype, cudaStream_t str
 // ---------------------------------------------------------------------------
 template <typename T, typename OT>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, const float* __restrict__ bias, int taps,
+short_conv_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, int w_c, int w_j, const float* __restrict__ bias, int taps,
                   float* __restrict__ state, long long state_stride, long long state_offset,
                   const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                   const int* __restrict__ seq_q_len, int move_single, int channels, int chunk, int unit_heads, int unit_dim,
@@ -463,7 +463,7 @@ short_conv_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, c
         for (int j = 0; j < taps; ++j) {
             const int back = taps - 1 - j;               // how many rows before this one
             const float xv = back <= r ? tw_to_float(x[(size_t)(row - back) * x_stride + c]) : tc[taps - 1 + r - back];
-            acc += w[(size_t)c * taps + j] * xv;
+            acc += w[(size_t)c * w_c + (size_t)j * w_j] * xv;
             if (move && j > 0) tc[j - 1] = xv;           // r == 0: xv is input j of (state, own row); place j - 1 has been read
         }
         sy[c - c0] = acc / (1.0f + expf(-acc));
@@ -494,7 +494,7 @@ short_conv_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, c
 #define TW_CONV_ROWS 8
 template <typename T, typename OT, int TAPS>
 __global__ void __launch_bounds__(256)
-short_conv_rows_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w,
+short_conv_rows_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stride, const float* __restrict__ w, int w_c, int w_j,
                        const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
                        const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                        const int* __restrict__ seq_q_len, int move_single, int n_rows, int channels, int chunk, int unit_heads,
@@ -509,7 +509,7 @@ short_conv_rows_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stri
     for (int c = c0 + threadIdx.x; c < c1; c += blockDim.x) {
         float wt[TAPS], xw[TAPS];
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[j] = w[(size_t)c * TAPS + j];
+        for (int j = 0; j < TAPS; ++j) wt[j] = w[(size_t)c * w_c + (size_t)j * w_j];
         const float b = bias ? bias[c] : 0.f;
         // xw[j] is the input TAPS - 1 - j rows before the current one (whichever request that row belongs to)
 #pragma unroll
@@ -586,7 +586,7 @@ __device__ __forceinline__ void tw_unpack8(uint4 raw, float (&f)[8]) {
 template <int TAPS>
 __global__ void __launch_bounds__(TW_CONV_WIDE_THREADS)
 short_conv_wide_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x, int x_stride, const float* __restrict__ w,
-                       const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
+                       int w_c, int w_j, const float* __restrict__ bias, float* __restrict__ state, long long state_stride, long long state_offset,
                        const int* __restrict__ seq_of_token, const int* __restrict__ seq_slot, const int* __restrict__ seq_q_start,
                        const int* __restrict__ seq_q_len, int move_single, int n_rows, int channels) {
     constexpr int R = TW_CONV_WIDE_ROWS, P = TAPS - 1;
@@ -595,13 +595,13 @@ short_conv_wide_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __r
     const int c = (blockIdx.y * TW_CONV_WIDE_THREADS + threadIdx.x) * 8;
     if (c >= channels) return;
     const int row0 = blockIdx.x * R, nr = min(R, n_rows - row0);
-    float wt[8][TAPS], b[8];
+    float wt[8][TAPS], b[8];             // (with w_c == 1, a tap's weights side by side, neighbouring threads read neighbouring lines)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
+    for (int j = 0; j < TAPS; ++j)
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c + e) * TAPS + j];
-        b[e] = bias ? bias[c + e] : 0.f;
-    }
+        for (int e = 0; e < 8; ++e) wt[e][j] = w[(size_t)(c + e) * w_c + (size_t)j * w_j];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) b[e] = bias ? bias[c + e] : 0.f;
     uint4 xr[P + R];                     // the rows before (whichever request they belong to), then the block's own
 #pragma unroll
     for (int i = 0; i < P + R; ++i) {
@@ -637,7 +637,7 @@ short_conv_wide_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __r
             acc[e] = b[e];
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) acc[e] += wt[e][j] * in[j][e];
-            acc[e] = acc[e] / (1.0f + expf(-acc[e]));
+            acc[e] = __fdividef(acc[e], 1.0f + __expf(-acc[e]));         // (rounded to bf16 next)
         }
         uint4 packed;
         __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&packed);
@@ -671,7 +671,7 @@ __global__ void short_conv_state_kernel(const T* __restrict__ x, int x_stride, i
 }
 
 template <typename T, typename OT>
-static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, const float* bias, int taps, float* state, long long state_stride,
+static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, int w_c, int w_j, const float* bias, int taps, float* state, long long state_stride,
                              long long state_offset, const int* seq_of_token, const int* seq_slot, const int* seq_q_start,
                              const int* seq_q_len, int move_single, int n_rows, int channels, int unit_heads, int unit_dim,
                              int scaled_heads, float head_scale, float unit_eps, cudaStream_t stream) {
@@ -680,7 +680,7 @@ static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, 
             && (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
             const dim3 wgrid((n_rows + TW_CONV_WIDE_ROWS - 1) / TW_CONV_WIDE_ROWS, (channels / 8 + TW_CONV_WIDE_THREADS - 1) / TW_CONV_WIDE_THREADS);
 #define TW_CONV_WIDE_LAUNCH(TAPS)                                                                                                 \
-            return tw_launch(short_conv_wide_kernel<TAPS>, wgrid, dim3(TW_CONV_WIDE_THREADS), 0, stream, 1, out, x, x_stride, w, bias,  \
+            return tw_launch(short_conv_wide_kernel<TAPS>, wgrid, dim3(TW_CONV_WIDE_THREADS), 0, stream, 1, out, x, x_stride, w, w_c, w_j, bias,  \
                              state, state_stride, state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels);
             if (taps == 2) { TW_CONV_WIDE_LAUNCH(2) }
             if (taps == 3) { TW_CONV_WIDE_LAUNCH(3) }
@@ -706,7 +706,7 @@ static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, 
                                                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)rsmem);             \
                 if (e != cudaSuccess) return (int)e;                                                                             \
             }                                                                                                                    \
-            return tw_launch(short_conv_rows_kernel<T, OT, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, bias, state, \
+            return tw_launch(short_conv_rows_kernel<T, OT, TAPS>, rgrid, dim3(256), rsmem, stream, 1, out, x, x_stride, w, w_c, w_j, bias, state, \
                              state_stride, state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows,   \
                              channels, chunk, unit_heads, unit_dim, scaled_heads, head_scale, unit_eps);                         \
         }
@@ -719,14 +719,14 @@ static int launch_short_conv(OT* out, const T* x, int x_stride, const float* w, 
 #undef TW_CONV_ROWS_LAUNCH
     }
     const dim3 grid(n_rows, (channels + chunk - 1) / chunk);
-    return tw_launch(short_conv_kernel<T, OT>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, bias, taps, state, state_stride,
+    return tw_launch(short_conv_kernel<T, OT>, grid, dim3(256), smem, stream, 1, out, x, x_stride, w, w_c, w_j, bias, taps, state, state_stride,
                      state_offset, seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, channels, chunk, unit_heads,
                      unit_dim, scaled_heads, head_scale, unit_eps);
 }
 
 // seq_q_len with move_single: requests that bring one row have their state moved on by this kernel (and
 // tw_short_conv_state is then told to skip them).
-TW_EXPORT int tw_short_conv(void* out, const void* x, int x_stride, const float* w, const float* bias, int taps, float* state,
+TW_EXPORT int tw_short_conv(void* out, const void* x, int x_stride, const float* w, int w_c, int w_j, const float* bias, int taps, float* state,
                             long long state_stride, long long state_offset, const int* seq_of_token, const int* seq_slot,
                             const int* seq_q_start, const int* seq_q_len, int move_single, int n_rows, int channels,
                             int unit_heads, int unit_dim, int scaled_heads, float head_scale, float unit_eps, int dtype,
@@ -734,14 +734,14 @@ TW_EXPORT int tw_short_conv(void* out, const void* x, int x_stride, const float*
     if (n_rows <= 0 || channels <= 0) return 0;
     if (taps < 1 || taps > 17 || unit_heads * unit_dim > channels || (move_single && !seq_q_len)) return (int)cudaErrorInvalidValue;
     if (dtype == TW_F32)
-        return out_dtype != TW_F32 ? (int)cudaErrorInvalidValue : launch_short_conv<float, float>((float*)out, (const float*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token,
+        return out_dtype != TW_F32 ? (int)cudaErrorInvalidValue : launch_short_conv<float, float>((float*)out, (const float*)x, x_stride, w, w_c, w_j, bias, taps, state, state_stride, state_offset, seq_of_token,
                                         seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels, unit_heads, unit_dim,
                                         scaled_heads, head_scale, unit_eps, stream);
     if (out_dtype != TW_F32)
         return launch_short_conv<__nv_bfloat16, __nv_bfloat16>(
-            (__nv_bfloat16*)out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset, seq_of_token, seq_slot,
+            (__nv_bfloat16*)out, (const __nv_bfloat16*)x, x_stride, w, w_c, w_j, bias, taps, state, state_stride, state_offset, seq_of_token, seq_slot,
             seq_q_start, seq_q_len, move_single, n_rows, channels, unit_heads, unit_dim, scaled_heads, head_scale, unit_eps, stream);
-    return launch_short_conv<__nv_bfloat16, float>((float*)out, (const __nv_bfloat16*)x, x_stride, w, bias, taps, state, state_stride, state_offset,
+    return launch_short_conv<__nv_bfloat16, float>((float*)out, (const __nv_bfloat16*)x, x_stride, w, w_c, w_j, bias, taps, state, state_stride, state_offset,
                                             seq_of_token, seq_slot, seq_q_start, seq_q_len, move_single, n_rows, channels,
                                             unit_heads, unit_dim, scaled_heads, head_scale, unit_eps, stream);
 }

@@ -11,6 +11,7 @@ COMMON_HEAD_DIMS = (16, 32, 64, 128)
 _SPECIALISED: dict[str, list[dict]] = {
     "attention_bf16": [{"TW_HEAD_DIM": d} for d in COMMON_HEAD_DIMS] + [{"TW_HEAD_DIM": 2 * v, "TW_V_DIM": v} for v in (32, 64)],
     "attention_tcgen05": [{"TW_HEAD_DIM": d} for d in (64, 128)] + [{"TW_HEAD_DIM": 2 * v, "TW_V_DIM": v} for v in (32, 64)],
+    "attention_latent_tcgen05": [{"TW_HEAD_DIM": d, "TW_V_COLS": v, "TW_KEY_TILE": 96} for d, v in ((256, 192), (128, 96))],
     "attention_decode_tma": [{"TW_HEAD_DIM": d} for d in (64, 128)] + [{"TW_HEAD_DIM": 128, "TW_V_DIM": 64}],
     "sigmoid_attention_bf16": [{"TW_HEAD_DIM": d} for d in (64, 128)],
     "sigmoid_attention_tcgen05": [{"TW_HEAD_DIM": d, "TW_SIG_KEY_TILE": 128} for d in (64, 128)],

@@ -39,17 +39,23 @@ class PagedSoftmaxMixer(Mixer):
         """(fed by TMA?, slices per request, blocks) of the decode attention this step will launch."""
         group = self.n_heads // self.n_kv_heads
         tma = not self.score_terms and ops.decode_tma_supported(self.runtime.dtype, self.head_dim, cache.page_size, self.v_dim)
-        splits = ops.decode_tma_splits if tma else ops.decode_splits
         # (the keys a request can see: a window or a chunk bounds them, and the kernels cut those into the slices)
-        nsplit = splits(ctx.n_seqs, self.n_kv_heads, group, min(ctx.max_kv_len, self.span) if self.span else ctx.max_kv_len)
+        seen = min(ctx.max_kv_len, self.span) if self.span else ctx.max_kv_len
+        nsplit = (ops.decode_tma_splits(ctx.n_seqs, self.n_kv_heads, group, seen) if tma
+                  else ops.decode_splits(ctx.n_seqs, self.n_kv_heads, group, seen, self.v_dim))
         return tma, nsplit, ctx.n_seqs * self.n_kv_heads * -(-group // 8) * nsplit
+
+    def _prefill_own(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView, gate: torch.Tensor | None,
+                     skip_single: bool) -> bool:
+        """Attention of the step's portions with a kernel of the mixer's own, where it has one for this step."""
+        return False
 
     def _attend_tensor_cores(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView,
                              gate: torch.Tensor | None = None) -> None:
         """bfloat16: flash attention for requests with several tokens, split-KV attention for
         requests with one; both read the same flat batch and skip the other's requests."""
         singles = ctx.decode_only or ctx.fixed_shape or any(n == 1 for n in ctx.host_q_len)
-        if not ctx.decode_only:
+        if not ctx.decode_only and not self._prefill_own(ctx, out, q, cache, gate, singles):
             # long portions: tcgen05 kernel (TMA, accumulators in tensor memory); short ones, and the shapes it
             # does not take, stay on the mma.sync kernel, which starts faster
             prefill = ops.attention_prefill

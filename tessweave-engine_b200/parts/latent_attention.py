@@ -31,7 +31,8 @@ class LatentAttention(PagedSoftmaxMixer):
     last rot_dim values of a result are not used); the head's value map is applied to the attention's result,
     o_h = Wuv_h (sum_j p_j c(j)).  The cache keeps [c | r] per token and nothing else (``values_are_keys``), and the
     paged kernels of the other attention mixers serve this one: exact, mma.sync prefill and split-KV decode (cached
-    rows of more than 256 values: the exact kernel in both run types).
+    rows of more than 256 values: the exact kernel in both run types); long portions have a tcgen05 kernel of their own
+    that copies a tile of rows once and reads it as keys and as values.
 
     The two per-head maps are batched library products.  The first one also moves b_h into place: head h multiplies by
     [[Wuk_h, 0], [0, I]], built once when the weights are in (the identity block copies bit for bit).
@@ -171,6 +172,16 @@ class LatentAttention(PagedSoftmaxMixer):
         if self.gate == "values":
             ops.gate_mul(out, out, proj[:, self.q_rank + self.head_dim:], ops.GATE_SIGMOID, n)
         return out
+
+    def _prefill_own(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView, gate: torch.Tensor | None,
+                     skip_single: bool) -> bool:
+        """Long portions: the tcgen05 kernel that reads a tile of cached rows once, as keys and as values."""
+        if not (self.scale > 0 and ops.prefer_latent_tcgen05(self.runtime.dtype, self.head_dim, cache.page_size, ctx.max_q_len)):
+            return False
+        ops.attention_latent_tcgen05(out, q, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot, cache.block_table,
+                                     cache.k_pages, ctx.n_seqs, ctx.max_q_len, self.n_heads, 1, self.head_dim, self.kv_rank, self.reach,
+                                     self.scale, skip_single, ctx.status, sink=self.sink, gate=gate)
+        return True
 
     def project_out(self, ctx: StepContext, out: torch.Tensor):
         return linear(ctx, "mixer.delta", out, self.w_o, allow_split=True, consumer_early=True)

@@ -493,7 +493,7 @@ class Mamba2(MatrixStateMixer):
         self.state_numel += self.conv_channels * (self.taps - 1)
         self.row_size = self.v_size + self.conv_channels         # [z | x | B | C]
         self.w_in = runtime.empty(self.row_size + n_heads, hidden)
-        self.conv = runtime.empty(self.conv_channels, self.taps, dtype=torch.float32)
+        self.conv = runtime.empty(self.taps, self.conv_channels, dtype=torch.float32).t()      # a tap's weights side by side
         self.conv_bias, self.norm = (runtime.empty(n, dtype=torch.float32) for n in (self.conv_channels, self.v_size))
         self.rate_log, self.dt_bias, self.skip = (runtime.empty(n_heads, dtype=torch.float32) for _ in range(3))
         self.w_o = runtime.empty(hidden, self.v_size)
