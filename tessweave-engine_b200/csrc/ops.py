@@ -1195,7 +1195,7 @@ def attention_prefill_tcgen05(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_sl
     _check(code, "attention_prefill_tcgen05")
 
 
-LATENT_TCGEN05_MIN_TOKENS = 64
+LATENT_TCGEN05_MIN_KEYS = 256
 
 
 def latent_tcgen05_key_tile(page_size: int) -> int | None:
@@ -1206,9 +1206,11 @@ def latent_tcgen05_key_tile(page_size: int) -> int | None:
     return 64 if page_size >= 4 and page_size % 64 == 0 else None
 
 
-def prefer_latent_tcgen05(dtype: torch.dtype, head_dim: int, page_size: int, max_q_len: int) -> bool:
-    """Whether a step whose longest portion has ``max_q_len`` tokens runs attention whose values are the keys on the tcgen05
-    kernel: bfloat16 and cached rows in multiples of 16 values up to 256.  TESSWEAVE_PREFILL_ATTENTION=mma|tcgen05 forces one
+def prefer_latent_tcgen05(dtype: torch.dtype, head_dim: int, page_size: int, max_keys: int) -> bool:
+    """Whether a step with portions whose rows see up to ``max_keys`` keys runs attention whose values are the keys on the
+    tcgen05 kernel: bfloat16 and cached rows in multiples of 16 values up to 256, and enough keys to make up for its later
+    start (28 heads over rows of 256 values: 13.4 us against 9.3 for a prompt of 64 tokens, 15.3 against 18.3 for 256, 40
+    against 103 for a portion of 16 tokens behind 2,048).  TESSWEAVE_PREFILL_ATTENTION=mma|tcgen05 forces one
     of the two (the latter only for shapes the kernel takes)."""
     import os
     if dtype != torch.bfloat16 or head_dim % 16 or not 16 <= head_dim <= 256 or latent_tcgen05_key_tile(page_size) is None:
@@ -1216,7 +1218,7 @@ def prefer_latent_tcgen05(dtype: torch.dtype, head_dim: int, page_size: int, max
     forced = os.environ.get("TESSWEAVE_PREFILL_ATTENTION")
     if forced in ("mma", "tcgen05"):
         return forced == "tcgen05"
-    return max_q_len >= LATENT_TCGEN05_MIN_TOKENS
+    return max_keys >= LATENT_TCGEN05_MIN_KEYS
 
 
 def attention_latent_tcgen05(out, q, seq_q_start, seq_q_len, seq_kv_len, seq_slot, block_table, pages, n_seqs, max_q_len, n_q_heads,
@@ -1601,7 +1603,7 @@ def linear_recurrence(mode: int, out: torch.Tensor, den: torch.Tensor | None, q:
 
 
 STATE_SPACE_CHUNK_STATES = (16, 32, 64, 128, 256)
-STATE_SPACE_CHUNK_MIN_TOKENS = 17       # portions of a chunk of the token-by-token kernel and less stay there
+STATE_SPACE_CHUNK_MIN_TOKENS = 12       # 112 heads of 128 x 64, one request / eight: 7 / 42 us in chunks, token by token 9 / 37 us for 12
 
 
 def state_space_chunks_supported(dtype: torch.dtype, state_dim: int, value_dim: int, channels: int, max_q_len: int) -> bool:

@@ -175,8 +175,9 @@ class LatentAttention(PagedSoftmaxMixer):
 
     def _prefill_own(self, ctx: StepContext, out: torch.Tensor, q: torch.Tensor, cache: PagedView, gate: torch.Tensor | None,
                      skip_single: bool) -> bool:
-        """Long portions: the tcgen05 kernel that reads a tile of cached rows once, as keys and as values."""
-        if not (self.scale > 0 and ops.prefer_latent_tcgen05(self.runtime.dtype, self.head_dim, cache.page_size, ctx.max_q_len)):
+        """Portions with many keys before them: the tcgen05 kernel that reads a tile of cached rows once, as keys and values."""
+        keys = ctx.max_kv_len if self.window is None else min(ctx.max_kv_len, self.window + ctx.max_q_len)
+        if not (self.scale > 0 and ops.prefer_latent_tcgen05(self.runtime.dtype, self.head_dim, cache.page_size, keys)):
             return False
         ops.attention_latent_tcgen05(out, q, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot, cache.block_table,
                                      cache.k_pages, ctx.n_seqs, ctx.max_q_len, self.n_heads, 1, self.head_dim, self.kv_rank, self.reach,

@@ -223,6 +223,69 @@ def test_one_far_key_of_hundreds(dtype, page, cr, r):
             assert err <= (2e-5 if dtype == torch.float32 else 0.1) * size, f"key at {j}, last {tail} tokens alone: {err:.3g} of {size:.3g}"
 
 
+LATENT_TC5 = [  # row, value columns, heads, page, window, portions as (rows of this step, rows held before)
+    (256, 192, 28, 16, None, [(300, 0), (97, 411), (1, 50)]), (128, 96, 6, 16, None, [(129, 1000), (64, 0), (2, 95)]),
+    (64, 48, 16, 8, None, [(200, 13), (33, 190)]), (80, 64, 5, 4, None, [(77, 0), (70, 26)]), (16, 16, 3, 32, None, [(150, 0), (95, 96)]),
+    (48, 32, 1, 48, None, [(400, 5)]), (96, 96, 130, 16, None, [(3, 700), (2, 0)]), (256, 256, 9, 64, None, [(130, 62), (65, 64)]),
+    (192, 176, 40, 128, None, [(66, 190)]), (144, 112, 7, 16, 33, [(200, 300), (96, 0)]), (256, 192, 4, 32, 150, [(290, 410), (96, 96)]),
+    (64, 64, 12, 16, 1, [(100, 37)]), (112, 80, 17, 12, None, [(96, 0), (97, 95)])]
+
+
+@pytest.mark.parametrize("sinks", [False, True])
+@pytest.mark.parametrize("shape", LATENT_TC5)
+def test_latent_attention_on_tcgen05_against_the_exact_kernel(shape, sinks):
+    """Row sizes and value columns off the 64-column blocks, groups of 1 to 130 heads, both key tiles, portions on both
+    sides of a tile's border and behind hundreds of cached rows, windows whose earlier pages are gone (and hold NaN), loud
+    keys in the first and last rows; a single row is left to the decode kernel."""
+    D, DV, H, page, window, portions = shape
+    rt = Runtime(torch.device("cuda"), torch.bfloat16)
+    g = torch.Generator().manual_seed(D + H)
+    lens, held = [n for n, _ in portions], [p for _, p in portions]
+    kv = [n + p for n, p in portions]
+    T = sum(lens)
+    width = max(-(-k // page) for k in kv)
+    per = [-(-k // page) for k in kv]
+    order = torch.randperm(sum(per) + 2, generator=g).tolist()
+    table = torch.full((len(kv) + 1, width), -1, dtype=torch.int32)
+    pages = torch.randn(sum(per) + 2, 1, page, D, generator=g)
+    slots = [len(kv) - i for i in range(len(kv))]
+    at = 0
+    for slot, n, k, p in zip(slots, per, kv, held):
+        mine = order[at:at + n]
+        at += n
+        table[slot, :n] = torch.tensor(mine, dtype=torch.int32)
+        for key in (0, k - 1, max(0, k - 97)):
+            pages[mine[key // page], 0, key % page] *= 3.0
+        pages[mine[-1], 0, (k - 1) % page + 1:] = float("nan")             # behind the last key
+        if window is not None:
+            for blk in range(max(0, p - window + 1) // page):              # given back: nobody may read them
+                pages[mine[blk]] = float("nan")
+                table[slot, blk] = -1
+    q = (torch.randn(T, H * D, generator=g) * 2).to(torch.bfloat16).cuda()
+    pages, table = pages.to(torch.bfloat16).cuda(), table.cuda()
+    sink = (torch.randn(H, generator=g) * 4).cuda() if sinks else None
+    gate = torch.rand(T, H, generator=g).cuda() if sinks else None
+    starts = [sum(lens[:i]) for i in range(len(lens))]
+    positions = [p + i for n, p in portions for i in range(n)]
+    seq_of = [i for i, n in enumerate(lens) for _ in range(n)]
+    ctx = ctx_of(rt, positions, seq_of, slots, starts, lens, kv)
+    exact = torch.zeros(T, H * D, dtype=torch.bfloat16, device="cuda")
+    ops.attention_generic(exact, q, ctx.positions, ctx.seq_of_token, ctx.seq_slot, table, pages, pages, T, H, 1, D,
+                          ops.visible_reach(window, None), D ** -0.5, ctx.status, sink=sink, gate=gate)
+    out = torch.full((T, H * D), 7.0, dtype=torch.bfloat16, device="cuda")
+    ops.attention_latent_tcgen05(out, q, ctx.seq_q_start, ctx.seq_q_len, ctx.seq_kv_len, ctx.seq_slot, table, pages, len(kv), max(lens),
+                                 H, 1, D, DV, ops.visible_reach(window, None), D ** -0.5, True, ctx.status, sink=sink, gate=gate)
+    assert int(ctx.status) == 0
+    got, want = out.float().cpu().view(T, H, D), exact.float().cpu().view(T, H, D)
+    for n, at in zip(lens, starts):
+        rows = slice(at, at + n)
+        if n == 1:
+            assert bool((got[rows] == 7.0).all())
+            continue
+        assert bool((got[rows][:, :, DV:] == 7.0).all())                   # columns that are no values are not written
+        close(got[rows][:, :, :DV], want[rows][:, :, :DV], torch.bfloat16, f"portion of {n}", bf16=1.5e-2)
+
+
 MAMBA_SHAPES = [  # hidden, heads, value size, state, groups, taps, norm parts
     (48, 4, 16, 16, 2, 4, 1), (40, 3, 6, 10, 3, 6, 2), (36, 4, 5, 7, 1, 1, 5), (64, 2, 24, 32, 1, 3, 3), (40, 1, 24, 16, 1, 2, 1),
     (96, 4, 48, 32, 2, 4, 2), (64, 2, 64, 128, 1, 4, 1), (64, 6, 64, 64, 3, 4, 2), (64, 4, 32, 48, 2, 5, 4), (40, 2, 40, 96, 1, 4, 8),
