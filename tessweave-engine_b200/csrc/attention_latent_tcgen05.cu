@@ -148,7 +148,7 @@ attn_latent_tc5_kernel(const __grid_constant__ CUtensorMap map, bf16* __restrict
     // the block's query rows into the swizzled K-major layout (rows beyond the portion, and columns beyond D, are zero)
     {
         constexpr int CH = KB * 8, ITEMS = BM * CH, QT = THREADS - 32;
-        constexpr int PER = (ITEMS + QT - 1) / QT, GROUP = 8;
+        constexpr int PER = (ITEMS + QT - 1) / QT, GROUP = PER < 14 ? PER : 14;
         for (int j0 = 0; warp != 0 && j0 < PER; j0 += GROUP) {
             uint4 vals[GROUP];
 #pragma unroll

@@ -573,7 +573,7 @@ short_conv_rows_kernel(OT* __restrict__ out, const T* __restrict__ x, int x_stri
 
 // bf16 in and out, no unit heads, four taps or fewer, channels in groups of eight on 16-byte boundaries: a thread serves
 // eight channels of TW_CONV_WIDE_ROWS consecutive rows with 16-byte accesses, the inputs of the rows before in registers.
-#define TW_CONV_WIDE_ROWS 16
+#define TW_CONV_WIDE_ROWS 8
 #define TW_CONV_WIDE_THREADS 128
 __device__ __forceinline__ void tw_unpack8(uint4 raw, float (&f)[8]) {
     const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
