@@ -7,7 +7,7 @@
 //                    gate of an expert that every token uses.  With `scoring` 1: s = softmax(z) over every router
 //                    output, the `top` largest s + correction are chosen, and their weights are s * weight_scale
 //                    (not renormalised); with `scoring` 2 their weights are s / (sum of the chosen s + 1e-20) * weight_scale.
-//                    With `group_count` > 0 the outputs form that many equal groups of neighbours; a group counts as much
+//                    With `group_count` > 0 the outputs form that many groups of consecutive outputs; a group counts as much
 //                    as its best output, and only outputs of the best `group_keep` groups may be chosen
 //   tw_moe_gate_up   act[token, j] = silu(Wg_e h) * (Wu_e h)          e = the j-th expert of the token
 //                    with `act` 1: g = min(Wg_e h, limit), u = clamp(Wu_e h, -limit, limit), g sigmoid(alpha g) (u + 1)

@@ -1794,7 +1794,7 @@ def moe_route(chosen: torch.Tensor, weight: torch.Tensor, shared_gate: torch.Ten
     softmax over those logits alone (fp32 [rows, top]), and ``sigmoid(w_shared_gate . h)`` (fp32 [rows]) if asked.
     With ``score_all`` the scores are the softmax over every router output, the choice goes by score + ``correction``
     (fp32 [outputs], may be None) and the weights are the chosen scores times ``weight_scale``, not renormalised -- or, with ``renormalise``, the chosen scores over their
-    sum (+ 1e-20) times ``weight_scale``.  ``groups`` = (count, keep): the outputs form ``count`` equal groups of neighbours
+    sum (+ 1e-20) times ``weight_scale``.  ``groups`` = (count, keep): the outputs form ``count`` groups of as many consecutive outputs
     and only those of the ``keep`` groups with the largest best score may be chosen."""
     _cuda(chosen, weight, shared_gate, h, w_router, b_router, w_shared_gate, correction)
     experts, width = w_router.shape

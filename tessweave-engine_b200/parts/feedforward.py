@@ -173,7 +173,7 @@ class RoutedExperts(FeedForward):
     Options of other designs.  ``score_all``: the scores are s = softmax(z) over *every* router output, the ``top``
     outputs with the largest s + ``correction`` (a stored fp32 vector named by ``correction``, or none) are chosen, and
     the weights are their s times ``weight_scale``, not renormalised; with ``renormalise`` they are divided by their sum
-    (+ 1e-20) first.  ``groups`` (``count``, ``keep``): the outputs form ``count`` equal groups of neighbours, a group counts
+    (+ 1e-20) first.  ``groups`` (``count``, ``keep``): the outputs form ``count`` groups of as many consecutive outputs, a group counts
     as much as its best score, and only outputs of the ``keep`` best groups can be chosen.  ``identity`` n: the router has n outputs more
     than there are experts; such an output is an expert without tensors whose result is the token's row itself.
     ``activation``: ``{"kind": "clamped", "limit": l, "alpha": a}`` makes an expert's inner rows
